@@ -11,7 +11,7 @@ architecture's typed configuration produces a ``ModelSpec`` and the engine build
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional, Tuple
+from typing import Any, Dict, List, Optional, Tuple, Union
 
 
 @dataclass(frozen=True)
@@ -71,18 +71,27 @@ class StreamAdd:
 
 
 @dataclass(frozen=True)
+class StreamProject:
+    """What a model puts in the residual stream's place right before an entry of the run order runs: ``W [stream; embedding
+    output]`` with the tensor ``tensor`` (``[hidden, 2 hidden]``, the stream's columns first) and the embedding output of the step's
+    tokens."""
+
+    tensor: str
+
+
+@dataclass(frozen=True)
 class RunEntry:
     """One position in the run order.
 
     ``layer`` indexes ``ModelSpec.layers``.  Every entry owns a cache of its own unless
     ``cache_of`` names an earlier entry (by its index in the run order): then this entry's
     mixer reads that entry's cache and stores nothing.  ``before`` is added to the residual
-    stream ahead of the entry.
+    stream ahead of the entry (``StreamAdd``) or takes its place (``StreamProject``).
     """
 
     layer: int
     cache_of: Optional[int] = None
-    before: Optional[StreamAdd] = None
+    before: Optional[Union[StreamAdd, StreamProject]] = None
 
 
 @dataclass

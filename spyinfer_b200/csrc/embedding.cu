@@ -163,3 +163,36 @@ extern "C" int spy_stream_add(float* stream, const void* table, int table_dtype,
     SPY_CHECK_LAUNCH("stream_add");
     return 0;
 }
+
+// out[t, :] = [stream[t, :] | table[ids[t], :] * scale]: the input of a projection that takes the stream and the embedding output
+// side by side.
+template <typename TW, typename TO>
+__global__ void stream_concat_kernel(const float* __restrict__ stream, const TW* __restrict__ table, const int* __restrict__ ids, float scale,
+                                     TO* __restrict__ out, int hidden, int vocab, int* status)
+{
+    pdl_enter();
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    const bool ok = id >= 0 && id < vocab;
+    if (!ok && threadIdx.x == 0) report_status(status, SPY_STATUS_BAD_TOKEN, t);
+    const float* src = stream + (size_t)t * hidden;
+    TO* dst = out + (size_t)t * 2 * hidden;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        dst[i] = from_f32<TO>(src[i]);
+        dst[hidden + i] = from_f32<TO>(ok ? to_f32(table[(size_t)id * hidden + i]) * scale : 0.f);
+    }
+}
+
+extern "C" int spy_stream_concat(const float* stream, const void* table, int table_dtype, const int* ids, float scale, void* out, int out_dtype, int tokens,
+                                 int hidden, int vocab, int* status, cudaStream_t stream_)
+{
+    if (tokens <= 0) return 0;
+    if (hidden <= 0 || vocab <= 0) SPY_FAIL("stream_concat: hidden %d and vocab %d must be positive", hidden, vocab);
+    SPY_DISPATCH_DTYPE(table_dtype, TW, {
+        SPY_DISPATCH_DTYPE(out_dtype, TO, {
+            spy_launch(stream_concat_kernel<TW, TO>, dim3(tokens), dim3(256), 0, stream_, stream, (const TW*)table, ids, scale, (TO*)out, hidden, vocab, status);
+        })
+    })
+    SPY_CHECK_LAUNCH("stream_concat");
+    return 0;
+}

@@ -12,8 +12,9 @@
 // `identity` of them standing for experts whose output is the token's input itself (the sum of the chosen ones' weights goes
 // to id_weight[t], and the caller adds id_weight[t] * input[t]); a `correction` vector is added to the scores for the CHOICE
 // only (the weights stay the plain scores); the outputs form `group_count` equal groups of neighbours, a group's score is its
-// largest choice score, and only the outputs of the `group_keep` best groups can be chosen.  `act` 1: an expert is
-// weight * silu(gate) * up, without clamps.
+// largest choice score (`group_score` 1: the sum of its two largest), and only the outputs of the `group_keep` best groups can be
+// chosen.  `act` 1: an expert is weight * silu(gate) * up, without clamps.  `score` 1: the scores are sigmoid(logit) instead of a
+// softmax over all outputs.
 #include "common.cuh"
 
 SPY_MODULE(spy_moe)
@@ -27,6 +28,8 @@ struct MoeRouting {
     int act;                       // 0: clamped g * sigmoid(alpha g) * (u + 1); 1: silu(g) * u
     float* id_weight;              // null, or [T]: the sum of the chosen identity experts' weights
     float* shared_weight;          // null, or [T]: the shared expert's weight (sigmoid of its gate's logit)
+    int score;                     // 0: softmax over all outputs; 1: sigmoid of each
+    int group_score;               // 0: a group counts by its largest choice score; 1: by the sum of its two largest
 };
 
 template <typename TA, typename TO>
@@ -43,26 +46,35 @@ __global__ void moe_activation_kernel(const TA* __restrict__ gu, long long gu_ld
     float* kept_w = w_s + total + 1;               // kept_w[e]: the weight if chosen, else 0
     float* choice = kept_w + total;                // the score the choice goes by
     float* group_s = choice + total;
-    // softmax over all outputs
-    float m = -INFINITY;
-    for (int e = tid; e < total; e += blockDim.x) m = fmaxf(m, lg[e]);
-    m = block_max(m, scratch);
-    float s = 0.f;
-    for (int e = tid; e < total; e += blockDim.x) s += expf(lg[e] - m);
-    s = block_sum(s, scratch);
+    // softmax over all outputs, or the sigmoid of each
+    float m = -INFINITY, s = 0.f;
+    if (r.score == 0) {
+        for (int e = tid; e < total; e += blockDim.x) m = fmaxf(m, lg[e]);
+        m = block_max(m, scratch);
+        for (int e = tid; e < total; e += blockDim.x) s += expf(lg[e] - m);
+        s = block_sum(s, scratch);
+    }
     for (int e = tid; e < total; e += blockDim.x) {
-        const float v = expf(lg[e] - m) / s;
+        const float v = r.score == 0 ? expf(lg[e] - m) / s : 1.0f / (1.0f + expf(-lg[e]));
         w_s[e] = v;
         choice[e] = r.correction != nullptr ? v + r.correction[e] : v;
     }
     __syncthreads();
     if (r.group_count > 0) {
-        // a group's score is its largest choice score; a group stays when fewer than group_keep groups beat it
+        // a group's score is its largest choice score, or the sum of its two largest; a group stays when fewer than group_keep groups beat it
         const int per = total / r.group_count;
         for (int g = tid; g < r.group_count; g += blockDim.x) {
-            float best = -INFINITY;
-            for (int e = g * per; e < g * per + per; ++e) best = fmaxf(best, choice[e]);
-            group_s[g] = best;
+            float best = -INFINITY, next = -INFINITY;
+            for (int e = g * per; e < g * per + per; ++e) {
+                const float v = choice[e];
+                if (v > best) {
+                    next = best;
+                    best = v;
+                } else {
+                    next = fmaxf(next, v);
+                }
+            }
+            group_s[g] = r.group_score == 1 && per > 1 ? best + next : best;
         }
         __syncthreads();
         for (int e = tid; e < total; e += blockDim.x) {
@@ -169,6 +181,7 @@ static int run_moe_activation(const void* gu, int gu_dtype, long long gu_ld, con
                                                     || (long long)r.group_keep * (total / r.group_count) < top)))
         SPY_FAIL("moe_activation: %d groups of which %d are kept do not fit %d router outputs and top %d", r.group_count, r.group_keep, total, top);
     if (r.act < 0 || r.act > 1) SPY_FAIL("moe_activation: activation code %d", r.act);
+    if (r.score < 0 || r.score > 1 || r.group_score < 0 || r.group_score > 1) SPY_FAIL("moe_activation: score code %d, group score code %d", r.score, r.group_score);
     const size_t smem = (size_t)(3 * total + 1 + (r.group_count > 0 ? r.group_count : 0)) * sizeof(float);
     const int vec = gu_dtype == SPY_BF16 && y_dtype == SPY_BF16 && ff % 8 == 0 && shared_ff % 8 == 0 && gu_ld % 8 == 0 && y_ld % 8 == 0
                     && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
@@ -186,7 +199,7 @@ extern "C" int spy_moe_activation(const void* gu, int gu_dtype, long long gu_ld,
                                   long long y_ld, int tokens, int experts, int top, int ff, float limit, int shared_ff, float shared_limit, float alpha,
                                   float* weights_out, cudaStream_t stream)
 {
-    MoeRouting r = {0, nullptr, 0, 0, 0, nullptr, nullptr};
+    MoeRouting r = {0, nullptr, 0, 0, 0, nullptr, nullptr, 0, 0};
     return run_moe_activation(gu, gu_dtype, gu_ld, logits, logits_ld, y, y_dtype, y_ld, tokens, experts, top, ff, limit, shared_ff, shared_limit, alpha,
                               weights_out, r, stream);
 }
@@ -196,10 +209,10 @@ extern "C" int spy_moe_activation(const void* gu, int gu_dtype, long long gu_ld,
 extern "C" int spy_moe_activation_routed(const void* gu, int gu_dtype, long long gu_ld, const float* logits, long long logits_ld, void* y, int y_dtype,
                                          long long y_ld, int tokens, int experts, int top, int ff, float limit, int shared_ff, float shared_limit,
                                          float alpha, float* weights_out, int identity, const float* correction, int group_count, int group_keep, int act,
-                                         float* id_weight, float* shared_weight, cudaStream_t stream)
+                                         float* id_weight, float* shared_weight, cudaStream_t stream, int score, int group_score)
 {
     if (gu == nullptr && weights_out == nullptr) SPY_FAIL("moe_activation: neither activations nor weights are asked for");
-    MoeRouting r = {identity, correction, group_count, group_keep, act, id_weight, shared_weight};
+    MoeRouting r = {identity, correction, group_count, group_keep, act, id_weight, shared_weight, score, group_score};
     return run_moe_activation(gu, gu_dtype, gu_ld, logits, logits_ld, y, y_dtype, y_ld, tokens, experts, top, ff, limit, shared_ff, shared_limit, alpha,
                               weights_out, r, stream);
 }

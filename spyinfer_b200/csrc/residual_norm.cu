@@ -163,3 +163,54 @@ extern "C" int spy_residual_norm(float* h, const void* y, int y_dtype, int split
     SPY_CHECK_LAUNCH("residual_norm");
     return 0;
 }
+
+// out = a_scale * rms_norm(a) * a_weight + b_scale * rms_norm(b) * b_weight, row by row: two sublayer outputs side by side, each normed over
+// the whole row (each possibly a stack of split-K partial sums).  One block a row; both rows stay in shared memory between the passes.
+template <typename TA, typename TB>
+__global__ void normed_sum_kernel(float* __restrict__ out, const TA* __restrict__ a, int a_splits, long long a_stride, const float* __restrict__ a_weight,
+                                  float a_scale, const TB* __restrict__ b, int b_splits, long long b_stride, const float* __restrict__ b_weight, float b_scale,
+                                  int len, float eps)
+{
+    extern __shared__ float rows_s[];
+    __shared__ float scratch[33];
+    pdl_enter();
+    const long long at = (long long)blockIdx.x * len;
+    float *ra = rows_s, *rb = rows_s + len;
+    float sa = 0.f, sb = 0.f;
+    for (int i = threadIdx.x; i < len; i += blockDim.x) {
+        float va = to_f32(a[at + i]), vb = to_f32(b[at + i]);
+#pragma unroll 4
+        for (int s = 1; s < a_splits; ++s) va += to_f32(a[s * a_stride + at + i]);
+#pragma unroll 4
+        for (int s = 1; s < b_splits; ++s) vb += to_f32(b[s * b_stride + at + i]);
+        ra[i] = va;
+        rb[i] = vb;
+        sa = fmaf(va, va, sa);
+        sb = fmaf(vb, vb, sb);
+    }
+    sa = block_sum(sa, scratch);
+    sb = block_sum(sb, scratch);
+    const float ia = a_scale / sqrtf(sa / (float)len + eps), ib = b_scale / sqrtf(sb / (float)len + eps);
+    for (int i = threadIdx.x; i < len; i += blockDim.x) out[at + i] = ra[i] * ia * a_weight[i] + rb[i] * ib * b_weight[i];
+}
+
+extern "C" int spy_normed_sum(float* out, const void* a, int a_dtype, int a_splits, long long a_stride, const float* a_weight, float a_scale, const void* b,
+                              int b_dtype, int b_splits, long long b_stride, const float* b_weight, float b_scale, int rows, int len, float eps,
+                              cudaStream_t stream)
+{
+    if (rows <= 0) return 0;
+    if (len <= 0 || a_splits < 1 || b_splits < 1) SPY_FAIL("normed_sum: rows of %d elements, %d and %d parts", len, a_splits, b_splits);
+    const size_t smem = 2 * (size_t)len * sizeof(float);
+    if (smem > 220 * 1024) SPY_FAIL("normed_sum: two rows of %d elements do not fit a block's shared memory", len);
+    const int threads = len >= 2048 ? 512 : len >= 512 ? 256 : 128;
+    SPY_DISPATCH_DTYPE(a_dtype, TA, {
+        SPY_DISPATCH_DTYPE(b_dtype, TB, {
+            auto kernel = normed_sum_kernel<TA, TB>;
+            if (smem > 48 * 1024) SPY_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            spy_launch(kernel, dim3(rows), dim3(threads), smem, stream, out, (const TA*)a, a_splits, a_stride, a_weight, a_scale, (const TB*)b, b_splits,
+                       b_stride, b_weight, b_scale, len, eps);
+        })
+    })
+    SPY_CHECK_LAUNCH("normed_sum");
+    return 0;
+}

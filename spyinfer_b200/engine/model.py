@@ -13,9 +13,9 @@ from typing import Dict, List, Optional
 import torch
 
 from .. import kernels
-from ..config.spec import ModelSpec
+from ..config.spec import ModelSpec, StreamAdd, StreamProject
 from ..csrc import build
-from ..parts import BuildContext, build_block, build_part
+from ..parts import BuildContext, Linear, build_block, build_part
 from ..weights.loader import LazyTensors, WeightDecl, open_checkpoint
 from ..weights.random_init import random_tensor
 
@@ -51,10 +51,14 @@ class Model:
         # tensors that the run order adds to the stream between layers (name -> rows), and the bound tensors
         self.stream_rows: Dict[str, int] = {}
         for e in spec.run_order:
-            if e.before is not None and e.before.tensor is not None:
+            if isinstance(e.before, StreamAdd) and e.before.tensor is not None:
                 if self.stream_rows.setdefault(e.before.tensor, e.before.rows) != e.before.rows or not 0 <= e.before.row < e.before.rows:
                     raise ValueError(f"run order: the rows of the stream offset {e.before.tensor!r} do not agree")
         self.stream_tensors: Dict[str, torch.Tensor] = {}
+        # projections of [stream; embedding output] that take the stream's place between layers
+        self.stream_products: Dict[str, Optional[Linear]] = {e.before.tensor: None for e in spec.run_order if isinstance(e.before, StreamProject)}
+        if self.stream_products and getattr(self.embedding, "pairs", None) is not None:
+            raise ValueError("run order: a projection of the stream and the embedding output needs an embedding that is a table's row")
 
     # ---- weights ---------------------------------------------------------------------------
     def weight_decls(self) -> List[WeightDecl]:
@@ -63,6 +67,7 @@ class Model:
             for part in layer.parts():
                 decls += _prefixed(part, layer.prefix)
         decls += [WeightDecl(name, (rows, self.spec.hidden_size)) for name, rows in self.stream_rows.items()]
+        decls += [WeightDecl(name, (self.spec.hidden_size, 2 * self.spec.hidden_size)) for name in self.stream_products]
         decls += _prefixed(self.final_norm, "") + _prefixed(self.head, "")
         return decls
 
@@ -83,11 +88,17 @@ class Model:
             for part in layer.parts():
                 part.bind(sub(part, layer.prefix))
         self.stream_tensors = {name: tensors[name] for name in self.stream_rows}
+        for name in self.stream_products:
+            self.stream_products[name] = Linear(tensors[name], self.ctx.dtype)
         self.final_norm.bind(sub(self.final_norm, ""))
         head_names = {d.name for d in self.head.weight_decls()} | {getattr(self.head, "weight_name", None)} - {None}
         self.head.bind({n: tensors[n] for n in head_names if n in tensors})
         # every product learns which weight the step reads after its own (the hint is a weight's address, nothing else)
-        chain = [lin for e in self.spec.run_order for part in self.layers[e.layer].parts() for lin in part.linears()] + self.head.linears()
+        chain = []
+        for e in self.spec.run_order:
+            chain += [self.stream_products[e.before.tensor]] if isinstance(e.before, StreamProject) else []
+            chain += [lin for part in self.layers[e.layer].parts() for lin in part.linears()]
+        chain += self.head.linears()
         for lin, following in zip(chain, chain[1:]):
             lin.next_weight = following.weight
         build.ensure_built(self.kernel_modules())
@@ -120,6 +131,8 @@ class Model:
             mods += list(getattr(layer.block, "kernel_modules", ()))
         if any(e.before is not None for e in self.spec.run_order):
             mods.append("embedding")
+        for lin in self.stream_products.values():
+            mods += lin.modules()
         return list(dict.fromkeys(mods))
 
     def graph_safe(self) -> bool:
@@ -152,6 +165,9 @@ class Model:
                 # the pending output of the block ahead goes in first: what is added here is added to the finished stream
                 hidden, delta = self.layers[self.spec.run_order[i - 1].layer].block.settle(hidden, delta) if i else hidden, None
                 add = entry.before
+                if isinstance(add, StreamProject):
+                    hidden = self._projected_stream(self.stream_products[add.tensor], hidden, batch)
+            if isinstance(entry.before, StreamAdd):
                 kernels.stream_add(hidden, self.embedding.table if add.embedding else None, batch.token_ids if add.embedding else None,
                                    self.stream_tensors[add.tensor][add.row] if add.tensor is not None else None, batch.status)
             view = cache_manager.view(i)
@@ -166,6 +182,11 @@ class Model:
         else:
             x = self.final_norm.forward_add(hidden, delta, rows=batch.logit_rows)
         return self.head.forward(x)
+
+    def _projected_stream(self, product: Linear, hidden: torch.Tensor, batch) -> torch.Tensor:
+        both = torch.empty((hidden.shape[0], 2 * hidden.shape[1]), dtype=self.ctx.dtype, device=hidden.device)
+        kernels.stream_concat(hidden, self.embedding.table, batch.token_ids, self.embedding.scale, both, batch.status)
+        return product(both, out_dtype=torch.float32)
 
 
 def declared_weights(spec: ModelSpec) -> List[WeightDecl]:

@@ -534,6 +534,67 @@ def gla_scan(proj: torch.Tensor, offsets, decay_pre: torch.Tensor, decay_bias: t
     return out
 
 
+def _head_gate_checks(what, proj, offsets, sizes, gates, cols, per_head, state, heads, dk, dv, share):
+    if share <= 0 or heads % share:
+        raise KernelError(f"{what}: {heads} heads do not share keys by {share}")
+    if state.dim() != 2 or state.shape[1] != heads * dk * dv:
+        raise KernelError(f"{what}: state {tuple(state.shape)} does not fit {heads} heads of {dk} x {dv}")
+    _check(gates, f"{what} gates", torch.float32, 2)
+    for t in per_head:
+        _check(t, f"{what} head parameter", torch.float32, 1)
+    if (any(o + n > proj.shape[1] for o, n in zip(offsets, sizes)) or gates.shape[0] != proj.shape[0] or any(c + heads > gates.shape[1] for c in cols)
+            or any(t.shape[0] != heads for t in per_head)):
+        raise KernelError(f"{what}: the column offsets or the heads' parameters do not fit")
+
+
+def gated_delta_scan(proj: torch.Tensor, offsets, gates: torch.Tensor, rate_col: int, decay_col: int, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                     state: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, num_seqs: int, out: torch.Tensor, heads: int, share: int, dk: int,
+                     dv: int, q_scale: float, status: Optional[torch.Tensor] = None, longest: Optional[int] = None) -> torch.Tensor:
+    """The gated delta rule over every request's tokens of this step, from and into ``state [slots, heads * dk * dv]``: with unit
+    vectors ``q`` (times ``q_scale``) and ``k`` (``x / sqrt(sum x^2 + 1e-6)``, made here), ``g = exp(-exp(a_log) softplus(gates[:, decay_col..] +
+    dt_bias))`` and ``beta = sigmoid(gates[:, rate_col..])``, one of each a head: ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``,
+    ``o = S^T q``.  ``proj [T, ld]`` float32 holds q, k (``heads / share`` heads of dk) and v (``heads`` of dv) at ``offsets``."""
+    _scan_common(proj, state, q_start, state_slot, out, heads, dv)
+    oq, ok, ov = (int(o) for o in offsets)
+    _head_gate_checks("gated delta rule", proj, (oq, ok, ov), (heads // max(share, 1) * dk,) * 2 + (heads * dv,), gates, (rate_col, decay_col), (a_log, dt_bias), state,
+                      heads, dk, dv, share)
+    _call("recurrence", "spy_gated_delta_scan", _ptr(proj), ctypes.c_longlong(proj.shape[1]), oq, ok, ov, _ptr(gates), ctypes.c_longlong(gates.shape[1]),
+          int(rate_col), int(decay_col), _ptr(a_log), _ptr(dt_bias), _ptr(state), state.shape[0], _ptr(q_start), _ptr(state_slot), int(num_seqs),
+          int(longest or proj.shape[0]), _ptr(out), int(heads), int(share), int(dk), int(dv), ctypes.c_float(q_scale), _ptr(status), _stream())
+    return out
+
+
+def ssd_scan(proj: torch.Tensor, offsets, gates: torch.Tensor, dt_col: int, a_log: torch.Tensor, dt_bias: torch.Tensor, d_skip: torch.Tensor,
+             state: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, num_seqs: int, out: torch.Tensor, heads: int, share: int, n: int, dv: int,
+             status: Optional[torch.Tensor] = None, longest: Optional[int] = None) -> torch.Tensor:
+    """The state-space dual scan over every request's tokens of this step, from and into ``state [slots, heads * n * dv]``: with
+    ``dt = softplus(gates[:, dt_col..] + dt_bias)``, one a head: ``S <- exp(-exp(a_log) dt) S + dt B x^T``, ``o = S^T C + d_skip x``.
+    ``proj [T, ld]`` float32 holds x (``heads`` of dv), B and C (``heads / share`` of n) at ``offsets = (x, B, C)``."""
+    _scan_common(proj, state, q_start, state_slot, out, heads, dv)
+    ox, ob, oc = (int(o) for o in offsets)
+    _head_gate_checks("state-space dual scan", proj, (ox, ob, oc), (heads * dv,) + (heads // max(share, 1) * n,) * 2, gates, (dt_col,), (a_log, dt_bias, d_skip), state,
+                      heads, n, dv, share)
+    _call("recurrence", "spy_ssd_scan", _ptr(proj), ctypes.c_longlong(proj.shape[1]), oc, ob, ox, _ptr(gates), ctypes.c_longlong(gates.shape[1]), int(dt_col),
+          _ptr(a_log), _ptr(dt_bias), _ptr(d_skip), _ptr(state), state.shape[0], _ptr(q_start), _ptr(state_slot), int(num_seqs),
+          int(longest or proj.shape[0]), _ptr(out), int(heads), int(share), int(n), int(dv), _ptr(status), _stream())
+    return out
+
+
+def gate_group_norm(o: torch.Tensor, proj: torch.Tensor, gate_offset: int, weight: torch.Tensor, out: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+    """``y = o * silu(proj[:, gate_offset : gate_offset + size])``, each of ``groups`` equal parts of a row divided by its own root mean
+    square, times ``weight``; ``o`` float32 ``[T, size]``."""
+    _check(o, "recurrence output", torch.float32, 2)
+    _check(proj, "fused projection", torch.float32, 2)
+    _check(weight, "group norm weight", torch.float32, 1)
+    _check(out, "gated output", ndim=2)
+    n = o.shape[1]
+    if tuple(out.shape) != tuple(o.shape) or weight.shape[0] != n or gate_offset + n > proj.shape[1] or proj.shape[0] != o.shape[0] or groups <= 0 or n % groups:
+        raise KernelError("gate_group_norm: shapes do not fit")
+    _call("recurrence", "spy_gate_group_norm", _ptr(o), _ptr(proj), ctypes.c_longlong(proj.shape[1]), int(gate_offset), _ptr(weight), _ptr(out),
+          _code(out, "gated output"), o.shape[0], n, int(groups), ctypes.c_float(eps), _stream())
+    return out
+
+
 def gated_head_norm(o: torch.Tensor, proj: torch.Tensor, gate_offset: int, weight: torch.Tensor, out: torch.Tensor, heads: int, dv: int, eps: float,
                     gate: str = "sigmoid") -> torch.Tensor:
     """``out = o / rms(o per head) * weight * gate(proj[:, gate_offset : gate_offset + heads * dv])``; ``o`` float32 ``[T, heads * dv]``;
@@ -1090,6 +1151,141 @@ def group_norm(hidden: torch.Tensor, groups: int, eps: float, y: Optional[torch.
     return out
 
 
+def dynamic_tanh(hidden: torch.Tensor, y: Optional[torch.Tensor] = None, y_norm: Optional[tuple] = None, y_scale: float = 1.0, norm: Optional[tuple] = None,
+                 out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, write_back: bool = True) -> Optional[torch.Tensor]:
+    """``dyt(x) = tanh(alpha x) * weight + bias`` element by element around the 32-bit stream ``hidden [T, len]``; a norm is the triple
+    ``(alpha [1] float32, weight [len], bias [len])``.  With ``y`` (a sublayer's output of hidden's shape, or a stack ``[splits, T, len]`` of
+    partial sums) first ``hidden += y_scale * dyt_y(y)`` (stored unless ``write_back`` is false or ``rows`` is given); with ``norm`` and
+    ``out [n, len]`` then ``out = dyt(hidden)``, of all rows or of the gathered ``rows``."""
+    _check(hidden, "residual stream", torch.float32, 2)
+    T, H = hidden.shape
+    yp, splits, stride = _stack_of(y, hidden, "dynamic_tanh sublayer output")
+    if y is not None and y_norm is None:
+        raise KernelError("dynamic_tanh: a sublayer output needs its norm")
+    w_code = None
+    for given, what in ((y_norm if y is not None else None, "output norm"), (norm, "norm")):
+        if given is None:
+            continue
+        alpha, w, b = given
+        _check(alpha, f"dynamic_tanh {what} alpha", torch.float32)
+        _check(w, f"dynamic_tanh {what} weight", ndim=1)
+        _check(b, f"dynamic_tanh {what} bias", w.dtype, 1)
+        if alpha.numel() != 1 or w.shape[0] != H or b.shape[0] != H:
+            raise KernelError(f"dynamic_tanh {what}: one alpha, and a weight and a bias of {H} elements")
+        if w_code is not None and _code(w, what) != w_code:
+            raise KernelError("dynamic_tanh: the two norms differ in dtype")
+        w_code = _code(w, what)
+    n = T
+    if rows is not None:
+        _check(rows, "dynamic_tanh rows", torch.int32, 1)
+        n = rows.shape[0]
+    if norm is not None:
+        _check(out, "dynamic_tanh output", ndim=2)
+        if tuple(out.shape) != (n, H):
+            raise KernelError(f"dynamic_tanh output: expected {(n, H)}, found {tuple(out.shape)}")
+    elif rows is not None:
+        raise KernelError("dynamic_tanh: gathered rows need a norm to go through")
+    ya, yw, yb = y_norm if y is not None else (None, None, None)
+    xa, xw, xb = norm if norm is not None else (None, None, None)
+    _call("dynamic_tanh", "spy_dynamic_tanh", _ptr(hidden), _ptr(yp), _code(yp, "dynamic_tanh sublayer output") if yp is not None else 0, max(splits, 1),
+          ctypes.c_longlong(stride if splits > 1 else 0), _ptr(ya), _ptr(yw), _ptr(yb), ctypes.c_float(y_scale), _ptr(rows), _ptr(xa), _ptr(xw), _ptr(xb),
+          w_code or 0, _ptr(out if norm is not None else None), _code(out, "dynamic_tanh output") if norm is not None else 0, n, H,
+          int(bool(write_back and rows is None)), _stream())
+    return out
+
+
+def qkv_store(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, bias: Optional[torch.Tensor], rope_table: Optional[torch.Tensor], positions: torch.Tensor,
+              seq_of_token: torch.Tensor, q_out: torch.Tensor, block_table: torch.Tensor, pages: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
+              pairing: str = "interleaved", status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The step ahead of the attention kernel for queries and keys without norms.  ``proj [T, ld]`` (or a stack ``[splits, T, ld]`` of
+    float32 partial products) holds, from the given columns, the queries (``heads`` x ``dim``), the keys (``kv_heads`` x ``dim``) and the
+    values (``kv_heads`` x ``vdim``); ``bias [ld]`` float32 is added; the pairs of every query and key head are rotated by ``rope_table
+    [positions, r, 2]``.  ``q_out [T, heads hd]`` and ``pages [num_pages, 2, kv_heads, page_size, hd]`` get rows of ``hd`` with zeros
+    behind their content."""
+    if pairing not in ("half", "interleaved"):
+        raise KernelError(f"qkv_store: unknown pairing rule {pairing!r}")
+    if proj.dim() == 3:
+        _check(proj, "projection parts", torch.float32, 3)
+        splits, stride = proj.shape[0], proj.shape[1] * proj.shape[2]
+    else:
+        _check(proj, "projection", ndim=2)
+        splits, stride = 1, 0
+    T, ld = proj.shape[-2:]
+    _check(q_out, "queries", ndim=2)
+    _check(pages, "cache pages", q_out.dtype, 5)
+    _check(block_table, "block table", torch.int32, 2)
+    _check(positions, "positions", torch.int32, 1)
+    _check(seq_of_token, "seq_of_token", torch.int32, 1)
+    num_pages, two, nkv, page_size, hd = pages.shape
+    if two != 2 or nkv != kv_heads or tuple(q_out.shape) != (T, heads * hd) or positions.shape[0] != T or seq_of_token.shape[0] != T:
+        raise KernelError(f"qkv_store: pages {tuple(pages.shape)} / queries {tuple(q_out.shape)} do not fit {heads} heads over {kv_heads} of rows {hd}")
+    if max(q_col + heads * dim, k_col + kv_heads * dim, v_col + kv_heads * vdim) > ld:
+        raise KernelError("qkv_store: the columns do not fit the projection")
+    if bias is not None:
+        _check(bias, "projection bias", torch.float32, 1)
+        if bias.shape[0] != ld:
+            raise KernelError("qkv_store: the bias has one entry per column of the projection")
+    rot_half = table_rows = 0
+    if rope_table is not None:
+        _check(rope_table, "rope table", torch.float32, 3)
+        table_rows, rot_half = rope_table.shape[0], rope_table.shape[1]
+    _call("qkv_store", "spy_qkv_store", _ptr(proj), _code(proj, "projection"), ctypes.c_longlong(ld), splits, ctypes.c_longlong(stride), int(q_col), int(k_col),
+          int(v_col), _ptr(bias), _ptr(rope_table), rot_half, table_rows, 1 if pairing == "half" else 0, _ptr(positions), _ptr(seq_of_token), _ptr(q_out),
+          _code(q_out, "queries"), _ptr(block_table), block_table.shape[1], _ptr(pages), page_size, num_pages, T, int(heads), int(kv_heads), int(dim), int(vdim),
+          hd, _ptr(status), _stream())
+    return q_out
+
+
+def gate_heads(attn: torch.Tensor, hd: int, gate: torch.Tensor, gate_col: int, out: torch.Tensor, heads: int, vdim: int) -> torch.Tensor:
+    """``out[t, h vdim + e] = attn[t, h hd + e] * sigmoid(gate[t, gate_col + h vdim + e])``; ``gate [T, ld]`` or a stack ``[splits, T, ld]``
+    of float32 partial products."""
+    _check(attn, "attention result", ndim=2)
+    _check(out, "gated heads", attn.dtype, 2)
+    if gate.dim() == 3:
+        _check(gate, "gate parts", torch.float32, 3)
+        splits, stride = gate.shape[0], gate.shape[1] * gate.shape[2]
+    else:
+        _check(gate, "gate", ndim=2)
+        splits, stride = 1, 0
+    T, ld = gate.shape[-2:]
+    if tuple(attn.shape) != (T, heads * hd) or tuple(out.shape) != (T, heads * vdim) or gate_col < 0 or gate_col + heads * vdim > ld:
+        raise KernelError(f"gate_heads: result {tuple(attn.shape)}, output {tuple(out.shape)} or the gate's columns do not fit {heads} heads of {vdim} in rows of {hd}")
+    _call("qkv_store", "spy_gate_heads", _ptr(attn), _code(attn, "attention result"), int(hd), _ptr(gate), _code(gate, "gate"), ctypes.c_longlong(ld), splits,
+          ctypes.c_longlong(stride), int(gate_col), _ptr(out), T, int(heads), int(vdim), _stream())
+    return out
+
+
+def normed_sum(out: torch.Tensor, a: torch.Tensor, a_weight: torch.Tensor, a_scale: float, b: torch.Tensor, b_weight: torch.Tensor, b_scale: float,
+               eps: float) -> torch.Tensor:
+    """``out = a_scale * rms_norm(a) * a_weight + b_scale * rms_norm(b) * b_weight`` row by row in 32-bit; ``a`` and ``b`` have out's shape
+    or are stacks of partial sums."""
+    _check(out, "normed sum", torch.float32, 2)
+    pa, sa, stride_a = _stack_of(a, out, "first result")
+    pb, sb, stride_b = _stack_of(b, out, "second result")
+    for w, what in ((a_weight, "first norm weight"), (b_weight, "second norm weight")):
+        _check(w, what, torch.float32, 1)
+        if w.shape[0] != out.shape[1]:
+            raise KernelError(f"{what}: {w.shape[0]} elements do not fit rows of {out.shape[1]}")
+    _call("residual_norm", "spy_normed_sum", _ptr(out), _ptr(pa), _code(pa, "first result"), sa, ctypes.c_longlong(stride_a), _ptr(a_weight), ctypes.c_float(a_scale),
+          _ptr(pb), _code(pb, "second result"), sb, ctypes.c_longlong(stride_b), _ptr(b_weight), ctypes.c_float(b_scale), out.shape[0], out.shape[1],
+          ctypes.c_float(eps), _stream())
+    return out
+
+
+def stream_concat(stream: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float, out: torch.Tensor, status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[t] = [stream[t] | table[ids[t]] * scale]``; stream float32 ``[T, H]``, out ``[T, 2 H]``."""
+    _check(stream, "residual stream", torch.float32, 2)
+    _check(table, "embedding table", ndim=2)
+    _check(ids, "token ids", torch.int32, 1)
+    _check(out, "concatenated rows", ndim=2)
+    T, H = stream.shape
+    if table.shape[1] != H or ids.shape[0] != T or tuple(out.shape) != (T, 2 * H):
+        raise KernelError("stream_concat: the table's rows, the token ids and the output must fit the stream")
+    _call("embedding", "spy_stream_concat", _ptr(stream), _ptr(table), _code(table, "embedding table"), _ptr(ids), ctypes.c_float(scale), _ptr(out),
+          _code(out, "concatenated rows"), T, H, table.shape[0], _ptr(status), _stream())
+    return out
+
+
 def time_conv(x: torch.Tensor, channels: int, kernel: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], q_start: torch.Tensor,
               state_slot: torch.Tensor, num_seqs: int, longest: int, out: torch.Tensor, residual: bool = False, activation: Optional[str] = None) -> torch.Tensor:
     """Causal convolution over time on the first ``channels`` columns of ``x [T, ld]``: ``kernel [channels, taps]`` (its last
@@ -1307,10 +1503,16 @@ def selective_scan(x: torch.Tensor, dt_pre: torch.Tensor, dt_bias: torch.Tensor,
     return out
 
 
+def _scoring_codes(scoring: str, group_score: str):
+    if scoring not in ("softmax", "sigmoid") or group_score not in ("best", "best_two"):
+        raise KernelError(f"expert choice: unknown scoring {scoring!r} or group score {group_score!r}")
+    return ("softmax", "sigmoid").index(scoring), ("best", "best_two").index(group_score)
+
+
 def moe_activation(gate_up: torch.Tensor, logits: torch.Tensor, out: torch.Tensor, experts: int, top: int, ff: int, limit: float, shared_ff: int = 0,
                    shared_limit: float = 0.0, alpha: float = 1.702, weights_out: Optional[torch.Tensor] = None, identity: int = 0,
                    correction: Optional[torch.Tensor] = None, groups: Optional[tuple] = None, activation: str = "clamped_swish",
-                   id_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   id_weight: Optional[torch.Tensor] = None, scoring: str = "softmax", group_score: str = "best") -> torch.Tensor:
     """Routing weights and expert activations of a mixture of experts in one pass.  ``logits [T, >= experts + identity (+ 1)]``
     float32: the router's logits and, with a shared expert, its gate's logit behind them.  ``gate_up [T, 2 (experts ff +
     shared_ff)]``: per expert ``[gate | up]``, the shared expert last.  ``out [T, experts ff + shared_ff]`` gets, per expert,
@@ -1321,7 +1523,8 @@ def moe_activation(gate_up: torch.Tensor, logits: torch.Tensor, out: torch.Tenso
     The choice: the softmax runs over ``experts + identity`` router outputs, the last ``identity`` of which are experts that
     return their input (``id_weight [T]`` float32 receives the sum of the chosen ones' weights); ``correction [experts +
     identity]`` float32 is added to the scores for the choice only; ``groups = (count, keep)``: the outputs form ``count`` equal
-    groups of neighbours and only those of the ``keep`` groups with the largest best choice score can be chosen."""
+    groups of neighbours and only those of the ``keep`` groups with the largest best choice score (``group_score="best_two"``: sum
+    of the two largest) can be chosen; ``scoring="sigmoid"``: the scores are the logits' sigmoids."""
     _check(gate_up, "expert gate|up", ndim=2)
     _check(logits, "router logits", torch.float32, 2)
     _check(out, "expert activations", ndim=2)
@@ -1345,7 +1548,8 @@ def moe_activation(gate_up: torch.Tensor, logits: torch.Tensor, out: torch.Tenso
             raise KernelError("moe_activation: one identity weight a token")
     if identity and id_weight is None:
         raise KernelError("moe_activation: identity experts need a place for their weights")
-    plain = not identity and correction is None and not groups and activation == "clamped_swish"
+    codes = _scoring_codes(scoring, group_score)
+    plain = not identity and correction is None and not groups and activation == "clamped_swish" and codes == (0, 0)
     args = (_ptr(gate_up), _code(gate_up, "expert gate|up"), ctypes.c_longlong(gate_up.shape[1]), _ptr(logits),
             ctypes.c_longlong(logits.shape[1]), _ptr(out), _code(out, "expert activations"), ctypes.c_longlong(out.shape[1]), T, int(experts), int(top),
             int(ff), ctypes.c_float(limit), int(shared_ff), ctypes.c_float(shared_limit), ctypes.c_float(alpha), _ptr(weights_out))
@@ -1354,12 +1558,12 @@ def moe_activation(gate_up: torch.Tensor, logits: torch.Tensor, out: torch.Tenso
     else:
         count, keep = (int(groups[0]), int(groups[1])) if groups else (0, 0)
         _call("moe", "spy_moe_activation_routed", *args, int(identity), _ptr(correction), count, keep, 1 if activation == "silu" else 0, _ptr(id_weight),
-              None, _stream())
+              None, _stream(), *codes)
     return out
 
 
 def moe_route_general(logits: torch.Tensor, experts: int, top: int, identity: int = 0, correction: Optional[torch.Tensor] = None,
-                      groups: Optional[tuple] = None, has_shared: bool = False):
+                      groups: Optional[tuple] = None, has_shared: bool = False, scoring: str = "softmax", group_score: str = "best"):
     """As ``moe_route`` for a choice with the options of ``moe_activation`` (identity experts, correction, groups): the (token,
     chosen real expert) pairs of a step sorted by expert.  Returns ``offsets [experts + 1]``, ``slot [T, top]`` (the row of each
     pair, -1 where a token chose fewer real experts than ``top``), ``row_token``, ``row_w`` (``[T top]``, the first ``offsets[-1]``
@@ -1374,7 +1578,8 @@ def moe_route_general(logits: torch.Tensor, experts: int, top: int, identity: in
     count, keep = (int(groups[0]), int(groups[1])) if groups else (0, 0)
     _call("moe", "spy_moe_activation_routed", None, BF16, ctypes.c_longlong(0), _ptr(logits), ctypes.c_longlong(logits.shape[1]), None, BF16,
           ctypes.c_longlong(0), T, int(experts), int(top), 1, ctypes.c_float(0.0), 1 if has_shared else 0, ctypes.c_float(0.0), ctypes.c_float(0.0),
-          _ptr(weights), int(identity), _ptr(correction), count, keep, 1, _ptr(idw if identity else None), _ptr(shared_w if has_shared else None), _stream())
+          _ptr(weights), int(identity), _ptr(correction), count, keep, 1, _ptr(idw if identity else None), _ptr(shared_w if has_shared else None), _stream(),
+          *_scoring_codes(scoring, group_score))
     ints = torch.empty((3 * T * top + 2 * experts + 1,), dtype=torch.int32, device=dev)
     choice, slot, row_token = ints[:T * top], ints[T * top:2 * T * top], ints[2 * T * top:3 * T * top]
     counts, offsets = ints[3 * T * top:3 * T * top + experts], ints[3 * T * top + experts:]

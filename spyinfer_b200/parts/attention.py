@@ -478,8 +478,72 @@ class DifferentialAttention(Attention):
         return self.o(o, defer=self.defer_output, out_dtype=self.output_dtype)
 
 
+class KeptWindowAttention(Attention):
+    """What attention over a sliding window that also keeps a sequence's first tokens in view has in common, whatever its
+    projections do: a query at position ``i`` sees ``j <= i`` with ``i - j < window`` or ``j < keep_first`` (kept keys stay at their
+    true positions; ``window`` None: every earlier key), under a softmax with or without a ``sink`` (one more in its
+    denominator).  The attention kernels see rows of ``max(dim, vdim)`` rounded up to 8 (zeros behind a row's content).  On the
+    bfloat16 path the window's keys run on the tensor-core kernels of ``attention``, which leave each row's logarithm of its sum of
+    exponentials where something is to be merged in, and ``sink_merge`` adds the kept first keys and the sink; the plain kernel
+    does all of it in one pass.
+
+    params: ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale`` (None: ``dim^(-1/2)``), ``window``, ``keep_first`` (default 0), ``sink``,
+    ``position`` and what ``attention`` takes beside them."""
+
+    any_head_dim = True
+
+    def __init__(self, params, ctx):
+        self.heads, self.groups = int(params["heads"]), int(params["kv_heads"])
+        self.d, self.vd = int(params["dim"]), int(params["vdim"])
+        if min(self.heads, self.groups, self.d, self.vd) <= 0:
+            raise ValueError(f"{self.kind}: sizes must be positive")
+        row = (max(self.d, self.vd) + 7) // 8 * 8
+        base = dict(params)
+        base.update(num_heads=self.heads, num_kv_heads=self.groups, head_dim=row, qk_norm_eps=None, chunk=None)
+        if base.get("scale") is None:
+            base["scale"] = 1.0 / math.sqrt(float(self.d))
+        super().__init__(base, ctx)
+        self.mma = False                 # the plain kernel is the one that knows the kept keys and the sink
+        self.keep_first = max(int(params.get("keep_first") or 0), 0) if self.window is not None else 0     # without a window every key is seen anyway
+        self.sink = bool(params.get("sink", False))
+        if self.position is not None and self.position.rotary_dim > self.d:
+            raise ValueError(f"{self.kind}: a rotation of {self.position.rotary_dim} elements exceeds a head of {self.d}")
+        self.n_q, self.n_k, self.n_v = self.heads * self.d, self.groups * self.d, self.groups * self.vd
+
+    def padded_output_weight(self, o):
+        """The output projection over the attention's rows: where they are wider than a value, the matching columns are zero."""
+        if self.hd == self.vd:
+            return o
+        return torch.nn.functional.pad(o.reshape(self.hidden, self.heads, self.vd), (0, self.hd - self.vd)).reshape(self.hidden, self.heads * self.hd).contiguous()
+
+    def attention_modules(self):
+        return ["attention_generic"] + (["attention_tc", "attention_decode"] if self.tc else []) + (["sink_attention"] if self.sink or self.keep_first else [])
+
+    def attend(self, q, out, batch, cache):
+        if not (self.tc and cache.page_size in kernels.ATTENTION_TMA_PAGE_SIZES):
+            # the float32 path, and sizes or pages that the tensor-core kernels do not take: everything in one plain kernel
+            return kernels.attention_generic(q, self.nh, self.hd, out, cache.pages, cache.block_table, batch.positions, batch.seq_of_token, self.scale,
+                                             window=self.window, status=batch.status, keep_first=self.keep_first, sink=self.sink)
+        head = batch.num_seqs if batch.one_token_each else batch.one_token_head
+        if not (0 < head <= kernels.ATTENTION_DECODE_MAX_SEQS and head * self.nkv <= kernels.ATTENTION_DECODE_MAX_PAIRS
+                and kernels.attention_decode_takes(self.nh, self.nkv, self.hd, cache.page_size, q.dtype)):
+            head = 0
+        merges = self.sink or self.keep_first > 0
+        lse = torch.empty((q.shape[0], self.nh), dtype=torch.float32, device=q.device) if merges else None
+        if head:
+            kernels.attention_decode(q, self.nh, self.hd, out, cache.pages, cache.block_table[:head], batch.positions, batch.q_start[:head + 1], head,
+                                     self.scale, window=self.window, status=batch.status, lse=lse)
+        if head < batch.num_seqs:
+            kernels.attention_tc(q, self.nh, self.hd, out, cache.pages, cache.block_table[head:], batch.positions, batch.q_start[head:],
+                                 batch.num_seqs - head, self.scale, window=self.window, status=batch.status, lse=lse)
+        if merges:
+            kernels.sink_merge(q, self.nh, self.hd, out, lse, cache.pages, cache.block_table, batch.positions, batch.seq_of_token, self.scale,
+                               self.window, self.keep_first, self.sink, status=batch.status)
+        return out
+
+
 @register_part("sink_window_attention")
-class SinkWindowAttention(Attention):
+class SinkWindowAttention(KeptWindowAttention):
     """Grouped-query attention over a sliding window that also keeps a sequence's first tokens in view, under a softmax with
     a sink: a query at position ``i`` sees ``j <= i`` with ``i - j < window`` or ``j < keep_first`` (kept keys stay at their
     true positions), and ``p_j = exp(s_j) / (1 + sum exp(s_j))`` when ``sink`` is set (a key of score 0 that has no value).
@@ -491,10 +555,6 @@ class SinkWindowAttention(Attention):
     reads (``RunEntry.cache_of``), with queries, mask, temperatures and output projection of its own; ``cache_window`` /
     ``cache_keep_first`` then tell the owning layer what its readers need kept (the widest window, the most kept tokens).
 
-    The attention kernels see rows of ``max(dim, vdim)`` rounded up to 8 (zeros behind a row's content).  On the bfloat16
-    path the window's keys run on the tensor-core kernels of ``attention``, which leave each row's logarithm of its sum of
-    exponentials, and ``sink_merge`` adds the kept first keys and the sink; the plain kernel does all of it in one pass.
-
     params: ``hidden_size``, ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``eps``, ``scale`` (None: ``dim^(-1/2)``), ``window``
     (None: every earlier key), ``keep_first`` (default 0), ``sink`` (default true), ``temperature`` (default true),
     ``shares_cache``, ``cache_window``, ``cache_keep_first``, ``position`` (a rotary part with the interleaved pairing, or None),
@@ -502,30 +562,15 @@ class SinkWindowAttention(Attention):
     dim]``, ``k.norm [kv_heads dim]``, ``temp [heads]``, ``o [hidden, heads vdim]``."""
 
     graph_safe = True
-    any_head_dim = True
 
     def __init__(self, params, ctx):
-        self.heads, self.groups = int(params["heads"]), int(params["kv_heads"])
-        self.d, self.vd, self.eps = int(params["dim"]), int(params["vdim"]), float(params["eps"])
-        if min(self.heads, self.groups, self.d, self.vd) <= 0:
-            raise ValueError("sink_window_attention: sizes must be positive")
-        row = (max(self.d, self.vd) + 7) // 8 * 8
-        base = dict(params)
-        base.update(num_heads=self.heads, num_kv_heads=self.groups, head_dim=row, qk_norm_eps=None, chunk=None)
-        if base.get("scale") is None:
-            base["scale"] = 1.0 / math.sqrt(float(self.d))
-        super().__init__(base, ctx)
-        self.mma = False                 # the plain kernel is the one that knows the kept keys and the sink
-        self.keep_first = int(params.get("keep_first") or 0)
-        if self.keep_first < 0 or (self.keep_first and self.window is None):
-            self.keep_first = max(self.keep_first, 0) if self.window is not None else 0     # without a window every key is seen anyway
-        self.sink, self.temperature = bool(params.get("sink", True)), bool(params.get("temperature", True))
+        super().__init__(dict(params, sink=params.get("sink", True)), ctx)
+        self.eps, self.temperature = float(params["eps"]), bool(params.get("temperature", True))
         self.shares_cache = bool(params.get("shares_cache", False))
         self.cache_window = params.get("cache_window", self.window)
         self.cache_keep_first = int(params.get("cache_keep_first", self.keep_first) or 0)
-        if self.position is not None and (self.position.pairing != "interleaved" or self.position.rotary_dim > self.d):
-            raise ValueError("sink_window_attention: the rotation pairs neighbouring elements and fits within a head")
-        self.n_q, self.n_k, self.n_v = self.heads * self.d, self.groups * self.d, self.groups * self.vd
+        if self.position is not None and self.position.pairing != "interleaved":
+            raise ValueError("sink_window_attention: the rotation pairs neighbouring elements")
         self.q_norm_w = self.k_norm_w = self.temp = None
 
     def weight_decls(self):
@@ -543,10 +588,7 @@ class SinkWindowAttention(Attention):
         if len({t.dtype for t in rows}) > 1:
             rows = [t.float() for t in rows]
         self.qkv = Linear(torch.cat(rows, dim=0).contiguous() if len(rows) > 1 else rows[0], self.ctx.dtype)
-        o = tensors[p + "o"]
-        if self.hd != self.vd:           # the attention's rows are wider than a value: the matching columns of the output projection are zero
-            o = torch.nn.functional.pad(o.reshape(self.hidden, self.heads, self.vd), (0, self.hd - self.vd)).reshape(self.hidden, self.heads * self.hd).contiguous()
-        self.o = Linear(o, self.ctx.dtype)
+        self.o = Linear(self.padded_output_weight(tensors[p + "o"]), self.ctx.dtype)
         names = ["q.norm"] + ([] if self.shares_cache else ["k.norm"]) + (["temp"] if self.temperature else [])
         small = {n: tensors[p + n] for n in names}
         if len({t.dtype for t in small.values()}) > 1:
@@ -554,7 +596,7 @@ class SinkWindowAttention(Attention):
         self.q_norm_w, self.k_norm_w, self.temp = small["q.norm"].contiguous(), small.get("k.norm"), small.get("temp")
 
     def modules(self):
-        mods = ["sink_attention", "attention_generic"] + (["attention_tc", "attention_decode"] if self.tc else []) + self.qkv.modules() + self.o.modules()
+        mods = ["sink_attention"] + self.attention_modules() + self.qkv.modules() + self.o.modules()
         if self.position is not None:
             mods += self.position.modules()
         return mods
@@ -583,24 +625,72 @@ class SinkWindowAttention(Attention):
         self.attend(q, out, batch, cache)
         return self.o(out, defer=self.defer_output, out_dtype=self.output_dtype)
 
-    def attend(self, q, out, batch, cache):
-        if not (self.tc and cache.page_size in kernels.ATTENTION_TMA_PAGE_SIZES):
-            # the float32 path, and sizes or pages that the tensor-core kernels do not take: everything in one plain kernel
-            return kernels.attention_generic(q, self.nh, self.hd, out, cache.pages, cache.block_table, batch.positions, batch.seq_of_token, self.scale,
-                                             window=self.window, status=batch.status, keep_first=self.keep_first, sink=self.sink)
-        head = batch.num_seqs if batch.one_token_each else batch.one_token_head
-        if not (0 < head <= kernels.ATTENTION_DECODE_MAX_SEQS and head * self.nkv <= kernels.ATTENTION_DECODE_MAX_PAIRS
-                and kernels.attention_decode_takes(self.nh, self.nkv, self.hd, cache.page_size, q.dtype)):
-            head = 0
-        merges = self.sink or self.keep_first > 0
-        lse = torch.empty((q.shape[0], self.nh), dtype=torch.float32, device=q.device) if merges else None
-        if head:
-            kernels.attention_decode(q, self.nh, self.hd, out, cache.pages, cache.block_table[:head], batch.positions, batch.q_start[:head + 1], head,
-                                     self.scale, window=self.window, status=batch.status, lse=lse)
-        if head < batch.num_seqs:
-            kernels.attention_tc(q, self.nh, self.hd, out, cache.pages, cache.block_table[head:], batch.positions, batch.q_start[head:],
-                                 batch.num_seqs - head, self.scale, window=self.window, status=batch.status, lse=lse)
-        if merges:
-            kernels.sink_merge(q, self.nh, self.hd, out, lse, cache.pages, cache.block_table, batch.positions, batch.seq_of_token, self.scale,
-                               self.window, self.keep_first, self.sink, status=batch.status)
-        return out
+
+@register_part("gated_window_attention")
+class GatedWindowAttention(KeptWindowAttention):
+    """Grouped-query attention with query/key and value sizes of their own, over every earlier key or over a window that keeps a
+    sequence's first tokens in view, without norms on queries and keys: optional biases on q, k and v, optional rotation, an
+    ordinary softmax (or one with a sink), and an optional gate that multiplies the concatenated heads by ``sigmoid(W_g h)`` ahead
+    of the output projection.  All projections of the input are one product; what makes queries and cache rows of it
+    (``qkv_store``) also sums its split-K parts and adds the biases.
+
+    params: ``hidden_size``, ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale`` (None: ``dim^(-1/2)``), ``window`` (None: every earlier
+    key), ``keep_first`` (default 0), ``sink`` (default false), ``position`` (a rotary part or None), ``bias`` (default false), ``gate``
+    (default false), ``prefix``.  Tensors: ``q [heads dim, hidden]``, ``k [kv_heads dim, hidden]``, ``v [kv_heads vdim, hidden]`` (with
+    ``bias``: ``q.b``, ``k.b``, ``v.b``), with ``gate`` ``g [heads vdim, hidden]``, ``o [hidden, heads vdim]``."""
+
+    graph_safe = True
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        self.has_bias, self.gated = bool(params.get("bias", False)), bool(params.get("gate", False))
+        self.cols = (0, self.n_q, self.n_q + self.n_k, self.n_q + self.n_k + self.n_v)       # q, k, v, gate in the fused projection
+        self.bias = None
+
+    def weight_decls(self):
+        p, W = self.prefix, self.hidden
+        decls = []
+        for name, rows in (("q", self.n_q), ("k", self.n_k), ("v", self.n_v)):
+            decls += [WeightDecl(p + name, (rows, W))] + ([WeightDecl(p + name + ".b", (rows,))] if self.has_bias else [])
+        if self.gated:
+            decls.append(WeightDecl(p + "g", (self.heads * self.vd, W)))
+        return decls + [WeightDecl(p + "o", (W, self.heads * self.vd))]
+
+    def bind(self, tensors):
+        p = self.prefix
+        rows = [tensors[p + n] for n in ("q", "k", "v") + (("g",) if self.gated else ())]
+        if len({t.dtype for t in rows}) > 1:
+            rows = [t.float() for t in rows]
+        self.qkv = Linear(torch.cat(rows, dim=0).contiguous(), self.ctx.dtype)
+        if self.has_bias:
+            rest = [torch.zeros(self.heads * self.vd, dtype=torch.float32, device=rows[0].device)] if self.gated else []
+            self.bias = torch.cat([tensors[p + n].float() for n in ("q.b", "k.b", "v.b")] + rest).contiguous()
+        # the gate's pass writes rows of vdim; without it the output projection reads the attention's rows
+        self.o = Linear(tensors[p + "o"] if self.gated else self.padded_output_weight(tensors[p + "o"]), self.ctx.dtype)
+
+    def modules(self):
+        mods = ["qkv_store"] + self.attention_modules() + self.qkv.modules() + self.o.modules()
+        return mods + (self.position.modules() if self.position is not None else [])
+
+    def linears(self):
+        return [self.qkv, self.o]
+
+    def cache_need(self):
+        window = int(self.window) if self.window is not None else None
+        return PagedCacheNeed(self.groups, self.hd, window, keep_first=self.keep_first)
+
+    def forward(self, x, batch, cache):
+        if self.rope_table is None and self.position is not None:
+            self.rope_table = self.position.rotation_table()
+        T = x.shape[0]
+        proj = self.qkv(x, defer=True)
+        q = torch.empty((T, self.nh * self.hd), dtype=x.dtype, device=x.device)
+        kernels.qkv_store(proj, self.cols[0], self.cols[1], self.cols[2], self.bias, self.rope_table, batch.positions, batch.seq_of_token, q,
+                          cache.block_table, cache.pages, self.heads, self.groups, self.d, self.vd,
+                          pairing=self.position.pairing if self.position is not None else "interleaved", status=batch.status)
+        out = torch.empty((T, self.nh * self.hd), dtype=x.dtype, device=x.device)
+        self.attend(q, out, batch, cache)
+        if self.gated:
+            rows = out if self.hd == self.vd else torch.empty((T, self.heads * self.vd), dtype=x.dtype, device=x.device)
+            out = kernels.gate_heads(out, self.hd, proj, self.cols[3], rows, self.heads, self.vd)
+        return self.o(out, defer=self.defer_output, out_dtype=self.output_dtype)

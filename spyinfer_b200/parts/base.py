@@ -69,6 +69,16 @@ class NormedDelta:
     scale: float = 1.0
 
 
+@dataclass
+class TanhDelta:
+    """A sublayer output that is still to go through a dynamic tanh and be added: ``residual += scale * (tanh(alpha y) * weight +
+    bias)`` with ``norm = (alpha, weight, bias)``; the next norm of the same kind forms it in its own launch.  ``y`` as above."""
+
+    y: torch.Tensor
+    norm: Tuple[torch.Tensor, torch.Tensor, torch.Tensor]
+    scale: float = 1.0
+
+
 class Part:
     kind: str = ""
     #: kernel modules (``csrc/<name>.cu``) this part launches; built before the first step

@@ -39,7 +39,9 @@ class ExpertMixture(FeedForward):
     (default 0: so many further router outputs, behind the experts', stand for experts without tensors that return their
     input), ``correction`` (default false: a tensor ``correction [experts + identity]`` is added to the scores for the choice
     only), ``groups`` (None or ``(count, keep)``: the router's outputs form ``count`` equal groups of neighbours, a group counts
-    by its best choice score, and only the ``keep`` best groups' outputs can be chosen).  Tensors: ``router [experts +
+    by its best choice score, and only the ``keep`` best groups' outputs can be chosen), ``scoring`` (``softmax`` over all outputs, the
+    default, or ``sigmoid`` of each output's logit) and ``group_score`` (``best``, the default, or ``best_two``: the sum of a group's two
+    largest choice scores).  Tensors: ``router [experts +
     identity, hidden]``, ``e<i>.{gate,up} [ff, hidden]``, ``e<i>.down [hidden, ff]``, and with a shared expert
     ``shared.{gate,up,down}`` and ``shared.sg [1, hidden]``."""
 
@@ -55,6 +57,9 @@ class ExpertMixture(FeedForward):
         self.identity, self.has_correction = int(params.get("identity") or 0), bool(params.get("correction", False))
         self.groups = tuple(int(v) for v in params["groups"]) if params.get("groups") else None
         self.outputs = self.experts + self.identity                 # the router's outputs
+        self.scoring, self.group_score = params.get("scoring", "softmax"), params.get("group_score", "best")
+        if self.scoring not in ("softmax", "sigmoid") or self.group_score not in ("best", "best_two"):
+            raise ValueError(f"expert_mixture: scoring {self.scoring!r} (softmax, sigmoid), group score {self.group_score!r} (best, best_two)")
         if min(self.hidden, self.experts, self.top, self.ff) <= 0 or self.top > self.outputs or self.shared_ff < 0 or self.identity < 0:
             raise ValueError(f"expert_mixture: {self.experts} experts of {self.ff}, top {self.top}, shared {self.shared_ff} are not served")
         if self.activation not in ("clamped_swish", "silu") or (self.activation == "clamped_swish" and not self.limit > 0.0):
@@ -63,7 +68,7 @@ class ExpertMixture(FeedForward):
             count, keep = self.groups
             if count <= 0 or self.outputs % count or not 0 < keep <= count or keep * (self.outputs // count) < self.top:
                 raise ValueError(f"expert_mixture: {count} groups of which {keep} are kept do not fit {self.outputs} router outputs and top {self.top}")
-        self.plain_choice = not self.identity and not self.has_correction and self.groups is None and self.activation == "clamped_swish"
+        self.plain_choice = not self.identity and not self.has_correction and self.groups is None and self.activation == "clamped_swish" and self.scoring == "softmax"
         self.correction = None
         self.prefix = params.get("prefix", "")
         self.cols = self.experts * self.ff + self.shared_ff
@@ -116,7 +121,8 @@ class ExpertMixture(FeedForward):
             return self.down(y, defer=self.defer_output)
         idw = torch.empty((x.shape[0],), dtype=torch.float32, device=x.device) if self.identity else None
         kernels.moe_activation(gu, logits, y, self.experts, self.top, self.ff, self.limit, self.shared_ff, self.shared_limit, self.slope,
-                               identity=self.identity, correction=self.correction, groups=self.groups, activation=self.activation, id_weight=idw)
+                               identity=self.identity, correction=self.correction, groups=self.groups, activation=self.activation, id_weight=idw,
+                               scoring=self.scoring, group_score=self.group_score)
         if not self.identity:
             return self.down(y, defer=self.defer_output)
         # the identity experts' share, weight * input, joins the experts' sum in 32-bit: in the consumer's kernel where it offers that
@@ -133,7 +139,8 @@ class ExpertMixture(FeedForward):
         if self.plain_choice:
             offsets, slot, row_token, row_w, shared_w = kernels.moe_route(logits, E, top, bool(sff))
         else:
-            offsets, slot, row_token, row_w, shared_w, idw = kernels.moe_route_general(logits, E, top, self.identity, self.correction, self.groups, bool(sff))
+            offsets, slot, row_token, row_w, shared_w, idw = kernels.moe_route_general(logits, E, top, self.identity, self.correction, self.groups, bool(sff),
+                                                                                               scoring=self.scoring, group_score=self.group_score)
         starts = offsets.cpu().tolist()                      # the layer's one read-back: the experts' row counts size their products
         R, n = T * top, starts[E]                            # n rows are in use: a token may have chosen fewer real experts than `top`
         results = torch.empty((R, self.hidden), dtype=torch.float32, device=dev)

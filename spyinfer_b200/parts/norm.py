@@ -11,7 +11,7 @@ import torch
 
 from .. import kernels
 from ..weights.loader import WeightDecl
-from .base import ChannelScaled, Norm, NormedDelta, ScaledParts
+from .base import ChannelScaled, Norm, NormedDelta, ScaledParts, TanhDelta
 from .registry import register_part
 
 
@@ -185,3 +185,61 @@ class GroupRMSNorm(Norm):
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.size), dtype=out_dtype or self.ctx.dtype, device=residual.device)
         return kernels.group_norm(residual, self.groups, self.eps, y=y, y_weight=w, y_scale=scale, weight=self.weight, out=out, rows=rows)
+
+
+@register_part("dynamic_tanh")
+class DynamicTanh(Norm):
+    """``tanh(alpha x) * weight + bias`` element by element: a norm without statistics.  params: ``size``, ``weight`` (the tensor's
+    relative name; the bias and the scalar alpha are beside it as ``<weight>.b`` and ``<weight>.alpha``).
+
+    It serves on both sides of a sublayer as ``group_rms_norm`` does: ``forward_add(residual, delta)`` ahead of one, with
+    ``delta`` possibly a ``TanhDelta`` that a norm of this kind left behind a sublayer (``defer``) and that the one kernel
+    adds first; ``add_normed`` adds such a record at once."""
+
+    graph_safe = True
+    kernel_modules = ("dynamic_tanh",)
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        self.size, self.weight_name = int(params["size"]), params.get("weight", "weight")
+        self.norm = None
+
+    def weight_decls(self):
+        n = self.weight_name
+        return [WeightDecl(n, (self.size,), init="one_plus_normal"), WeightDecl(n + ".b", (self.size,)), WeightDecl(n + ".alpha", (), init="one_plus_normal")]
+
+    def bind(self, tensors):
+        n = self.weight_name
+        w, b = tensors[n], tensors[n + ".b"]
+        if w.dtype != torch.bfloat16 or b.dtype != torch.bfloat16:
+            w, b = w.float(), b.float()
+        self.norm = (tensors[n + ".alpha"].float().reshape(1).contiguous(), w.contiguous(), b.contiguous())
+
+    def defer(self, y, scale=1.0):
+        return TanhDelta(y, self.norm, float(scale))
+
+    def _pending(self, delta):
+        if delta is None:
+            return None, None, 1.0
+        if not isinstance(delta, TanhDelta):
+            raise ValueError("dynamic_tanh: what is pending on the stream must be a sublayer output that a norm of this kind deferred")
+        # one storage type for the two norms of a launch
+        norm = delta.norm if self.norm is None or delta.norm[1].dtype == self.norm[1].dtype else tuple(t.to(self.norm[1].dtype) if t.numel() > 1 else t for t in delta.norm)
+        return delta.y, norm, delta.scale
+
+    def add_normed(self, residual, delta):
+        """``residual += scale * dyt(y)`` for a ``TanhDelta`` (32-bit, in place)."""
+        y, norm, scale = self._pending(delta)
+        if y is not None:
+            kernels.dynamic_tanh(residual, y=y, y_norm=norm, y_scale=scale)
+        return residual
+
+    def forward(self, x, out_dtype=None):
+        out = torch.empty(x.shape, dtype=out_dtype or self.ctx.dtype, device=x.device)
+        return kernels.dynamic_tanh(x, norm=self.norm, out=out)
+
+    def forward_add(self, residual, delta, rows=None, out_dtype=None):
+        y, norm, scale = self._pending(delta)
+        n = residual.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, self.size), dtype=out_dtype or self.ctx.dtype, device=residual.device)
+        return kernels.dynamic_tanh(residual, y=y, y_norm=norm, y_scale=scale, norm=self.norm, out=out, rows=rows)
