@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--shape 8b|14b|32b] [--batch B] [--context C] [--impl ours|reference]
     python bench.py --workload mixed [--shape 14b] [--requests 64] [--budget 2048]     (a continuous batch through LLMEngine; its own line)
-    python bench.py --workload nezolorn | daronex | naforax | dogilorn [--layers 6] [--prefill-tokens 2048]   (another design beside Qwen3 at equal layer sizes; its own line)
+    python bench.py --workload nezolorn | daronex | naforax | dogilorn | zonevik [--layers 6] [--prefill-tokens 2048]   (another design beside Qwen3 at equal layer sizes; its own line)
 
 The model has the layer sizes of Qwen3-8B (36 layers, hidden 4096, 32 query heads, 8 key/value
 heads, head size 128, intermediate 12288, vocabulary 151936, untied head) with seeded random
@@ -784,6 +784,123 @@ def dogilorn_workload(args) -> int:
     return 0
 
 
+def zonevik_workload(args) -> int:
+    """``--workload zonevik``: prefill and decode throughput of the Zonevik design (gated attention over every key with YaRN rotation; a
+    parallel layer of window attention that keeps the first tokens beside the state-space dual scan; the gated delta rule; an expert
+    mixture with sigmoid scores and grouped choice in every layer; dynamic tanh norms; a looped stretch behind a projection of the
+    stream and the embedding output) at two layer sizes that resemble real models, beside the engine's Qwen3 model with the same width,
+    heads, head size, vocabulary and number of layers and a feed-forward of the chosen experts' size, and beside its Nezolorn model
+    (window attention beside a matrix memory, and a delta rule), whose scans are the like kernels of this design's, all with seeded
+    random weights in bfloat16.  Measured as ``--workload nezolorn`` is: one prompt of ``--prefill-tokens`` tokens, decoding at batch 8
+    and 64 from ``--context`` tokens through the decode graphs, and each kernel's time inside one prompt step and one decode step of
+    batch 64."""
+    from spyinfer_b200 import kernels
+
+    hbm_gbs, bf16_tflops, _, peak_src = peaks()
+    layers, vocab, page = args.layers or 6, 32000, 16
+    T, ctx = args.prefill_tokens, min(args.context, 4096)
+    window, keep = 1024, 4
+    sizes = {"width2048": dict(width=2048, heads=16, kv=4, hd=128, experts=8, top=2, groups=(4, 2), expert_ff=2048, ssd_heads=64, ssd_vdim=64, ssd_state=128,
+                               ssd_groups=4, delta_heads=16, delta_kv=8, delta_dim=128, delta_vdim=128),
+             "width4096": dict(width=4096, heads=32, kv=8, hd=128, experts=8, top=2, groups=(4, 2), expert_ff=3072, ssd_heads=128, ssd_vdim=64, ssd_state=128,
+                               ssd_groups=8, delta_heads=32, delta_kv=16, delta_dim=128, delta_vdim=128)}
+
+    def configs(z):
+        attn = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["hd"], "vdim": z["hd"], "scale": z["hd"] ** -0.5}
+        rot = {"base": 1000000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}
+        moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": z["groups"][0], "keep": z["groups"][1]}},
+               "expert": {"ff": z["expert_ff"]}}
+        kinds = [{"type": "attention", "mixer": dict(attn, rot=rot), "mlp": moe},
+                 {"type": "parallel", "mlp": moe, "mixer": {
+                     "left": dict(attn, mask={"size": window, "keep_first": keep}),
+                     "right": {"heads": z["ssd_heads"], "vdim": z["ssd_vdim"], "state": z["ssd_state"], "groups": z["ssd_groups"], "conv": 4,
+                               "norm_groups": z["ssd_groups"]}}},
+                 {"type": "delta", "mlp": moe, "mixer": {"heads": z["delta_heads"], "kv_heads": z["delta_kv"], "dim": z["delta_dim"], "vdim": z["delta_vdim"],
+                                                         "conv": 4}}]
+        zn = {"architecture": "Zonevik", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 4.0},
+              "layers": [kinds[i % 3] for i in range(layers)], "loop": {"start": 0, "stop": layers, "times": 1}}
+        qw = dict(QWEN3_8B)
+        qw.update({"num_hidden_layers": layers, "hidden_size": z["width"], "num_attention_heads": z["heads"], "num_key_value_heads": z["kv"],
+                   "head_dim": z["hd"], "intermediate_size": z["top"] * z["expert_ff"], "vocab_size": vocab})
+        par = {"type": "parallel", "mlp": {"kind": "dense", "ff": z["top"] * z["expert_ff"]},
+               "mixer": {"left": dict(attn, mask={"size": window, "pool": 64}), "left_scale": 1.0, "right_scale": 1.0,
+                         "right": {"heads": z["kv"], "dim": z["hd"], "vdim": 2 * z["hd"], "gate_cap": 15.0}}}
+        delta = {"type": "general_delta", "mlp": {"kind": "dense", "ff": z["top"] * z["expert_ff"]},
+                 "mixer": {"heads": z["delta_heads"], "dim": z["delta_dim"], "decay_rank": 64}}
+        nz = {"architecture": "Nezolorn", "vocab": vocab, "width": z["width"], "residual_mult": 0.5, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+              "layers": [par if i % 3 != 2 else delta for i in range(layers)]}
+        return {"zonevik": zn, "qwen3": qw, "nezolorn": nz}
+
+    def measure(cfg_json, z, name):
+        def annotate(res, rate):
+            W, H, kv, hd = z["width"], z["heads"], z["kv"], z["hd"]
+            per_kind = [sum(1 for i in range(layers) if i % 3 == k) for k in range(3)]
+            full, windowed = T * (T + 1) / 2, sum(min(p + 1, window) for p in range(T))
+            attn = lambda n, keys: 4.0 * n * keys * H * hd
+            cache = lambda n, keys: 64.0 * n * kv * keys * hd * 2 * 2
+            if name == "zonevik":
+                n_att, n_par, n_delta = per_kind
+                rate("kernels_prefill", "attention_tc.spy_attention_tc", flops=attn(n_att, full))
+                rate("kernels_prefill", "attention_tc.spy_attention_tc_lse", flops=attn(n_par, windowed))
+                rate("kernels_decode_b64", "attention_decode.spy_attention_decode", nbytes=cache(n_att, ctx + 1))
+                rate("kernels_decode_b64", "attention_decode.spy_attention_decode_lse", nbytes=cache(n_par, min(ctx + 1, window)))
+                inner, group = z["ssd_heads"] * z["ssd_vdim"], z["ssd_groups"] * z["ssd_state"]
+                d_k, d_v = z["delta_kv"] * z["delta_dim"], z["delta_heads"] * z["delta_vdim"]
+                # a state is read and written once a step and request; a prompt's scan reads its inputs and writes its outputs, and works
+                # 6 operations an element of the state and token (decay, update, read-out; the delta rule 8: it also reads what it removes)
+                rate("kernels_decode_b64", "recurrence.spy_ssd_scan", nbytes=64.0 * n_par * 2 * inner * z["ssd_state"] * 4)
+                rate("kernels_decode_b64", "recurrence.spy_gated_delta_scan", nbytes=64.0 * n_delta * 2 * d_v * z["delta_dim"] * 4)
+                rate("kernels_prefill", "recurrence.spy_ssd_scan", nbytes=float(n_par) * T * (2 * inner + 2 * group) * 4)
+                rate("kernels_prefill", "recurrence.spy_gated_delta_scan", nbytes=float(n_delta) * T * (2 * d_v + 2 * d_k) * 4)
+                for block, rows in (("kernels_prefill", T), ("kernels_decode_b64", 64)):
+                    # reads the sublayer's output (16-bit behind a mixture of few tokens, else 32-bit) and the stream, writes the stream and the row
+                    rate(block, "dynamic_tanh.spy_dynamic_tanh", nbytes=float(2 * layers) * rows * W * (4 + 4 + 4 + 2))
+                    rate(block, "time_conv.spy_time_conv", nbytes=float(rows) * 8 * (n_par * (inner + 2 * group) + n_delta * (d_v + 2 * d_k)))
+                    rate(block, "qkv_store.spy_qkv_store", nbytes=float(rows) * (n_att + n_par) * (H + 2 * kv) * hd * 4)
+                    rate(block, "qkv_store.spy_gate_heads", nbytes=float(rows) * n_att * H * hd * 6)
+                    rate(block, "sink_attention.spy_sink_merge", nbytes=float(rows) * n_par * H * hd * 6)
+                    rate(block, "residual_norm.spy_normed_sum", nbytes=float(rows) * n_par * W * 12)
+                    rate(block, "recurrence.spy_gate_group_norm", nbytes=float(rows) * n_par * inner * (4 + 4 + 2))
+                    rate(block, "recurrence.spy_gated_head_norm", nbytes=float(rows) * n_delta * d_v * (4 + 4 + 2))
+                    cols = z["experts"] * z["expert_ff"]
+                    rate(block, "moe.spy_moe_activation_routed", nbytes=float(layers) * rows * (z["top"] * z["expert_ff"] * 4 + cols * 2))
+            elif name == "qwen3":
+                rate("kernels_prefill", "attention_tc.spy_attention_tc", flops=attn(layers, full))
+                rate("kernels_decode_b64", "attention_decode.spy_attention_decode", nbytes=cache(layers, ctx + 1))
+                for block, rows in (("kernels_prefill", T), ("kernels_decode_b64", 64)):
+                    rate(block, "rmsnorm.spy_rmsnorm", nbytes=float(2 * layers) * rows * W * (4 + 4 + 4 + 2))
+                    rate(block, "qk_rope_store.spy_qk_rope_store", nbytes=float(layers) * rows * (H + 2 * kv) * hd * 4)
+            else:
+                n_par, n_delta = per_kind[0] + per_kind[1], per_kind[2]
+                d_n = z["delta_heads"] * z["delta_dim"]
+                rate("kernels_prefill", "attention_tc.spy_attention_tc_lse", flops=attn(n_par, windowed))
+                rate("kernels_decode_b64", "attention_decode.spy_attention_decode_lse", nbytes=cache(n_par, min(ctx + 1, window)))
+                rate("kernels_decode_b64", "recurrence.spy_mlstm_scan", nbytes=64.0 * n_par * 2 * kv * kernels.mlstm_record(hd, 2 * hd) * 4)
+                rate("kernels_decode_b64", "recurrence.spy_delta_scan", nbytes=64.0 * n_delta * 2 * d_n * z["delta_dim"] * 4)
+                rate("kernels_prefill", "recurrence.spy_mlstm_scan", nbytes=float(n_par) * T * kv * hd * 6 * 4)
+                rate("kernels_prefill", "recurrence.spy_delta_scan", nbytes=float(n_delta) * T * d_n * 6 * 4)
+                for block, rows in (("kernels_prefill", T), ("kernels_decode_b64", 64)):
+                    rate(block, "layernorm.spy_layernorm", nbytes=float(2 * layers) * rows * W * (4 + 4 + 4 + 2))
+                    rate(block, "recurrence.spy_gated_head_norm", nbytes=float(rows) * (n_par * kv * 2 * hd + n_delta * d_n) * (4 + 4 + 2))
+
+        return _measure_design(args, cfg_json, vocab, page, T, ctx, annotate)
+
+    out_sizes = {}
+    with ClockSampler() as clocks:
+        for tag, z in sizes.items():
+            out_sizes[tag] = {"layer_sizes": z, "layers": layers}
+            for name, cfg_json in configs(z).items():
+                out_sizes[tag][name] = measure(cfg_json, z, name)
+    print(json.dumps({"metric": "prefill and decode tokens/s of the Zonevik design beside Qwen3 and Nezolorn at equal layer sizes (bf16, random weights)",
+                      "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": 3, "dtype": "bf16",
+                      "data": "synthetic: seeded random weights and random token ids",
+                      "config": {"layers": layers, "vocab": vocab, "prefill_tokens": T, "decode_context": ctx, "window": window, "keep_first": keep, "page_size": page,
+                                 "pattern": "gated attention, window attention beside the state-space dual scan, the gated delta rule; repeated, an expert mixture in each",
+                                 "timing": "CUDA events; inputs (weights, caches and states of 64 requests) exceed L2"},
+                      "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": bf16_tflops, "source": peak_src}, "sizes": out_sizes, "clocks": clocks.summary()}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -798,9 +915,9 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1/64 and short-context points")
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-kernels", action="store_true", help="skip the per-kernel rooflines")
-    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "nezolorn", "daronex", "naforax", "dogilorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "nezolorn", "daronex", "naforax", "dogilorn", "zonevik"],
                     help="decode: the contract's line (default); mixed: a continuous batch of --requests requests with prompts of 64 to 2,048 "
-                         "tokens and 128 generated tokens each through LLMEngine, its own line; nezolorn, daronex, naforax, dogilorn: prefill and decode of that design "
+                         "tokens and 128 generated tokens each through LLMEngine, its own line; nezolorn, daronex, naforax, dogilorn, zonevik: prefill and decode of that design "
                          "beside Qwen3 at equal layer sizes, its own line")
     ap.add_argument("--requests", type=int, default=64, help="mixed workload: number of requests")
     ap.add_argument("--budget", type=int, default=2048, help="mixed workload: max_num_batched_tokens")
@@ -825,6 +942,8 @@ def main() -> int:
         return naforax_workload(args)
     if args.workload == "dogilorn":
         return dogilorn_workload(args)
+    if args.workload == "zonevik":
+        return zonevik_workload(args)
     hbm_gbs, bf16_tflops, bf16_sustained, peak_src = peaks()
     cfg_json = dict(QWEN3_8B)
     cfg_json.update(SHAPES[args.shape])

@@ -298,7 +298,7 @@ def tensor_shapes(cfg):
 
 def random_weights(cfg, seed, gain=1.0):
     """Seeded weights in bfloat16 (as a checkpoint stores them): matrices of a size that keeps activations of order one, norm
-    weights around one, decays that forget over a few to a few dozen tokens."""
+    weights around one, decays that forget over a few to a few hundred tokens."""
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, shape in tensor_shapes(cfg).items():
@@ -314,7 +314,7 @@ def random_weights(cfg, seed, gain=1.0):
         elif last == "A_log":
             t = 0.5 * torch.randn(shape, generator=g)
         elif last == "dt_bias":
-            t = -2.0 + torch.randn(shape, generator=g)
+            t = -3.0 + 1.5 * torch.randn(shape, generator=g)
         elif last == "conv":
             t = 0.6 * torch.randn(shape, generator=g)
         elif last == "router":
