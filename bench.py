@@ -848,10 +848,10 @@ def zonevik_workload(args) -> int:
                 d_k, d_v = z["delta_kv"] * z["delta_dim"], z["delta_heads"] * z["delta_vdim"]
                 # a state is read and written once a step and request; a prompt's scan reads its inputs and writes its outputs, and works
                 # 6 operations an element of the state and token (decay, update, read-out; the delta rule 8: it also reads what it removes)
-                rate("kernels_decode_b64", "recurrence.spy_ssd_scan", nbytes=64.0 * n_par * 2 * inner * z["ssd_state"] * 4)
-                rate("kernels_decode_b64", "recurrence.spy_gated_delta_scan", nbytes=64.0 * n_delta * 2 * d_v * z["delta_dim"] * 4)
-                rate("kernels_prefill", "recurrence.spy_ssd_scan", nbytes=float(n_par) * T * (2 * inner + 2 * group) * 4)
-                rate("kernels_prefill", "recurrence.spy_gated_delta_scan", nbytes=float(n_delta) * T * (2 * d_v + 2 * d_k) * 4)
+                rate("kernels_decode_b64", "head_scan.spy_ssd_scan", nbytes=64.0 * n_par * 2 * inner * z["ssd_state"] * 4)
+                rate("kernels_decode_b64", "head_scan.spy_gated_delta_scan", nbytes=64.0 * n_delta * 2 * d_v * z["delta_dim"] * 4)
+                rate("kernels_prefill", "head_scan.spy_ssd_scan", nbytes=float(n_par) * T * (2 * inner + 2 * group) * 4)
+                rate("kernels_prefill", "head_scan.spy_gated_delta_scan", nbytes=float(n_delta) * T * (2 * d_v + 2 * d_k) * 4)
                 for block, rows in (("kernels_prefill", T), ("kernels_decode_b64", 64)):
                     # reads the sublayer's output (16-bit behind a mixture of few tokens, else 32-bit) and the stream, writes the stream and the row
                     rate(block, "dynamic_tanh.spy_dynamic_tanh", nbytes=float(2 * layers) * rows * W * (4 + 4 + 4 + 2))

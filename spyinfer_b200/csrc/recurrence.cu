@@ -6,11 +6,6 @@
 //                                            both terms reading the old S, w a decay and r a removal rate per key channel;
 //   * gated linear attention:                S = diag(a) S + k v^T,  o = S^T q,  a = sigmoid(z)^(1/tau) = exp(logsigmoid(z) / tau)
 //                                            a decay per key channel from the pre-activation z;
-//   * the gated delta rule:                  S = g S,  u = beta (v - S^T k),  S = S + k u^T,  o = S^T q,  one decay and one rate a head
-//                                            (g = exp(-exp(A_log) softplus(za + dt_bias)), beta = sigmoid(zb)), q and k unit vectors
-//                                            made here (x / sqrt(sum x^2 + 1e-6)), shared by groups of heads;
-//   * the state-space dual scan:             S = exp(-exp(A_log) dt) S + dt k v^T,  o = S^T q + D v,  dt = softplus(zd + dt_bias),
-//                                            k and q (its B and C) shared by groups of heads;
 // and what follows them: each head's output divided by its root mean square, times a weight, times a gate (sigmoid or SiLU).
 //
 // A block owns a tile of value columns of one (request, head) (32, 16 or 8 of them: whatever gives the SMs a block each) and
@@ -57,22 +52,7 @@ struct ScanArgs {
     int H, dk, dv;
     float q_scale, cap;     // cap: mLSTM: the gates' cap;   gated linear attention: 1 / tau
     int* status;
-    // the two with one decay a head: q and k of head h are those of head h / share; the gates' pre-activations are columns of
-    // `gates` [T, gates_ld] (x1 the rate's, gated delta rule only; x2 the decay's or step's); a_log, dt_bias, d_skip [H]
-    int share;
-    const float* gates;
-    long long gates_ld;
-    const float *a_log, *dt_bias, *d_skip;
 };
-
-// a head's decay and rate for one token: x1, x2 the gates' pre-activations
-__device__ __forceinline__ float softplusf_(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
-template <int MODE> __device__ __forceinline__ void head_gates(const ScanArgs& A, int h, float x1, float x2, float& keep, float& add)
-{
-    const float dt = softplusf_(x2 + A.dt_bias[h]);
-    keep = expf(-expf(A.a_log[h]) * dt);
-    add = MODE == 3 ? sigmoidf_(x1) : dt;
-}
 
 constexpr int THREADS = 256;      // 8 warps; warp w owns the columns 4w .. 4w + 3 of the tile, lane = 4 * (row group) + (column of the four)
 
@@ -88,7 +68,7 @@ constexpr int THREADS = 256;      // 8 warps; warp w owns the columns 4w .. 4w +
 // token run beside those of the others and beside the next token's rows (nothing in S waits for them).
 // RG row groups share a warp's lanes (8, 16 or 32), so a warp owns 32 / RG columns and a block CTB = 8 * 32 / RG of them:
 // with few requests and heads the tiles are made narrow, so that there are blocks for every SM, and a thread's rows few.
-template <int MODE, int NR, int RG>   // MODE 0: gated matrix memory, 1: delta rule, 2: gated linear attention, 3: gated delta rule, 4: state-space dual scan
+template <int MODE, int NR, int RG>   // MODE 0: gated matrix memory, 1: delta rule, 2: gated linear attention
 __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs A, int TC)
 {
     constexpr int CW = 32 / RG, CTB = 8 * CW, SPB = CTB + 4;   // columns a warp and a block own; floats between the rows of the state tile in shared memory
@@ -105,12 +85,11 @@ __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs
     float* o_s = sm + 2 * stage_floats;            // [TC][CTB]
     float* m_s = o_s + TC * CTB;                   // [TC] memory: the running maximum after each token
     float* nqp = m_s + TC;                         // [TC][8] memory: n . q, one partial sum a warp
-    float* a_s = nqp + TC * 8;                     // [TC] memory: what a token keeps of the state, exp(f + m_before - m_after); one decay a head: the decay
-    float* b_s = a_s + TC;                         // [TC] memory: what it adds, exp(i - m_after); one decay a head: the rate or step
+    float* a_s = nqp + TC * 8;                     // [TC] memory: what a token keeps of the state, exp(f + m_before - m_after)
+    float* b_s = a_s + TC;                         // [TC] memory: what it adds, exp(i - m_after)
     float* tile = sm;                              // [dk][SPB], only before the first and after the last chunk
 
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * CTB;
-    const int hk = MODE >= 3 ? h / A.share : h;        // whose q and k the head uses
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int col = warp * CW + lane % CW, rg = lane / CW, r0 = rg * NR;
     const int t_begin = A.q_start[seq], t_end = A.q_start[seq + 1];
@@ -143,7 +122,7 @@ __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs
 
     // whether a token's vectors start on 16-byte boundaries in the projection (and in the decay's pre-activation)
     const bool aligned = (dk & 3) == 0 && (A.ld & 3) == 0 && ((A.off_k | A.off_q) & 3) == 0 && (reinterpret_cast<uintptr_t>(A.proj) & 15) == 0 &&
-                         (MODE == 0 || MODE >= 3 || (((MODE == 1 ? A.off_x1 : 0) & 3) == 0 && (reinterpret_cast<uintptr_t>(A.extra) & 15) == 0));
+                         (MODE == 0 || (((MODE == 1 ? A.off_x1 : 0) & 3) == 0 && (reinterpret_cast<uintptr_t>(A.extra) & 15) == 0));
     // Requests a chunk's vectors into a stage: 16-byte asynchronous copies where the columns allow it (all under way at once),
     // else plain loads; v and the gates' pre-activations by 4-byte copies.  What is made of them (the scaled q, the sigmoid of
     // the removal rate, the decay, the capped gates) is worked out in place once they have landed.
@@ -153,27 +132,27 @@ __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs
         float* q_s = k_s + (size_t)TC * KS;
         float* x1_s = q_s + (size_t)TC * KS;
         float* x2_s = x1_s + (MODE == 1 ? (size_t)TC * KS : 0);
-        float* v_s = x2_s + (MODE == 1 || MODE == 2 ? (size_t)TC * KS : 0);
+        float* v_s = x2_s + (MODE != 0 ? (size_t)TC * KS : 0);
         float* g1_s = v_s + TC * CTB;
         float* g2_s = g1_s + TC;
         if (aligned) {
             const int quads = dk >> 2;
             for (int idx = tid; idx < n_tok * quads; idx += THREADS) {
-                const int tt = idx / quads, qd = idx - tt * quads, c = hk * dk + 4 * qd;
+                const int tt = idx / quads, qd = idx - tt * quads, c = h * dk + 4 * qd;
                 const float* row = A.proj + (size_t)(t0 + tt) * A.ld;
                 cp_async16(k_s + tt * KS + 4 * qd, row + A.off_k + c);
                 cp_async16(q_s + tt * KS + 4 * qd, row + A.off_q + c);
                 if (MODE == 1) cp_async16(x1_s + tt * KS + 4 * qd, row + A.off_x1 + c);
-                if (MODE == 1 || MODE == 2) cp_async16(x2_s + tt * KS + 4 * qd, A.extra + (size_t)(t0 + tt) * H * dk + c);
+                if (MODE != 0) cp_async16(x2_s + tt * KS + 4 * qd, A.extra + (size_t)(t0 + tt) * H * dk + c);
             }
         } else {
             for (int idx = tid; idx < n_tok * dk; idx += THREADS) {
-                const int tt = idx / dk, r = idx - tt * dk, c = hk * dk + r;
+                const int tt = idx / dk, r = idx - tt * dk, c = h * dk + r;
                 const float* row = A.proj + (size_t)(t0 + tt) * A.ld;
                 cp_async4(k_s + tt * KS + r, row + A.off_k + c);
                 cp_async4(q_s + tt * KS + r, row + A.off_q + c);
                 if (MODE == 1) cp_async4(x1_s + tt * KS + r, row + A.off_x1 + c);
-                if (MODE == 1 || MODE == 2) cp_async4(x2_s + tt * KS + r, A.extra + (size_t)(t0 + tt) * H * dk + c);
+                if (MODE != 0) cp_async4(x2_s + tt * KS + r, A.extra + (size_t)(t0 + tt) * H * dk + c);
             }
         }
         if (KS > dk) {
@@ -183,7 +162,7 @@ __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs
                 k_s[tt * KS + r] = 0.f;
                 q_s[tt * KS + r] = 0.f;
                 if (MODE == 1) x1_s[tt * KS + r] = 0.f;
-                if (MODE == 1 || MODE == 2) x2_s[tt * KS + r] = 0.f;
+                if (MODE != 0) x2_s[tt * KS + r] = 0.f;
             }
         }
         for (int idx = tid; idx < n_tok * CTB; idx += THREADS) {
@@ -196,11 +175,6 @@ __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs
             cp_async4(g1_s + tid, row + A.off_x1 + h);
             cp_async4(g2_s + tid, row + A.off_x2 + h);
         }
-        if (MODE >= 3 && tid < n_tok) {
-            const float* row = A.gates + (size_t)(t0 + tid) * A.gates_ld;
-            if (MODE == 3) cp_async4(g1_s + tid, row + A.off_x1 + h);
-            cp_async4(g2_s + tid, row + A.off_x2 + h);
-        }
     };
     __syncthreads();                               // the tile has been read: its place is the stages' now
     request(t_begin, 0);
@@ -211,32 +185,12 @@ __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs
         float* q_s = k_s + (size_t)TC * KS;
         float* x1_s = q_s + (size_t)TC * KS;
         float* x2_s = x1_s + (MODE == 1 ? (size_t)TC * KS : 0);
-        float* v_s = x2_s + (MODE == 1 || MODE == 2 ? (size_t)TC * KS : 0);
+        float* v_s = x2_s + (MODE != 0 ? (size_t)TC * KS : 0);
         float* g1_s = v_s + TC * CTB;
         float* g2_s = g1_s + TC;
         cp_async_wait_all();
         __syncthreads();                           // this chunk's vectors have landed; the chunk before has been stored
-        if (MODE >= 3 && tid < n_tok) {
-            float keep, add;
-            head_gates<MODE>(A, h, MODE == 3 ? g1_s[tid] : 0.f, g2_s[tid], keep, add);
-            a_s[tid] = keep;
-            b_s[tid] = add;
-        }
-        if (MODE == 3) {                           // unit keys and queries, a warp a token
-            for (int tt = warp; tt < n_tok; tt += THREADS / 32) {
-                float ksq = 0.f, qsq = 0.f;
-                for (int r = lane; r < dk; r += 32) {
-                    ksq += k_s[tt * KS + r] * k_s[tt * KS + r];
-                    qsq += q_s[tt * KS + r] * q_s[tt * KS + r];
-                }
-                const float ik = 1.0f / sqrtf(warp_sum(ksq) + 1e-6f), iq = A.q_scale / sqrtf(warp_sum(qsq) + 1e-6f);
-                for (int r = lane; r < dk; r += 32) {
-                    k_s[tt * KS + r] *= ik;
-                    q_s[tt * KS + r] *= iq;
-                }
-            }
-        }
-        for (int idx = tid; MODE < 3 && idx < n_tok * dk; idx += THREADS) {
+        for (int idx = tid; idx < n_tok * dk; idx += THREADS) {
             const int tt = idx / dk, r = idx - tt * dk, c = h * dk + r;
             if (MODE == 0) {
                 q_s[tt * KS + r] *= A.q_scale;
@@ -329,64 +283,6 @@ __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs
                             nq[u] += n_reg[j] * q_s[tt * KS + r];
                         }
                     }
-                } else if (MODE == 3) {
-                    const float a_t = a_s[tt], b_t = b_s[tt];
-                    float part[4] = {0.f, 0.f, 0.f, 0.f};
-                    float kk[NR];
-#pragma unroll
-                    for (int i0 = 0; i0 < NR; i0 += V4) {
-                        if (V4 == 4) {
-                            *reinterpret_cast<float4*>(kk + i0) = *reinterpret_cast<const float4*>(k + i0);
-                        } else {
-#pragma unroll
-                            for (int e = 0; e < V4; ++e) kk[i0 + e] = k[i0 + e];
-                        }
-#pragma unroll
-                        for (int e = 0; e < V4; ++e) part[e & 3] = fmaf(kk[i0 + e], Sr[i0 + e], part[e & 3]);
-                    }
-                    float ks = (part[0] + part[1]) + (part[2] + part[3]);
-#pragma unroll
-                    for (int o = CW; o <= 16; o <<= 1) ks += __shfl_xor_sync(0xffffffffu, ks, o);
-                    const float write = b_t * (v_c - a_t * ks);
-                    part[0] = part[1] = part[2] = part[3] = 0.f;
-#pragma unroll
-                    for (int i0 = 0; i0 < NR; i0 += V4) {
-                        float qq[V4];
-                        if (V4 == 4) {
-                            *reinterpret_cast<float4*>(qq) = *reinterpret_cast<const float4*>(q + i0);
-                        } else {
-#pragma unroll
-                            for (int e = 0; e < V4; ++e) qq[e] = q[i0 + e];
-                        }
-#pragma unroll
-                        for (int e = 0; e < V4; ++e) {
-                            const float s = fmaf(kk[i0 + e], write, a_t * Sr[i0 + e]);
-                            Sr[i0 + e] = s;
-                            part[e & 3] = fmaf(s, qq[e], part[e & 3]);
-                        }
-                    }
-                    acc[u] = (part[0] + part[1]) + (part[2] + part[3]);
-                } else if (MODE == 4) {
-                    const float a_t = a_s[tt], dx = b_s[tt] * v_c;
-                    float part[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-                    for (int i0 = 0; i0 < NR; i0 += V4) {
-                        float kk[V4], qq[V4];
-                        if (V4 == 4) {
-                            *reinterpret_cast<float4*>(kk) = *reinterpret_cast<const float4*>(k + i0);
-                            *reinterpret_cast<float4*>(qq) = *reinterpret_cast<const float4*>(q + i0);
-                        } else {
-#pragma unroll
-                            for (int e = 0; e < V4; ++e) { kk[e] = k[i0 + e]; qq[e] = q[i0 + e]; }
-                        }
-#pragma unroll
-                        for (int e = 0; e < V4; ++e) {
-                            const float s = fmaf(kk[e], dx, a_t * Sr[i0 + e]);
-                            Sr[i0 + e] = s;
-                            part[e & 3] = fmaf(s, qq[e], part[e & 3]);
-                        }
-                    }
-                    acc[u] = (part[0] + part[1]) + (part[2] + part[3]);
                 } else if (MODE == 2) {
                     const float* __restrict__ decay = x2_s + tt * KS + r0;
                     float part[4] = {0.f, 0.f, 0.f, 0.f};
@@ -474,7 +370,6 @@ __global__ void __launch_bounds__(THREADS, NR <= 8 ? 2 : 1) scan_kernel(ScanArgs
                 for (int w = 0; w < 8; ++w) nq += nqp[tt * 8 + w];
                 o = o / (fmaxf(fabsf(nq), expf(-m_s[tt])) + 1e-6f);
             }
-            if (MODE == 4) o = fmaf(A.d_skip[h], v_s[idx], o);
             A.out[(size_t)(t0 + tt) * H * dv + h * dv + c0 + c] = o;
         }
     }
@@ -510,7 +405,6 @@ __global__ void __launch_bounds__(THREADS, NR <= 16 ? 4 : 1) scan_decode_kernel(
     pdl_enter();
     const int dk = A.dk, dv = A.dv, H = A.H;
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * CT;
-    const int hk = MODE >= 3 ? h / A.share : h;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r0 = warp * NR;
     const int t = A.q_start[seq];
     if (A.q_start[seq + 1] <= t) return;
@@ -538,7 +432,7 @@ __global__ void __launch_bounds__(THREADS, NR <= 16 ? 4 : 1) scan_decode_kernel(
         b = expf(ig - m_new);
     }
     for (int r = tid; r < dk; r += THREADS) {
-        const int c = hk * dk + r;
+        const int c = h * dk + r;
         const float kr = row[A.off_k + c], qr = row[A.off_q + c] * A.q_scale;
         k_s[r] = kr;
         q_s[r] = qr;
@@ -548,10 +442,7 @@ __global__ void __launch_bounds__(THREADS, NR <= 16 ? 4 : 1) scan_decode_kernel(
             nq += n * qr;
         } else if (MODE == 2) {
             x2_s[r] = expf(log_sigmoidf_(A.extra[(size_t)t * H * dk + c] + A.bias2[c]) * A.cap);
-        } else if (MODE == 3) {
-            ksq += kr * kr;
-            nq += row[A.off_q + c] * row[A.off_q + c];
-        } else if (MODE == 1) {
+        } else {
             x1_s[r] = sigmoidf_(row[A.off_x1 + c] + A.bias1[c]);
             x2_s[r] = expf(-0.60653065971263342f * sigmoidf_(A.extra[(size_t)t * H * dk + c] + A.bias2[c]));
             ksq += kr * kr;
@@ -560,17 +451,9 @@ __global__ void __launch_bounds__(THREADS, NR <= 16 ? 4 : 1) scan_decode_kernel(
     if (MODE == 0) {
         nq = warp_sum(nq);
         if (lane == 0) nqp[warp] = nq;
-    } else if (MODE == 1 || MODE == 3) {
+    } else if (MODE == 1) {
         ksq = warp_sum(ksq);
         if (lane == 0) part[warp] = ksq;
-        if (MODE == 3) {
-            nq = warp_sum(nq);
-            if (lane == 0) nqp[warp] = nq;
-        }
-    }
-    if (MODE >= 3) {
-        const float* gt = A.gates + (size_t)t * A.gates_ld;
-        head_gates<MODE>(A, h, MODE == 3 ? gt[A.off_x1 + h] : 0.f, gt[A.off_x2 + h], a, b);
     }
     __syncthreads();
     const float v_c = col_ok ? row[A.off_v + h * dv + c0 + lane] : 0.f;
@@ -595,57 +478,6 @@ __global__ void __launch_bounds__(THREADS, NR <= 16 ? 4 : 1) scan_decode_kernel(
         }
         if (tid == 0)
             for (int cp = 0; cp < copies; ++cp) st_nm[(size_t)cp * (dk + 1) + dk] = m_new;
-    } else if (MODE == 3) {
-        float sq = 0.f, sqq = 0.f;
-#pragma unroll
-        for (int w = 0; w < 8; ++w) { sq += part[w]; sqq += nqp[w]; }
-        const float ik = 1.0f / sqrtf(sq + 1e-6f), iq = 1.0f / sqrtf(sqq + 1e-6f);      // q_scale is in q_s already
-        float ks = 0.f;
-#pragma unroll
-        for (int i = 0; i < NR; ++i)
-            if (r0 + i < dk) ks = fmaf(k_s[r0 + i] * ik, Sr[i], ks);
-        red[warp][lane] = ks;
-        __syncthreads();
-        ks = 0.f;
-#pragma unroll
-        for (int w = 0; w < 8; ++w) ks += red[w][lane];
-        const float write = b * (v_c - a * ks);
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int r = r0 + i;
-            if (r < dk) {
-                const float s = fmaf(k_s[r] * ik, write, a * Sr[i]);
-                if (col_ok) st[(size_t)r * dv + c0 + lane] = s;
-                acc = fmaf(s, q_s[r] * iq, acc);
-            }
-        }
-        red2[warp][lane] = acc;
-        __syncthreads();
-        if (warp == 0 && col_ok) {
-            float o = 0.f;
-#pragma unroll
-            for (int w = 0; w < 8; ++w) o += red2[w][lane];
-            A.out[(size_t)t * H * dv + h * dv + c0 + lane] = o;
-        }
-    } else if (MODE == 4) {
-        const float dx = b * v_c;
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int r = r0 + i;
-            if (r < dk) {
-                const float s = fmaf(k_s[r], dx, a * Sr[i]);
-                if (col_ok) st[(size_t)r * dv + c0 + lane] = s;
-                acc = fmaf(s, q_s[r], acc);
-            }
-        }
-        red2[warp][lane] = acc;
-        __syncthreads();
-        if (warp == 0 && col_ok) {
-            float o = A.d_skip[h] * v_c;
-#pragma unroll
-            for (int w = 0; w < 8; ++w) o += red2[w][lane];
-            A.out[(size_t)t * H * dv + h * dv + c0 + lane] = o;
-        }
     } else if (MODE == 2) {
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
@@ -778,8 +610,6 @@ static int launch_scan(int mode, ScanArgs& A, int num_seqs, int longest, cudaStr
     if (A.H > 65535) SPY_FAIL("recurrence: %d heads exceed the grid limit", A.H);
     if ((A.dv + CT - 1) / CT > 65535) SPY_FAIL("recurrence: a value size of %d exceeds the grid limit", A.dv);
     if (mode == 2) return launch_scan_mode<2>(A, num_seqs, longest, stream);
-    if (mode == 3) return launch_scan_mode<3>(A, num_seqs, longest, stream);
-    if (mode == 4) return launch_scan_mode<4>(A, num_seqs, longest, stream);
     return mode == 0 ? launch_scan_mode<0>(A, num_seqs, longest, stream) : launch_scan_mode<1>(A, num_seqs, longest, stream);
 }
 
@@ -815,29 +645,6 @@ extern "C" int spy_gla_scan(const float* proj, long long ld, int off_q, int off_
     ScanArgs A = {proj, ld, off_q, off_k, off_v, 0, 0, decay_pre, nullptr, decay_bias, state, (long long)dk * dv, num_slots, q_start, state_slot, out,
                   H, dk, dv, q_scale, inv_tau, status};
     return launch_scan(2, A, num_seqs, longest, stream);
-}
-
-// The two with one decay a head.  proj [T, ld] holds q, k ([heads / share, dk] each) and v ([H, dv]) at `off_*`; gates [T, gates_ld] the
-// pre-activations; a_log, dt_bias (and d_skip) [H].  State [slots, H, dk, dv].
-extern "C" int spy_gated_delta_scan(const float* proj, long long ld, int off_q, int off_k, int off_v, const float* gates, long long gates_ld, int off_rate,
-                                    int off_decay, const float* a_log, const float* dt_bias, float* state, int num_slots, const int* q_start,
-                                    const int* state_slot, int num_seqs, int longest, float* out, int H, int share, int dk, int dv, float q_scale,
-                                    int* status, cudaStream_t stream)
-{
-    if (share <= 0 || H % share != 0) SPY_FAIL("gated delta rule: %d heads do not share keys by %d", H, share);
-    ScanArgs A = {proj, ld, off_q, off_k, off_v, off_rate, off_decay, nullptr, nullptr, nullptr, state, (long long)dk * dv, num_slots, q_start, state_slot, out,
-                  H, dk, dv, q_scale, 1.0f, status, share, gates, gates_ld, a_log, dt_bias, nullptr};
-    return launch_scan(3, A, num_seqs, longest, stream);
-}
-
-extern "C" int spy_ssd_scan(const float* proj, long long ld, int off_c, int off_b, int off_x, const float* gates, long long gates_ld, int off_dt,
-                            const float* a_log, const float* dt_bias, const float* d_skip, float* state, int num_slots, const int* q_start,
-                            const int* state_slot, int num_seqs, int longest, float* out, int H, int share, int n, int dv, int* status, cudaStream_t stream)
-{
-    if (share <= 0 || H % share != 0) SPY_FAIL("state-space dual scan: %d heads do not share B and C by %d", H, share);
-    ScanArgs A = {proj, ld, off_c, off_b, off_x, 0, off_dt, nullptr, nullptr, nullptr, state, (long long)n * dv, num_slots, q_start, state_slot, out,
-                  H, n, dv, 1.0f, 1.0f, status, share, gates, gates_ld, a_log, dt_bias, d_skip};
-    return launch_scan(4, A, num_seqs, longest, stream);
 }
 
 // ---- what follows a recurrence: unit root mean square per head, a weight, a gate (sigmoid, or SiLU) -------------

@@ -547,6 +547,15 @@ def _head_gate_checks(what, proj, offsets, sizes, gates, cols, per_head, state, 
         raise KernelError(f"{what}: the column offsets or the heads' parameters do not fit")
 
 
+def _head_scan_scratch(tokens: int, num_seqs: int, heads: int, longest: int, device):
+    """The coefficients' scratch of a step with prompt portions, or None when every request brings one token."""
+    if longest <= 1:
+        return None
+    lib = build.load("head_scan")
+    lib.spy_head_scan_scratch.restype = ctypes.c_longlong
+    return torch.empty(int(lib.spy_head_scan_scratch(tokens, num_seqs, heads)), dtype=torch.float32, device=device)
+
+
 def gated_delta_scan(proj: torch.Tensor, offsets, gates: torch.Tensor, rate_col: int, decay_col: int, a_log: torch.Tensor, dt_bias: torch.Tensor,
                      state: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, num_seqs: int, out: torch.Tensor, heads: int, share: int, dk: int,
                      dv: int, q_scale: float, status: Optional[torch.Tensor] = None, longest: Optional[int] = None) -> torch.Tensor:
@@ -558,9 +567,11 @@ def gated_delta_scan(proj: torch.Tensor, offsets, gates: torch.Tensor, rate_col:
     oq, ok, ov = (int(o) for o in offsets)
     _head_gate_checks("gated delta rule", proj, (oq, ok, ov), (heads // max(share, 1) * dk,) * 2 + (heads * dv,), gates, (rate_col, decay_col), (a_log, dt_bias), state,
                       heads, dk, dv, share)
-    _call("recurrence", "spy_gated_delta_scan", _ptr(proj), ctypes.c_longlong(proj.shape[1]), oq, ok, ov, _ptr(gates), ctypes.c_longlong(gates.shape[1]),
+    longest = int(longest or proj.shape[0])
+    scratch = _head_scan_scratch(proj.shape[0], int(num_seqs), int(heads), longest, proj.device)
+    _call("head_scan", "spy_gated_delta_scan", _ptr(proj), ctypes.c_longlong(proj.shape[1]), oq, ok, ov, _ptr(gates), ctypes.c_longlong(gates.shape[1]),
           int(rate_col), int(decay_col), _ptr(a_log), _ptr(dt_bias), _ptr(state), state.shape[0], _ptr(q_start), _ptr(state_slot), int(num_seqs),
-          int(longest or proj.shape[0]), _ptr(out), int(heads), int(share), int(dk), int(dv), ctypes.c_float(q_scale), _ptr(status), _stream())
+          proj.shape[0], longest, _ptr(out), int(heads), int(share), int(dk), int(dv), ctypes.c_float(q_scale), _ptr(scratch), _ptr(status), _stream())
     return out
 
 
@@ -574,9 +585,11 @@ def ssd_scan(proj: torch.Tensor, offsets, gates: torch.Tensor, dt_col: int, a_lo
     ox, ob, oc = (int(o) for o in offsets)
     _head_gate_checks("state-space dual scan", proj, (ox, ob, oc), (heads * dv,) + (heads // max(share, 1) * n,) * 2, gates, (dt_col,), (a_log, dt_bias, d_skip), state,
                       heads, n, dv, share)
-    _call("recurrence", "spy_ssd_scan", _ptr(proj), ctypes.c_longlong(proj.shape[1]), oc, ob, ox, _ptr(gates), ctypes.c_longlong(gates.shape[1]), int(dt_col),
+    longest = int(longest or proj.shape[0])
+    scratch = _head_scan_scratch(proj.shape[0], int(num_seqs), int(heads), longest, proj.device)
+    _call("head_scan", "spy_ssd_scan", _ptr(proj), ctypes.c_longlong(proj.shape[1]), oc, ob, ox, _ptr(gates), ctypes.c_longlong(gates.shape[1]), int(dt_col),
           _ptr(a_log), _ptr(dt_bias), _ptr(d_skip), _ptr(state), state.shape[0], _ptr(q_start), _ptr(state_slot), int(num_seqs),
-          int(longest or proj.shape[0]), _ptr(out), int(heads), int(share), int(n), int(dv), _ptr(status), _stream())
+          proj.shape[0], longest, _ptr(out), int(heads), int(share), int(n), int(dv), _ptr(scratch), _ptr(status), _stream())
     return out
 
 

@@ -233,7 +233,7 @@ class _ConvRecurrent(_Recurrent):
         return [self.fused, self.o]
 
     def modules(self):
-        return ["recurrence"] + self.conv.modules() + self.fused.modules() + self.o.modules()
+        return ["head_scan", "recurrence"] + self.conv.modules() + self.fused.modules() + self.o.modules()
 
 
 @register_part("gated_delta_rule")
