@@ -305,12 +305,14 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long log
 }
 
 // One block an expert: its rows' places, in the order of the tokens.  Each warp takes a run of the pairs, counts the expert's
-// pairs in it, and after a prefix over the warps' counts hands out the places.  offsets [experts + 1]; slot [tokens * top]: the
+// pairs in it, and after a prefix over the warps' counts hands out the places.  `pad`: every expert's run starts at a multiple of so
+// many rows (the rows between are nobody's: row_token -1, set by the caller), and tile_expert [num_tiles] tells, for every `pad` rows,
+// whose they are (-1 behind the last run).  offsets [experts + 1]; slot [tokens * top]: the
 // row of each (token, k); row_token, row_w [tokens * top]: each row's token and weight.
 __global__ void __launch_bounds__(1024)
 moe_slots_kernel(const int* __restrict__ choice, const float* __restrict__ choice_w, const int* __restrict__ counts, int pairs,
                  int top, int experts, int* __restrict__ offsets, int* __restrict__ slot, int* __restrict__ row_token,
-                 float* __restrict__ row_w)
+                 float* __restrict__ row_w, int pad, int* __restrict__ tile_expert, int num_tiles)
 {
     __shared__ int warp_count[32];
     __shared__ int first_row;
@@ -327,12 +329,18 @@ moe_slots_kernel(const int* __restrict__ choice, const float* __restrict__ choic
     if (lane == 0) warp_count[warp] = mine_count;
     if (warp == 0) {
         int base = 0;
-        for (int o = lane; o < e; o += 32) base += counts[o];
+        for (int o = lane; o < e; o += 32) base += (counts[o] + pad - 1) / pad * pad;
         for (int o = 16; o > 0; o >>= 1) base += __shfl_xor_sync(0xffffffffu, base, o);
         if (lane == 0) {
             first_row = base;
             offsets[e] = base;
-            if (e == experts - 1) offsets[experts] = base + counts[e];
+            if (e == experts - 1) offsets[experts] = base + (counts[e] + pad - 1) / pad * pad;
+        }
+        if (tile_expert != nullptr) {
+            const int own = (counts[e] + pad - 1) / pad, first = base / pad;
+            for (int i = lane; i < own && first + i < num_tiles; i += 32) tile_expert[first + i] = e;
+            if (e == experts - 1)
+                for (int i = first + own + lane; i < num_tiles; i += 32) tile_expert[i] = -1;
         }
     }
     __syncthreads();
@@ -352,11 +360,13 @@ moe_slots_kernel(const int* __restrict__ choice, const float* __restrict__ choic
     }
 }
 
-// out[r] = in[row_token[r]]: rows of `len` elements of 2 bytes (bf16) or 4, copied 16 bytes at a time where the rows allow it.
+// out[r] = in[row_token[r]] (a row of nobody, token -1, is left as it is): rows of `len` elements of 2 bytes (bf16) or 4, copied 16 bytes at a time where the rows allow it.
 __global__ void gather_rows_kernel(const uint8_t* __restrict__ in, const int* __restrict__ row_token, uint8_t* __restrict__ out, long long row_bytes)
 {
     pdl_enter();
-    const uint8_t* src = in + (long long)row_token[blockIdx.x] * row_bytes;
+    const int token = row_token[blockIdx.x];
+    if (token < 0) return;
+    const uint8_t* src = in + (long long)token * row_bytes;
     uint8_t* dst = out + (long long)blockIdx.x * row_bytes;
     if ((row_bytes & 15) == 0) {
         for (long long i = threadIdx.x * 16LL; i < row_bytes; i += blockDim.x * 16LL) *reinterpret_cast<uint4*>(dst + i) = *reinterpret_cast<const uint4*>(src + i);
@@ -428,10 +438,22 @@ __global__ void moe_combine_kernel(const TR* __restrict__ rows, const int* __res
     }
 }
 
+// Padded runs: enough rows for any counts, and every row nobody's until a pair takes it.
+static int prepare_rows(int tokens, int experts, int top, int pad, const int* tile_expert, int num_rows, int* row_token, cudaStream_t stream)
+{
+    if (pad <= 1) return 0;
+    if (tile_expert == nullptr || num_rows % pad != 0 || (long long)num_rows / pad < (long long)tokens * top / pad + experts)
+        SPY_FAIL("moe_route: %d rows do not hold %d pairs in runs of whole %d rows for %d experts", num_rows, tokens * top, pad, experts);
+    SPY_CUDA(cudaMemsetAsync(row_token, 0xff, sizeof(int) * (size_t)num_rows, stream));
+    return 0;
+}
+
 extern "C" int spy_moe_route(const float* logits, long long logits_ld, int tokens, int experts, int top, int has_shared, int* choice, float* choice_w,
-                             float* shared_w, int* counts, int* offsets, int* slot, int* row_token, float* row_w, cudaStream_t stream)
+                             float* shared_w, int* counts, int* offsets, int* slot, int* row_token, float* row_w, cudaStream_t stream,
+                             int pad, int* tile_expert, int num_rows)
 {
     if (tokens <= 0) return 0;
+    if (int rc = prepare_rows(tokens, experts, top, pad, tile_expert, num_rows, row_token, stream)) return rc;
     if (experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0 || top > experts) SPY_FAIL("moe_route: %d experts (at most %d), top %d", experts, MOE_MAX_EXPERTS, top);
     SPY_CUDA(cudaMemsetAsync(counts, 0, sizeof(int) * experts, stream));
     const int warps = 4;
@@ -440,7 +462,7 @@ extern "C" int spy_moe_route(const float* logits, long long logits_ld, int token
                         tokens, experts, top, has_shared, choice, choice_w, shared_w, counts);
     SPY_CHECK_LAUNCH("moe_route");
     spy_launch(moe_slots_kernel, dim3(experts), dim3(1024), 0, stream, (const int*)choice, (const float*)choice_w, (const int*)counts,
-               tokens * top, top, experts, offsets, slot, row_token, row_w);
+               tokens * top, top, experts, offsets, slot, row_token, row_w, pad < 1 ? 1 : pad, tile_expert, pad > 1 ? num_rows / pad : 0);
     SPY_CHECK_LAUNCH("moe_slots");
     return 0;
 }
@@ -485,9 +507,10 @@ __global__ void moe_pairs_kernel(const float* __restrict__ weights, long long ld
 
 // weights [tokens, ld] float32 (the first `experts` columns are looked at); the other arrays as for spy_moe_route.
 extern "C" int spy_moe_route_weights(const float* weights, long long ld, int tokens, int experts, int top, int* choice, float* choice_w, int* counts,
-                                     int* offsets, int* slot, int* row_token, float* row_w, cudaStream_t stream)
+                                     int* offsets, int* slot, int* row_token, float* row_w, cudaStream_t stream, int pad, int* tile_expert, int num_rows)
 {
     if (tokens <= 0) return 0;
+    if (int rc = prepare_rows(tokens, experts, top, pad, tile_expert, num_rows, row_token, stream)) return rc;
     if (experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0) SPY_FAIL("moe_route_weights: %d experts (at most %d), top %d", experts, MOE_MAX_EXPERTS, top);
     SPY_CUDA(cudaMemsetAsync(counts, 0, sizeof(int) * experts, stream));
     const int warps = 4;
@@ -496,7 +519,7 @@ extern "C" int spy_moe_route_weights(const float* weights, long long ld, int tok
                         choice_w, slot, counts);
     SPY_CHECK_LAUNCH("moe_pairs");
     spy_launch(moe_slots_kernel, dim3(experts), dim3(1024), 0, stream, (const int*)choice, (const float*)choice_w, (const int*)counts,
-               tokens * top, top, experts, offsets, slot, row_token, row_w);
+               tokens * top, top, experts, offsets, slot, row_token, row_w, pad < 1 ? 1 : pad, tile_expert, pad > 1 ? num_rows / pad : 0);
     SPY_CHECK_LAUNCH("moe_slots");
     return 0;
 }

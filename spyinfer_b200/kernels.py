@@ -1575,30 +1575,39 @@ def moe_activation(gate_up: torch.Tensor, logits: torch.Tensor, out: torch.Tenso
     return out
 
 
+def _route_buffers(T: int, experts: int, top: int, pad: int, dev):
+    R = T * top if pad == 1 else (T * top // pad + experts) * pad
+    ints = torch.empty((2 * T * top + R + 2 * experts + 1,), dtype=torch.int32, device=dev)
+    floats = torch.empty((T * top + R,), dtype=torch.float32, device=dev)
+    choice, slot, row_token, rest = ints[:T * top], ints[T * top:2 * T * top], ints[2 * T * top:2 * T * top + R], ints[2 * T * top + R:]
+    tile_expert = torch.empty((R // pad,), dtype=torch.int32, device=dev) if pad > 1 else None
+    return choice, floats[:T * top], rest[:experts], rest[experts:], slot, row_token, floats[T * top:], tile_expert, R
+
+
 def moe_route_general(logits: torch.Tensor, experts: int, top: int, identity: int = 0, correction: Optional[torch.Tensor] = None,
-                      groups: Optional[tuple] = None, has_shared: bool = False, scoring: str = "softmax", group_score: str = "best"):
+                      groups: Optional[tuple] = None, has_shared: bool = False, scoring: str = "softmax", group_score: str = "best", pad: int = 1):
     """As ``moe_route`` for a choice with the options of ``moe_activation`` (identity experts, correction, groups): the (token,
     chosen real expert) pairs of a step sorted by expert.  Returns ``offsets [experts + 1]``, ``slot [T, top]`` (the row of each
     pair, -1 where a token chose fewer real experts than ``top``), ``row_token``, ``row_w`` (``[T top]``, the first ``offsets[-1]``
-    rows count), ``shared_w [T]`` or None, and ``id_weight [T]`` (the chosen identity experts' summed weights) or None."""
+    rows count), ``shared_w [T]`` or None, and ``id_weight [T]`` (the chosen identity experts' summed weights) or None.  ``pad`` as for
+    ``moe_route``."""
     _check(logits, "router logits", torch.float32, 2)
     T, total, dev = logits.shape[0], experts + int(identity), logits.device
     if logits.shape[1] < total + (1 if has_shared else 0):
         raise KernelError("moe_route_general: the logits lack columns")
     weights = torch.empty((T, total + 1), dtype=torch.float32, device=dev)
-    floats = torch.empty((2 * T * top + 2 * T,), dtype=torch.float32, device=dev)
-    choice_w, row_w, shared_w, idw = floats[:T * top], floats[T * top:2 * T * top], floats[2 * T * top:2 * T * top + T], floats[2 * T * top + T:]
+    choice, choice_w, counts, offsets, slot, row_token, row_w, tile_expert, R = _route_buffers(T, experts, top, pad, dev)
+    floats = torch.empty((2 * T,), dtype=torch.float32, device=dev)
+    shared_w, idw = floats[:T], floats[T:]
     count, keep = (int(groups[0]), int(groups[1])) if groups else (0, 0)
     _call("moe", "spy_moe_activation_routed", None, BF16, ctypes.c_longlong(0), _ptr(logits), ctypes.c_longlong(logits.shape[1]), None, BF16,
           ctypes.c_longlong(0), T, int(experts), int(top), 1, ctypes.c_float(0.0), 1 if has_shared else 0, ctypes.c_float(0.0), ctypes.c_float(0.0),
           _ptr(weights), int(identity), _ptr(correction), count, keep, 1, _ptr(idw if identity else None), _ptr(shared_w if has_shared else None), _stream(),
           *_scoring_codes(scoring, group_score))
-    ints = torch.empty((3 * T * top + 2 * experts + 1,), dtype=torch.int32, device=dev)
-    choice, slot, row_token = ints[:T * top], ints[T * top:2 * T * top], ints[2 * T * top:3 * T * top]
-    counts, offsets = ints[3 * T * top:3 * T * top + experts], ints[3 * T * top + experts:]
     _call("moe", "spy_moe_route_weights", _ptr(weights), ctypes.c_longlong(total + 1), T, int(experts), int(top), _ptr(choice), _ptr(choice_w), _ptr(counts),
-          _ptr(offsets), _ptr(slot), _ptr(row_token), _ptr(row_w), _stream())
-    return offsets, slot.view(T, top), row_token, row_w, (shared_w if has_shared else None), (idw if identity else None)
+          _ptr(offsets), _ptr(slot), _ptr(row_token), _ptr(row_w), _stream(), int(pad), _ptr(tile_expert), R)
+    out = (offsets, slot.view(T, top), row_token, row_w, (shared_w if has_shared else None), (idw if identity else None))
+    return out if pad == 1 else out + (tile_expert,)
 
 
 def add_scaled_rows(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -1674,24 +1683,48 @@ def stream_add(stream: torch.Tensor, table: Optional[torch.Tensor], ids: Optiona
     return stream
 
 
-def moe_route(logits: torch.Tensor, experts: int, top: int, has_shared: bool):
+def moe_route(logits: torch.Tensor, experts: int, top: int, has_shared: bool, pad: int = 1):
     """Sorts the (token, chosen expert) pairs of a step by expert.  ``logits [T, >= experts (+ 1)]`` float32 as for
     ``moe_activation``.  Returns ``offsets [experts + 1]`` (where each expert's run of rows starts), ``slot [T, top]`` (the row
     of each pair, the chosen experts in ascending order), ``row_token [T top]``, ``row_w [T top]`` (each row's token and its
-    softmax score over all experts) and ``shared_w [T]`` (sigmoid of the shared gate's logit) or None."""
+    softmax score over all experts) and ``shared_w [T]`` (sigmoid of the shared gate's logit) or None.  ``pad`` above 1: every expert's run
+    starts at a multiple of so many rows, rows of nobody have the token -1, and one more result, ``tile_expert [rows / pad]``, tells whose
+    every ``pad`` rows are (-1 behind the last run)."""
     _check(logits, "router logits", torch.float32, 2)
     T = logits.shape[0]
     if logits.shape[1] < experts + (1 if has_shared else 0):
         raise KernelError("moe_route: the logits lack columns")
     dev = logits.device
-    ints = torch.empty((2 * T * top + T * top + experts + experts + 1,), dtype=torch.int32, device=dev)
-    choice, slot, row_token = ints[:T * top], ints[T * top:2 * T * top], ints[2 * T * top:3 * T * top]
-    counts, offsets = ints[3 * T * top:3 * T * top + experts], ints[3 * T * top + experts:]
-    floats = torch.empty((2 * T * top + T,), dtype=torch.float32, device=dev)
-    choice_w, row_w, shared_w = floats[:T * top], floats[T * top:2 * T * top], floats[2 * T * top:]
+    choice, choice_w, counts, offsets, slot, row_token, row_w, tile_expert, R = _route_buffers(T, experts, top, pad, dev)
+    shared_w = torch.empty((T,), dtype=torch.float32, device=dev)
     _call("moe", "spy_moe_route", _ptr(logits), ctypes.c_longlong(logits.shape[1]), T, int(experts), int(top), int(bool(has_shared)), _ptr(choice),
-          _ptr(choice_w), _ptr(shared_w), _ptr(counts), _ptr(offsets), _ptr(slot), _ptr(row_token), _ptr(row_w), _stream())
-    return offsets, slot.view(T, top), row_token, row_w, (shared_w if has_shared else None)
+          _ptr(choice_w), _ptr(shared_w), _ptr(counts), _ptr(offsets), _ptr(slot), _ptr(row_token), _ptr(row_w), _stream(), int(pad), _ptr(tile_expert), R)
+    out = (offsets, slot.view(T, top), row_token, row_w, (shared_w if has_shared else None))
+    return out if pad == 1 else out + (tile_expert,)
+
+
+def grouped_tile_rows() -> int:
+    """The rows of a tile of ``gemm_grouped``: what an expert's run of rows is padded to."""
+    return int(build.load("gemm_grouped").spy_gemm_grouped_tile_rows())
+
+
+def gemm_grouped(a: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, experts: int, n: int, row_step: int = 0, col_step: int = 0,
+                 out_dtype: Optional[torch.dtype] = None, status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[r] = a[r] @ w[e row_step : e row_step + n, e col_step : e col_step + K]^T`` with ``e = tile_expert[r // tile rows]`` (read on the device;
+    -1: the tile is skipped and its rows of ``out`` are undefined): one product of rows sorted by expert, each tile with its own expert's
+    part of a fused weight, on the tensor cores.  ``a [rows, K]`` bfloat16, rows a multiple of ``grouped_tile_rows()``."""
+    _check(a, "grouped input", torch.bfloat16, 2)
+    ldw = _check_weight(w, "grouped weight", torch.bfloat16)
+    _check(tile_expert, "tile experts", torch.int32, 1)
+    rows, K = a.shape
+    if tile_expert.shape[0] * grouped_tile_rows() != rows:
+        raise KernelError(f"gemm_grouped: {tile_expert.shape[0]} tiles do not fit {rows} rows")
+    out = torch.empty((rows, n), dtype=out_dtype or torch.bfloat16, device=a.device)
+    if status is None:
+        status = status_word(a.device)
+    _call("gemm_grouped", "spy_gemm_grouped", _ptr(a), ctypes.c_longlong(K), rows, K, _ptr(w), ctypes.c_longlong(ldw), w.shape[0], w.shape[1], _ptr(out),
+          _code(out, "grouped output"), ctypes.c_longlong(n), int(n), _ptr(tile_expert), int(experts), int(row_step), int(col_step), _ptr(status), _stream())
+    return out
 
 
 def gather_rows(x: torch.Tensor, row_token: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -1727,7 +1760,7 @@ def moe_combine(rows: torch.Tensor, slot: torch.Tensor, shared: Optional[torch.T
     _check(slot, "slots", torch.int32, 2)
     _check(out, "mixture output", torch.float32, 2)
     T, top = slot.shape
-    if tuple(out.shape) != (T, rows.shape[1]) or rows.shape[0] != T * top:
+    if tuple(out.shape) != (T, rows.shape[1]) or rows.shape[0] < T * top:
         raise KernelError("moe_combine: shapes do not fit")
     if shared is not None:
         _check(shared, "shared expert result", rows.dtype, 2)

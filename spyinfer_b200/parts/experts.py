@@ -9,13 +9,14 @@ All experts' gate and up projections are one product, their down projections one
 side; the kernel between the two multiplies each expert's activation by the token's weight for it, which is exactly zero
 for an expert that the token did not choose.  A token's result therefore does not depend on what else is in the batch.
 
-A step of many tokens (``routed_from`` or more: by default so many that an expert gets 1,024 rows on average, below which its
-products fill too little of the GPU to gain; ``SPYINFER_MOE_ROUTED_FROM`` in the environment sets the number, 0 turns the form
+A step of many tokens (``routed_from`` or more; ``SPYINFER_MOE_ROUTED_FROM`` in the environment sets the number, 0 turns the form
 off; never inside a captured graph) takes the routed form instead: the (token, chosen expert) pairs are sorted by expert on the
 device, the tokens' rows gathered in that order, each expert's two products run on its own run of rows (views of the same
 fused weights, nothing stored twice), and every token's ``top`` results and the shared expert's are added in a fixed order in
-32-bit.  The experts' row counts are read back once a layer to size the products.  Weights and arithmetic are the same, so the
-two forms differ by the order of sums only.  Both forms serve the options of the choice (a correction for the choice only, groups
+32-bit.  On the bfloat16 path the products of all experts are one launch each (``gemm_grouped``: the runs are padded to whole tiles, a
+tile finds its expert on the device, nothing is read back); with sizes that launch does not take, and in 32-bit, the experts' row
+counts are read back once a layer to size a product for each.  Weights and arithmetic are the same, so the two forms differ by the
+order of sums only.  Both forms serve the options of the choice (a correction for the choice only, groups
 of router outputs, identity experts, whose pairs take no rows) and both activations.
 """
 from __future__ import annotations
@@ -73,11 +74,18 @@ class ExpertMixture(FeedForward):
         self.prefix = params.get("prefix", "")
         self.cols = self.experts * self.ff + self.shared_ff
         self.router = self.gate_up = self.down = None
-        default = -(-1024 * self.experts // self.top)
+        # the products' rows: tokens * experts in the dense form; tokens * top in the routed one, and for every expert half a tile of padding
+        # (one launch) or, with a product for each expert, so many that it fills the GPU
+        self.grouped = ctx.dtype == torch.bfloat16 and self.ff % 8 == 0 and self.hidden % 8 == 0
+        default = self._grouped_from() if self.grouped else -(-1024 * self.experts // self.top)
         try:
             self.routed_from = int(os.environ.get("SPYINFER_MOE_ROUTED_FROM", params.get("routed_from", default)))
         except ValueError:
             self.routed_from = default
+
+    def _grouped_from(self) -> int:
+        spare = 2 * self.experts - 3 * self.top                    # half the dense form's rows must be enough and some over
+        return max(512, -(-3 * 128 * self.experts // spare)) if spare > 0 else 0
 
     def weight_decls(self):
         p, W = self.prefix, self.hidden
@@ -105,10 +113,13 @@ class ExpertMixture(FeedForward):
             self.correction = tensors[p + "correction"].float().contiguous()
 
     def modules(self):
-        return ["moe"] + self.router.modules() + self.gate_up.modules() + self.down.modules()
+        return ["moe"] + (["gemm_grouped"] if self._one_launch() else []) + self.router.modules() + self.gate_up.modules() + self.down.modules()
 
     def linears(self):
         return [self.router, self.gate_up, self.down]
+
+    def _one_launch(self) -> bool:
+        return self.grouped and self.gate_up is not None and self.gate_up.fast and self.down.fast
 
     def forward(self, x):
         if 0 < self.routed_from <= x.shape[0] and self.top < self.outputs and not torch.cuda.is_current_stream_capturing():
@@ -132,18 +143,11 @@ class ExpertMixture(FeedForward):
             return self.down(y, defer=self.defer_output)
         return kernels.add_scaled_rows(self.down(y, out_dtype=torch.float32), x, idw)
 
-    def _routed(self, x):
-        T, E, top, ff, sff, dev = x.shape[0], self.experts, self.top, self.ff, self.shared_ff, x.device
-        logits = self.router(x, out_dtype=torch.float32)
-        idw = None
-        if self.plain_choice:
-            offsets, slot, row_token, row_w, shared_w = kernels.moe_route(logits, E, top, bool(sff))
-        else:
-            offsets, slot, row_token, row_w, shared_w, idw = kernels.moe_route_general(logits, E, top, self.identity, self.correction, self.groups, bool(sff),
-                                                                                               scoring=self.scoring, group_score=self.group_score)
+    def _products_one_by_one(self, x, offsets, row_token, row_w):
+        T, E, top, ff, dev = x.shape[0], self.experts, self.top, self.ff, x.device
         starts = offsets.cpu().tolist()                      # the layer's one read-back: the experts' row counts size their products
-        R, n = T * top, starts[E]                            # n rows are in use: a token may have chosen fewer real experts than `top`
-        results = torch.empty((R, self.hidden), dtype=torch.float32, device=dev)
+        n = starts[E]                                        # n rows are in use: a token may have chosen fewer real experts than `top`
+        results = torch.empty((T * top, self.hidden), dtype=torch.float32, device=dev)
         if n:
             rows = kernels.gather_rows(x, row_token[:n], torch.empty((n, self.hidden), dtype=x.dtype, device=dev))
             gu = torch.empty((n, 2 * ff), dtype=self.ctx.dtype, device=dev)
@@ -156,6 +160,27 @@ class ExpertMixture(FeedForward):
                 a, b = starts[e], starts[e + 1]
                 if b > a:
                     self.down.part(y[a:b], cols=(ff * e, ff * (e + 1)), out=results[a:b])
+        return results
+
+    def _routed(self, x):
+        T, E, top, ff, sff, dev = x.shape[0], self.experts, self.top, self.ff, self.shared_ff, x.device
+        logits = self.router(x, out_dtype=torch.float32)
+        idw = None
+        grouped = self._one_launch()
+        pad = kernels.grouped_tile_rows() if grouped else 1
+        if self.plain_choice:
+            offsets, slot, row_token, row_w, shared_w, *tiles = kernels.moe_route(logits, E, top, bool(sff), pad=pad)
+        else:
+            offsets, slot, row_token, row_w, shared_w, idw, *tiles = kernels.moe_route_general(
+                logits, E, top, self.identity, self.correction, self.groups, bool(sff), scoring=self.scoring, group_score=self.group_score, pad=pad)
+        if grouped:
+            rows = kernels.gather_rows(x, row_token, torch.empty((row_token.shape[0], self.hidden), dtype=x.dtype, device=dev))
+            gu = kernels.gemm_grouped(rows, self.gate_up.weight, tiles[0], E, 2 * ff, row_step=2 * ff)
+            y = kernels.expert_activation(gu, row_w, torch.empty((rows.shape[0], ff), dtype=self.ctx.dtype, device=dev), self.limit, self.slope,
+                                          activation=self.activation)
+            results = kernels.gemm_grouped(y, self.down.weight, tiles[0], E, self.hidden, col_step=ff, out_dtype=torch.float32)
+        else:
+            results = self._products_one_by_one(x, offsets, row_token, row_w)
         shared = None
         if sff:
             sgu = self.gate_up.part(x, rows=(2 * ff * E, 2 * ff * E + 2 * sff), out_dtype=self.ctx.dtype)

@@ -663,6 +663,45 @@ def test_sigmoid_scores_and_groups_by_their_two_best(dtype, experts, top, ff, gr
         assert np.allclose([float(row_w[i]) for i in rows], [float(x) for x in want_w[:, e] if x != 0], atol=1e-6)
 
 
+@gpu
+@pytest.mark.parametrize("experts,top,hidden,ff,T", [(6, 2, 64, 24, 50), (8, 3, 136, 200, 700), (1, 1, 256, 64, 300), (5, 1, 40, 16, 9), (16, 4, 512, 320, 1100)])
+def test_one_launch_multiplies_every_tile_with_its_own_experts_weight(experts, top, hidden, ff, T):
+    """Pairs sorted by expert into runs of whole tiles: every pair has a row of its own expert's run, the rows between belong to nobody,
+    and the two products (row parts of one fused weight, column parts of another) equal each expert's own; an expert that nobody
+    chose has no tile."""
+    from spyinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(T + ff)
+    logits = torch.randn(T, experts, generator=g) * 1.5
+    if experts > 2:
+        logits[:, 1] = -30.0                                       # an expert without rows
+    idx = torch.topk(torch.sigmoid(logits), top, dim=-1).indices.sort(dim=-1).values
+    pad = kernels.grouped_tile_rows()
+    offsets, slot, row_token, row_w, _, _, tiles = kernels.moe_route_general(logits.cuda(), experts, top, scoring="sigmoid", pad=pad)
+    starts, slots, tokens, owner = offsets.cpu().tolist(), slot.cpu(), row_token.cpu(), tiles.cpu().tolist()
+    assert all(v % pad == 0 for v in starts) and tokens.shape[0] == len(owner) * pad >= starts[experts]
+    for t in range(T):
+        for k in range(top):
+            r = int(slots[t, k])
+            assert int(tokens[r]) == t and owner[r // pad] == int(idx[t, k])
+    assert int((tokens >= 0).sum()) == T * top and owner[starts[experts] // pad:] == [-1] * (len(owner) - starts[experts] // pad)
+    x = torch.randn(T, hidden, generator=g).to(torch.bfloat16)
+    w = (torch.randn(experts * 2 * ff, hidden, generator=g) / hidden ** 0.5).to(torch.bfloat16)
+    rows = kernels.gather_rows(x.cuda(), row_token, torch.empty((tokens.shape[0], hidden), dtype=torch.bfloat16, device="cuda"))
+    gu = kernels.gemm_grouped(rows, w.cuda(), tiles, experts, 2 * ff, row_step=2 * ff)
+    d = (torch.randn(hidden, experts * ff, generator=g) / ff ** 0.5).to(torch.bfloat16)
+    y = torch.randn(tokens.shape[0], ff, generator=g).to(torch.bfloat16)
+    down = kernels.gemm_grouped(y.cuda(), d.cuda(), tiles, experts, hidden, col_step=ff, out_dtype=torch.float32)
+    gu, down = gu.float().cpu().double(), down.cpu().double()
+    for e in range(experts):
+        mine = [r for r in range(starts[e], starts[e + 1]) if tokens[r] >= 0]
+        if not mine:
+            continue
+        want = x[tokens[mine].long()].double() @ w[2 * ff * e:2 * ff * (e + 1)].double().T
+        assert torch.allclose(gu[mine], want, atol=2e-2, rtol=1e-2), e
+        assert torch.allclose(down[mine], y[mine].double() @ d[:, ff * e:ff * (e + 1)].double().T, atol=1e-4, rtol=1e-4), e
+
+
 # ---- whole models through the step function ---------------------------------------------------------------
 
 @gpu
