@@ -863,7 +863,15 @@ def zonevik_workload(args) -> int:
                     rate(block, "recurrence.spy_gate_group_norm", nbytes=float(rows) * n_par * inner * (4 + 4 + 2))
                     rate(block, "recurrence.spy_gated_head_norm", nbytes=float(rows) * n_delta * d_v * (4 + 4 + 2))
                     cols = z["experts"] * z["expert_ff"]
-                    rate(block, "moe.spy_moe_activation_routed", nbytes=float(layers) * rows * (z["top"] * z["expert_ff"] * 4 + cols * 2))
+                    if "moe.spy_moe_combine" in res[block]:               # the routed form: two products of a token's chosen experts only
+                        pairs = float(layers) * rows * z["top"]
+                        rate(block, "gemm_grouped.spy_gemm_grouped", flops=pairs * 3 * W * z["expert_ff"] * 2)
+                        rate(block, "moe.spy_expert_activation", nbytes=pairs * z["expert_ff"] * 6)
+                        rate(block, "moe.spy_gather_rows", nbytes=pairs * W * 4)
+                        rate(block, "moe.spy_moe_combine", nbytes=(pairs + layers * rows) * W * 4)
+                    else:
+                        rate(block, "moe.spy_moe_activation_routed", nbytes=float(layers) * rows * (z["top"] * z["expert_ff"] * 4 + cols * 2))
+                    rate(block, "gemm_simt.spy_gemm_simt", nbytes=float(layers) * rows * W * 2)
             elif name == "qwen3":
                 rate("kernels_prefill", "attention_tc.spy_attention_tc", flops=attn(layers, full))
                 rate("kernels_decode_b64", "attention_decode.spy_attention_decode", nbytes=cache(layers, ctx + 1))

@@ -129,6 +129,61 @@ gemm_skinny_kernel(const TA* __restrict__ A, long long lda, const TW* __restrict
     }
 }
 
+// The same in runs of four (16-byte accesses of 32-bit rows, 8-byte ones of bfloat16 rows) where the rows allow it.
+__device__ __forceinline__ void load4(const float* p, float (&v)[4])
+{
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+}
+__device__ __forceinline__ void load4(const bf16* p, float (&v)[4])
+{
+    const uint2 x = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&x.x), b = *reinterpret_cast<const __nv_bfloat162*>(&x.y);
+    v[0] = __low2float(a); v[1] = __high2float(a); v[2] = __low2float(b); v[3] = __high2float(b);
+}
+
+template <typename TA, typename TW, typename TC, int NG>
+__global__ void __launch_bounds__(SKINNY_THREADS)
+gemm_skinny_quads_kernel(const TA* __restrict__ A, long long lda, const TW* __restrict__ W, long long ldw, TC* __restrict__ C, long long ldc, int N, int K)
+{
+    __shared__ float part[SKINNY_THREADS / 32][NG];
+    pdl_enter();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const long long m = blockIdx.x;
+    const TA* a = A + m * lda;
+    for (int n0 = 0; n0 < N; n0 += NG) {
+        float acc[NG];
+#pragma unroll
+        for (int j = 0; j < NG; ++j) acc[j] = 0.f;
+        for (int k = 4 * threadIdx.x; k < K; k += 4 * SKINNY_THREADS) {
+            float av[4];
+            load4(a + k, av);
+#pragma unroll
+            for (int j = 0; j < NG; ++j)
+                if (n0 + j < N) {
+                    float w[4];
+                    load4(W + (size_t)(n0 + j) * ldw + k, w);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) acc[j] = fmaf(av[e], w[e], acc[j]);
+                }
+        }
+#pragma unroll
+        for (int j = 0; j < NG; ++j) {
+            if (n0 + j >= N) break;                       // the same for every thread
+            const float sum = warp_sum(acc[j]);
+            if (lane == 0) part[warp][j] = sum;
+        }
+        __syncthreads();
+        if (threadIdx.x < NG && n0 + threadIdx.x < N) {
+            float sum = 0.f;
+#pragma unroll
+            for (int w = 0; w < SKINNY_THREADS / 32; ++w) sum += part[w][threadIdx.x];
+            C[m * ldc + n0 + threadIdx.x] = from_f32<TC>(sum);
+        }
+        __syncthreads();
+    }
+}
+
 extern "C" int spy_gemm_simt(const void* A, int a_dtype, long long lda, const void* W, int w_dtype, long long ldw, void* C, int c_dtype,
                              long long ldc, int M, int N, int K, cudaStream_t stream)
 {
@@ -139,7 +194,16 @@ extern "C" int spy_gemm_simt(const void* A, int a_dtype, long long lda, const vo
         SPY_DISPATCH_DTYPE(a_dtype, TA, {
             SPY_DISPATCH_DTYPE(w_dtype, TW, {
                 SPY_DISPATCH_DTYPE(c_dtype, TC, {
-                    spy_launch(gemm_skinny_kernel<TA, TW, TC, 1>, dim3((unsigned)M), dim3(SKINNY_THREADS), 0, stream, (const TA*)A, lda,
+                    const bool quads = K % 4 == 0 && lda % 4 == 0 && ldw % 4 == 0 && reinterpret_cast<uintptr_t>(A) % (4 * sizeof(TA)) == 0
+                                       && reinterpret_cast<uintptr_t>(W) % (4 * sizeof(TW)) == 0;
+                    if (quads && N <= 8)
+                        spy_launch(gemm_skinny_quads_kernel<TA, TW, TC, 8>, dim3((unsigned)M), dim3(SKINNY_THREADS), 0, stream, (const TA*)A, lda,
+                                   (const TW*)W, ldw, (TC*)C, ldc, N, K);
+                    else if (quads)
+                        spy_launch(gemm_skinny_quads_kernel<TA, TW, TC, 16>, dim3((unsigned)M), dim3(SKINNY_THREADS), 0, stream, (const TA*)A, lda,
+                                   (const TW*)W, ldw, (TC*)C, ldc, N, K);
+                    else
+                        spy_launch(gemm_skinny_kernel<TA, TW, TC, 1>, dim3((unsigned)M), dim3(SKINNY_THREADS), 0, stream, (const TA*)A, lda,
                                (const TW*)W, ldw, (TC*)C, ldc, M, N, K);
                 })
             })

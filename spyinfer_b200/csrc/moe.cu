@@ -427,6 +427,27 @@ __global__ void moe_combine_kernel(const TR* __restrict__ rows, const int* __res
 {
     pdl_enter();
     const long long t = blockIdx.x;
+    if constexpr (sizeof(TR) == 4) {
+        if ((len & 3) == 0) {                        // rows of whole quads (the tensors start on 16-byte borders)
+            for (int i = threadIdx.x * 4; i < len; i += blockDim.x * 4) {
+                float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+                auto add = [&](const float4 v) {
+                    acc.x += v.x;
+                    acc.y += v.y;
+                    acc.z += v.z;
+                    acc.w += v.w;
+                };
+#pragma unroll 4
+                for (int k = 0; k < top; ++k) {
+                    const int r = slot[t * top + k];
+                    if (r >= 0) add(*reinterpret_cast<const float4*>(rows + (long long)r * len + i));
+                }
+                if (shared != nullptr) add(*reinterpret_cast<const float4*>(shared + t * len + i));
+                *reinterpret_cast<float4*>(out + t * len + i) = acc;
+            }
+            return;
+        }
+    }
     for (int i = threadIdx.x; i < len; i += blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {

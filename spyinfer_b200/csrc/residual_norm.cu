@@ -166,32 +166,68 @@ extern "C" int spy_residual_norm(float* h, const void* y, int y_dtype, int split
 
 // out = a_scale * rms_norm(a) * a_weight + b_scale * rms_norm(b) * b_weight, row by row: two sublayer outputs side by side, each normed over
 // the whole row (each possibly a stack of split-K partial sums).  One block a row; both rows stay in shared memory between the passes.
-template <typename TA, typename TB>
+template <typename T, int V> __device__ __forceinline__ void load_run(const T* p, float (&v)[V])
+{
+    if constexpr (V == 1) {
+        v[0] = to_f32(p[0]);
+    } else if constexpr (sizeof(T) == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+    } else {
+        const uint2 x = *reinterpret_cast<const uint2*>(p);
+        const __nv_bfloat162 c = *reinterpret_cast<const __nv_bfloat162*>(&x.x), d = *reinterpret_cast<const __nv_bfloat162*>(&x.y);
+        v[0] = __low2float(c); v[1] = __high2float(c); v[2] = __low2float(d); v[3] = __high2float(d);
+    }
+}
+
+// V = 4: runs of four where rows, parts and tensors allow them
+template <typename TA, typename TB, int V>
 __global__ void normed_sum_kernel(float* __restrict__ out, const TA* __restrict__ a, int a_splits, long long a_stride, const float* __restrict__ a_weight,
                                   float a_scale, const TB* __restrict__ b, int b_splits, long long b_stride, const float* __restrict__ b_weight, float b_scale,
                                   int len, float eps)
 {
-    extern __shared__ float rows_s[];
+    extern __shared__ __align__(16) float rows_s[];
     __shared__ float scratch[33];
     pdl_enter();
     const long long at = (long long)blockIdx.x * len;
-    float *ra = rows_s, *rb = rows_s + len;
+    float *ra = rows_s, *rb = rows_s + (len + 3) / 4 * 4;
     float sa = 0.f, sb = 0.f;
-    for (int i = threadIdx.x; i < len; i += blockDim.x) {
-        float va = to_f32(a[at + i]), vb = to_f32(b[at + i]);
+    for (int i = threadIdx.x * V; i < len; i += blockDim.x * V) {
+        float va[V], vb[V], p[V];
+        load_run<TA, V>(a + at + i, va);
+        load_run<TB, V>(b + at + i, vb);
 #pragma unroll 4
-        for (int s = 1; s < a_splits; ++s) va += to_f32(a[s * a_stride + at + i]);
+        for (int s = 1; s < a_splits; ++s) {
+            load_run<TA, V>(a + s * a_stride + at + i, p);
+#pragma unroll
+            for (int e = 0; e < V; ++e) va[e] += p[e];
+        }
 #pragma unroll 4
-        for (int s = 1; s < b_splits; ++s) vb += to_f32(b[s * b_stride + at + i]);
-        ra[i] = va;
-        rb[i] = vb;
-        sa = fmaf(va, va, sa);
-        sb = fmaf(vb, vb, sb);
+        for (int s = 1; s < b_splits; ++s) {
+            load_run<TB, V>(b + s * b_stride + at + i, p);
+#pragma unroll
+            for (int e = 0; e < V; ++e) vb[e] += p[e];
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            ra[i + e] = va[e];
+            rb[i + e] = vb[e];
+            sa = fmaf(va[e], va[e], sa);
+            sb = fmaf(vb[e], vb[e], sb);
+        }
     }
     sa = block_sum(sa, scratch);
     sb = block_sum(sb, scratch);
     const float ia = a_scale / sqrtf(sa / (float)len + eps), ib = b_scale / sqrtf(sb / (float)len + eps);
-    for (int i = threadIdx.x; i < len; i += blockDim.x) out[at + i] = ra[i] * ia * a_weight[i] + rb[i] * ib * b_weight[i];
+    for (int i = threadIdx.x * V; i < len; i += blockDim.x * V) {
+        float wa[V], wb[V], o[V];
+        load_run<float, V>(a_weight + i, wa);
+        load_run<float, V>(b_weight + i, wb);
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[e] = ra[i + e] * ia * wa[e] + rb[i + e] * ib * wb[e];
+        if constexpr (V == 4) *reinterpret_cast<float4*>(out + at + i) = make_float4(o[0], o[1], o[2], o[3]);
+        else out[at + i] = o[0];
+    }
 }
 
 extern "C" int spy_normed_sum(float* out, const void* a, int a_dtype, int a_splits, long long a_stride, const float* a_weight, float a_scale, const void* b,
@@ -200,12 +236,14 @@ extern "C" int spy_normed_sum(float* out, const void* a, int a_dtype, int a_spli
 {
     if (rows <= 0) return 0;
     if (len <= 0 || a_splits < 1 || b_splits < 1) SPY_FAIL("normed_sum: rows of %d elements, %d and %d parts", len, a_splits, b_splits);
-    const size_t smem = 2 * (size_t)len * sizeof(float);
+    const size_t smem = 2 * (((size_t)len + 3) / 4 * 4) * sizeof(float);
     if (smem > 220 * 1024) SPY_FAIL("normed_sum: two rows of %d elements do not fit a block's shared memory", len);
-    const int threads = len >= 2048 ? 512 : len >= 512 ? 256 : 128;
+    auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const bool vec = len % 4 == 0 && a_stride % 4 == 0 && b_stride % 4 == 0 && aligned(out) && aligned(a) && aligned(b) && aligned(a_weight) && aligned(b_weight);
+    const int per = vec ? len / 4 : len, threads = per >= 512 ? 256 : 128;
     SPY_DISPATCH_DTYPE(a_dtype, TA, {
         SPY_DISPATCH_DTYPE(b_dtype, TB, {
-            auto kernel = normed_sum_kernel<TA, TB>;
+            auto kernel = vec ? normed_sum_kernel<TA, TB, 4> : normed_sum_kernel<TA, TB, 1>;
             if (smem > 48 * 1024) SPY_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             spy_launch(kernel, dim3(rows), dim3(threads), smem, stream, out, (const TA*)a, a_splits, a_stride, a_weight, a_scale, (const TB*)b, b_splits,
                        b_stride, b_weight, b_scale, len, eps);

@@ -62,13 +62,14 @@ __global__ void time_conv_kernel(const TI* __restrict__ in, long long ld_in, con
         for (int i = 0; i < MAXT - 1; ++i)
             if (i < hist_n) hist[i] = to_f32(in[(long long)(t0 - hist_n + i) * ld_in + c]);
     }
-    // four tokens' inputs are requested together, then used in order
-    for (int tb = t0; tb < t1; tb += 4) {
-        float xs[4];
+    // eight tokens' inputs are requested together, then used in order
+    constexpr int AHEAD = MAXT <= 4 ? 8 : 4;
+    for (int tb = t0; tb < t1; tb += AHEAD) {
+        float xs[AHEAD];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) xs[u] = tb + u < t1 ? to_f32(in[(long long)(tb + u) * ld_in + c]) : 0.f;
+        for (int u = 0; u < AHEAD; ++u) xs[u] = tb + u < t1 ? to_f32(in[(long long)(tb + u) * ld_in + c]) : 0.f;
 #pragma unroll
-        for (int u = 0; u < 4; ++u) {
+        for (int u = 0; u < AHEAD; ++u) {
             const int t = tb + u;
             if (t >= t1) break;
             const float x = xs[u];
