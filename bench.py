@@ -860,8 +860,8 @@ def zonevik_workload(args) -> int:
                     rate(block, "qkv_store.spy_gate_heads", nbytes=float(rows) * n_att * H * hd * 6)
                     rate(block, "sink_attention.spy_sink_merge", nbytes=float(rows) * n_par * H * hd * 6)
                     rate(block, "residual_norm.spy_normed_sum", nbytes=float(rows) * n_par * W * 12)
-                    rate(block, "recurrence.spy_gate_group_norm", nbytes=float(rows) * n_par * inner * (4 + 4 + 2))
-                    rate(block, "recurrence.spy_gated_head_norm", nbytes=float(rows) * n_delta * d_v * (4 + 4 + 2))
+                    rate(block, "gated_norm.spy_gate_group_norm", nbytes=float(rows) * n_par * inner * (4 + 4 + 2))
+                    rate(block, "gated_norm.spy_gated_head_norm", nbytes=float(rows) * n_delta * d_v * (4 + 4 + 2))
                     cols = z["experts"] * z["expert_ff"]
                     if "moe.spy_moe_combine" in res[block]:               # the routed form: two products of a token's chosen experts only
                         pairs = float(layers) * rows * z["top"]
@@ -889,7 +889,7 @@ def zonevik_workload(args) -> int:
                 rate("kernels_prefill", "recurrence.spy_delta_scan", nbytes=float(n_delta) * T * d_n * 6 * 4)
                 for block, rows in (("kernels_prefill", T), ("kernels_decode_b64", 64)):
                     rate(block, "layernorm.spy_layernorm", nbytes=float(2 * layers) * rows * W * (4 + 4 + 4 + 2))
-                    rate(block, "recurrence.spy_gated_head_norm", nbytes=float(rows) * (n_par * kv * 2 * hd + n_delta * d_n) * (4 + 4 + 2))
+                    rate(block, "gated_norm.spy_gated_head_norm", nbytes=float(rows) * (n_par * kv * 2 * hd + n_delta * d_n) * (4 + 4 + 2))
 
         return _measure_design(args, cfg_json, vocab, page, T, ctx, annotate)
 

@@ -6,7 +6,7 @@
 //                                            both terms reading the old S, w a decay and r a removal rate per key channel;
 //   * gated linear attention:                S = diag(a) S + k v^T,  o = S^T q,  a = sigmoid(z)^(1/tau) = exp(logsigmoid(z) / tau)
 //                                            a decay per key channel from the pre-activation z;
-// and what follows them: each head's output divided by its root mean square, times a weight, times a gate (sigmoid or SiLU).
+// (what follows them is in gated_norm.cu)
 //
 // A block owns a tile of value columns of one (request, head) (32, 16 or 8 of them: whatever gives the SMs a block each) and
 // walks the request's tokens of this step in order, with its part of S in registers.  The columns of S do not depend on one
@@ -645,104 +645,6 @@ extern "C" int spy_gla_scan(const float* proj, long long ld, int off_q, int off_
     ScanArgs A = {proj, ld, off_q, off_k, off_v, 0, 0, decay_pre, nullptr, decay_bias, state, (long long)dk * dv, num_slots, q_start, state_slot, out,
                   H, dk, dv, q_scale, inv_tau, status};
     return launch_scan(2, A, num_seqs, longest, stream);
-}
-
-// ---- what follows a recurrence: unit root mean square per head, a weight, a gate (sigmoid, or SiLU) -------------
-// One warp a (token, head) row, eight rows a block: the row's sum of squares is a sum inside the warp.
-template <typename TO>
-__global__ void gated_head_norm_kernel(const float* __restrict__ o, const float* __restrict__ proj, long long ld, int off_g, const float* __restrict__ weight,
-                                       TO* __restrict__ out, long long rows, int H, int dv, float eps, int gate_act)
-{
-    pdl_enter();
-    const long long row = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (row >= rows) return;
-    const int lane = threadIdx.x & 31;
-    const long long t = row / H;
-    const int h = (int)(row - t * H);
-    const float* src = o + row * dv;
-    float ss = 0.f;
-    for (int c = lane; c < dv; c += 32) ss += src[c] * src[c];
-    ss = warp_sum(ss);
-    const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
-    const float* g = proj + t * ld + off_g + h * dv;
-    for (int c = lane; c < dv; c += 32) {
-        const float gate = gate_act == 1 ? g[c] * sigmoidf_(g[c]) : sigmoidf_(g[c]);
-        out[row * dv + c] = from_f32<TO>(((src[c] * inv) * weight[h * dv + c]) * gate);
-    }
-}
-
-extern "C" int spy_gated_head_norm(const float* o, const float* proj, long long ld, int off_g, const float* weight, void* out, int out_dtype, int tokens,
-                                   int H, int dv, float eps, cudaStream_t stream, int gate_act)
-{
-    if (gate_act != 0 && gate_act != 1) SPY_FAIL("gated_head_norm: gate activation %d (0: sigmoid, 1: SiLU)", gate_act);
-    if (tokens <= 0) return 0;
-    if (H <= 0 || dv <= 0) SPY_FAIL("gated_head_norm: %d heads of %d", H, dv);
-    const long long rows = (long long)tokens * H, blocks = (rows + 7) / 8;
-    if (blocks > 0x7fffffffLL) SPY_FAIL("gated_head_norm: %lld rows exceed the grid limit", rows);
-    SPY_DISPATCH_DTYPE(out_dtype, TO, {
-        spy_launch(gated_head_norm_kernel<TO>, dim3((unsigned)blocks), dim3(256), 0, stream, o, proj, ld, off_g, weight, (TO*)out, rows, H, dv, eps, gate_act);
-    })
-    SPY_CHECK_LAUNCH("gated_head_norm");
-    return 0;
-}
-
-// The gate ahead of the norm: y = o * silu(gate), cut into `groups` equal parts a row, each divided by its own root mean square, times a
-// weight.  One block a (token, part); the products stay in shared memory between the two passes.
-template <typename TO, int V>
-__global__ void __launch_bounds__(256)
-gate_group_norm_kernel(const float* __restrict__ o, const float* __restrict__ proj, long long ld, int off_g, const float* __restrict__ weight,
-                       TO* __restrict__ out, int size, int groups, float eps)
-{
-    extern __shared__ __align__(16) float y_s[];
-    __shared__ float scratch[33];
-    pdl_enter();
-    const long long t = blockIdx.x;
-    const int part = size / groups, c0 = blockIdx.y * part;
-    const float* src = o + t * size + c0;
-    const float* g = proj + t * ld + off_g + c0;
-    float ss = 0.f;
-    for (int c = threadIdx.x * V; c < part; c += blockDim.x * V) {
-        float a[V], b[V];
-        if (V == 4) {
-            *reinterpret_cast<float4*>(a) = *reinterpret_cast<const float4*>(src + c);
-            *reinterpret_cast<float4*>(b) = *reinterpret_cast<const float4*>(g + c);
-        } else {
-            a[0] = src[c];
-            b[0] = g[c];
-        }
-#pragma unroll
-        for (int e = 0; e < V; ++e) {
-            const float y = a[e] * (b[e] * sigmoidf_(b[e]));
-            y_s[c + e] = y;
-            ss = fmaf(y, y, ss);
-        }
-    }
-    ss = block_sum(ss, scratch);
-    const float inv = 1.0f / sqrtf(ss / (float)part + eps);
-    for (int c = threadIdx.x * V; c < part; c += blockDim.x * V) {
-#pragma unroll
-        for (int e = 0; e < V; ++e) out[t * size + c0 + c + e] = from_f32<TO>(y_s[c + e] * inv * weight[c0 + c + e]);
-    }
-}
-
-extern "C" int spy_gate_group_norm(const float* o, const float* proj, long long ld, int off_g, const float* weight, void* out, int out_dtype, int tokens,
-                                   int size, int groups, float eps, cudaStream_t stream)
-{
-    if (tokens <= 0) return 0;
-    if (size <= 0 || groups <= 0 || size % groups != 0 || groups > 65535) SPY_FAIL("gate_group_norm: rows of %d in %d parts", size, groups);
-    const int part = size / groups;
-    const size_t smem = (size_t)part * sizeof(float);
-    if (smem > 200 * 1024) SPY_FAIL("gate_group_norm: a part of %d elements does not fit a block's shared memory", part);
-    const bool vec = part % 4 == 0 && ld % 4 == 0 && off_g % 4 == 0 && ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(proj)) & 15) == 0;
-    const int per = part / (vec ? 4 : 1);
-    const int threads = per >= 256 ? 256 : per >= 128 ? 128 : per >= 64 ? 64 : 32;
-    SPY_DISPATCH_DTYPE(out_dtype, TO, {
-        auto kernel = vec ? gate_group_norm_kernel<TO, 4> : gate_group_norm_kernel<TO, 1>;
-        if (smem > 48 * 1024) SPY_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        spy_launch(kernel, dim3(tokens, groups), dim3(threads), smem, stream, o, proj, ld, off_g, weight, (TO*)out, size, groups, eps);
-    })
-    SPY_CHECK_LAUNCH("gate_group_norm");
-    return 0;
 }
 
 // out[t, j] = act(proj[t, off + j]) for j < n: the inner activation of a two-step (low-rank) projection; act 0: tanh, 1: none.

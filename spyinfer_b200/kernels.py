@@ -603,7 +603,7 @@ def gate_group_norm(o: torch.Tensor, proj: torch.Tensor, gate_offset: int, weigh
     n = o.shape[1]
     if tuple(out.shape) != tuple(o.shape) or weight.shape[0] != n or gate_offset + n > proj.shape[1] or proj.shape[0] != o.shape[0] or groups <= 0 or n % groups:
         raise KernelError("gate_group_norm: shapes do not fit")
-    _call("recurrence", "spy_gate_group_norm", _ptr(o), _ptr(proj), ctypes.c_longlong(proj.shape[1]), int(gate_offset), _ptr(weight), _ptr(out),
+    _call("gated_norm", "spy_gate_group_norm", _ptr(o), _ptr(proj), ctypes.c_longlong(proj.shape[1]), int(gate_offset), _ptr(weight), _ptr(out),
           _code(out, "gated output"), o.shape[0], n, int(groups), ctypes.c_float(eps), _stream())
     return out
 
@@ -621,7 +621,7 @@ def gated_head_norm(o: torch.Tensor, proj: torch.Tensor, gate_offset: int, weigh
     n = heads * dv
     if o.shape[1] != n or tuple(out.shape) != tuple(o.shape) or weight.shape[0] != n or gate_offset + n > proj.shape[1] or proj.shape[0] != o.shape[0]:
         raise KernelError("gated_head_norm: shapes do not fit")
-    _call("recurrence", "spy_gated_head_norm", _ptr(o), _ptr(proj), ctypes.c_longlong(proj.shape[1]), int(gate_offset), _ptr(weight), _ptr(out),
+    _call("gated_norm", "spy_gated_head_norm", _ptr(o), _ptr(proj), ctypes.c_longlong(proj.shape[1]), int(gate_offset), _ptr(weight), _ptr(out),
           _code(out, "gated output"), o.shape[0], heads, dv, ctypes.c_float(eps), _stream(), ("sigmoid", "silu").index(gate))
     return out
 

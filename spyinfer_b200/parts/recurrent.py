@@ -95,7 +95,7 @@ class MatrixMemory(_Recurrent):
         self.bias_f = tensors[self.prefix + "f.b"].float().contiguous()
 
     def modules(self):
-        return ["recurrence"] + self.fused.modules() + self.o.modules()
+        return ["recurrence", "gated_norm"] + self.fused.modules() + self.o.modules()
 
     def linears(self):
         return [self.fused, self.o]
@@ -143,7 +143,7 @@ class DeltaRule(_Recurrent):
         self.decay_offset = tensors[self.prefix + "w0"].float().contiguous()
 
     def modules(self):
-        return ["recurrence"] + self.fused.modules() + self.w2.modules() + self.o.modules()
+        return ["recurrence", "gated_norm"] + self.fused.modules() + self.w2.modules() + self.o.modules()
 
     def linears(self):
         return [self.fused, self.w2, self.o]
@@ -197,7 +197,7 @@ class GatedLinearAttention(_Recurrent):
         self.decay_bias = tensors[self.prefix + "a2.b"].float().contiguous()
 
     def modules(self):
-        return ["recurrence"] + self.fused.modules() + self.a2.modules() + self.o.modules()
+        return ["recurrence", "gated_norm"] + self.fused.modules() + self.a2.modules() + self.o.modules()
 
     def linears(self):
         return [self.fused, self.a2, self.o]
@@ -233,7 +233,7 @@ class _ConvRecurrent(_Recurrent):
         return [self.fused, self.o]
 
     def modules(self):
-        return ["head_scan", "recurrence"] + self.conv.modules() + self.fused.modules() + self.o.modules()
+        return ["head_scan", "gated_norm"] + self.conv.modules() + self.fused.modules() + self.o.modules()
 
 
 @register_part("gated_delta_rule")
