@@ -48,10 +48,11 @@ struct Tanh {
     const void* b;
 };
 
-template <typename TY, typename TW, typename TO, int V>
+// ROWS rows a block (1; 4 when there are many): a thread's weights are loaded once for all of them, and their inputs are under way together.
+template <typename TY, typename TW, typename TO, int V, int ROWS>
 __global__ void __launch_bounds__(THREADS)
 dynamic_tanh_kernel(float* __restrict__ hidden, const TY* __restrict__ y, int splits, long long split_stride, Tanh ty, float y_scale,
-                    const int* __restrict__ rows, Tanh tx, TO* __restrict__ out, int len, int write_back)
+                    const int* __restrict__ rows, Tanh tx, TO* __restrict__ out, int n, int len, int write_back)
 {
     pdl_launch_dependents();
     const int i = (blockIdx.y * THREADS + threadIdx.x) * V;
@@ -71,27 +72,36 @@ dynamic_tanh_kernel(float* __restrict__ hidden, const TY* __restrict__ y, int sp
     }
     pdl_wait();
     if (i >= len) return;
-    const int r = blockIdx.x;
-    const long long at = (long long)(rows != nullptr ? rows[r] : r) * len + i;
-    float h[V];
-    Run<float, V>::load(hidden + at, h);
-    if (y != nullptr) {
-        float v[V], p[V];
-        Run<TY, V>::load(y + at, v);
-#pragma unroll 4
-        for (int s = 1; s < splits; ++s) {
-            Run<TY, V>::load(y + s * split_stride + at, p);
+    const int r0 = blockIdx.x * ROWS, live = min(ROWS, n - r0);
+    long long at[ROWS];
+    float h[ROWS][V], v[ROWS][V];
 #pragma unroll
-            for (int e = 0; e < V; ++e) v[e] += p[e];
-        }
-#pragma unroll
-        for (int e = 0; e < V; ++e) h[e] += y_scale * fmaf(tanhf(ay * v[e]), wy[e], by[e]);
-        if (write_back) Run<float, V>::store(hidden + at, h);
+    for (int j = 0; j < ROWS; ++j) {
+        if (j >= live) break;
+        at[j] = (long long)(rows != nullptr ? rows[r0 + j] : r0 + j) * len + i;
+        Run<float, V>::load(hidden + at[j], h[j]);
+        if (y != nullptr) Run<TY, V>::load(y + at[j], v[j]);
     }
-    if (out == nullptr) return;
 #pragma unroll
-    for (int e = 0; e < V; ++e) h[e] = fmaf(tanhf(ax * h[e]), wx[e], bx[e]);
-    Run<TO, V>::store(out + (long long)r * len + i, h);
+    for (int j = 0; j < ROWS; ++j) {
+        if (j >= live) break;
+        if (y != nullptr) {
+            float p[V];
+#pragma unroll 4
+            for (int s = 1; s < splits; ++s) {
+                Run<TY, V>::load(y + s * split_stride + at[j], p);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[j][e] += p[e];
+            }
+#pragma unroll
+            for (int e = 0; e < V; ++e) h[j][e] += y_scale * fmaf(tanhf(ay * v[j][e]), wy[e], by[e]);
+            if (write_back) Run<float, V>::store(hidden + at[j], h[j]);
+        }
+        if (out == nullptr) continue;
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[j][e] = fmaf(tanhf(ax * h[j][e]), wx[e], bx[e]);
+        Run<TO, V>::store(out + (long long)(r0 + j) * len + i, h[j]);
+    }
 }
 
 // hidden [*, len] float32.  y (optional): [splits][rows][len] of y_dtype with its alpha, weight, bias and scale.  alpha/weight/
@@ -118,12 +128,11 @@ extern "C" int spy_dynamic_tanh(float* hidden, const void* y, int y_dtype, int s
     SPY_DISPATCH_DTYPE(y_dtype, TY, {
         SPY_DISPATCH_DTYPE(weight_dtype, TW, {
             SPY_DISPATCH_DTYPE(out_dtype, TO, {
-                if (vec)
-                    spy_launch(dynamic_tanh_kernel<TY, TW, TO, 4>, dim3(n, pieces), dim3(THREADS), 0, stream, hidden, (const TY*)y, splits, split_stride, ty,
-                               y_scale, rows, tx, (TO*)out, len, write_back);
-                else
-                    spy_launch(dynamic_tanh_kernel<TY, TW, TO, 1>, dim3(n, pieces), dim3(THREADS), 0, stream, hidden, (const TY*)y, splits, split_stride, ty,
-                               y_scale, rows, tx, (TO*)out, len, write_back);
+                const bool many = n >= 512;
+                auto kernel = vec ? (many ? dynamic_tanh_kernel<TY, TW, TO, 4, 4> : dynamic_tanh_kernel<TY, TW, TO, 4, 1>)
+                                  : (many ? dynamic_tanh_kernel<TY, TW, TO, 1, 4> : dynamic_tanh_kernel<TY, TW, TO, 1, 1>);
+                spy_launch(kernel, dim3(many ? (n + 3) / 4 : n, pieces), dim3(THREADS), 0, stream, hidden, (const TY*)y, splits, split_stride, ty, y_scale, rows,
+                           tx, (TO*)out, n, len, write_back);
             })
         })
     })

@@ -84,7 +84,7 @@ extern "C" int spy_gated_head_norm(const float* o, const float* proj, long long 
     if (blocks > 0x7fffffffLL) SPY_FAIL("gated_head_norm: %lld rows exceed the grid limit", rows);
     SPY_DISPATCH_DTYPE(out_dtype, TO, {
         auto kernel = vec ? gated_head_norm_kernel<TO, true> : gated_head_norm_kernel<TO, false>;
-                spy_launch(kernel, dim3((unsigned)blocks), dim3(256), 0, stream, o, proj, ld, off_g, weight, (TO*)out, rows, H, dv, eps, gate_act);
+        spy_launch(kernel, dim3((unsigned)blocks), dim3(256), 0, stream, o, proj, ld, off_g, weight, (TO*)out, rows, H, dv, eps, gate_act);
     })
     SPY_CHECK_LAUNCH("gated_head_norm");
     return 0;

@@ -310,7 +310,7 @@ def test_dynamic_tanh_adds_a_result_and_norms_the_stream(dtype):
     from spyinfer_b200 import kernels
 
     g = torch.Generator().manual_seed(4)
-    for rows, n, splits in ((5, 40, 1), (3, 200, 3), (9, 1000, 2), (4, 4096, 7), (600, 256, 2), (2, 50, 1), (7, 6145, 1), (1, 3, 4)):
+    for rows, n, splits in ((5, 40, 1), (3, 200, 3), (9, 1000, 2), (4, 4096, 7), (601, 256, 2), (2, 50, 1), (7, 6145, 1), (1, 3, 4), (514, 37, 1)):
         h, y = torch.randn(rows, n, generator=g) * 2, torch.randn(splits, rows, n, generator=g)
         ty, tx = ((torch.rand(1, generator=g) + 0.3, (1.0 + 0.3 * torch.randn(n, generator=g)).to(torch.bfloat16), (0.3 * torch.randn(n, generator=g)).to(torch.bfloat16))
                   for _ in range(2))
@@ -324,6 +324,12 @@ def test_dynamic_tanh_adds_a_result_and_norms_the_stream(dtype):
         tol = dict(atol=2e-6, rtol=2e-6) if dtype == torch.float32 else dict(atol=2e-2, rtol=1e-2)
         assert torch.allclose(hd.cpu().double(), want_h, atol=5e-6, rtol=1e-6), (rows, n)
         assert torch.allclose(out.cpu().double(), want_x, **tol)
+        # the stream's own sum is 32-bit in both formats, from tiny to saturated arguments
+        ramp = torch.cat([torch.logspace(-6, 1.3, n // 2), -torch.logspace(-6, 1.3, n - n // 2)])[None].repeat(rows, 1)
+        acc = torch.zeros(rows, n, device="cuda")
+        one = (torch.ones(1), torch.ones(n).to(torch.bfloat16), torch.zeros(n).to(torch.bfloat16))
+        kernels.dynamic_tanh(acc, y=ramp.cuda(), y_norm=dev(one), norm=dev(tx), out=torch.empty((rows, n), dtype=dtype, device="cuda"))
+        assert torch.allclose(acc.cpu().double(), torch.tanh(ramp.double()), rtol=1e-6, atol=1e-12)
         before = hd.clone()
         pick = torch.tensor([rows - 1, 0], dtype=torch.int32, device="cuda")           # gathered rows: the pending result counts, the stream stays
         few = torch.empty((2, n), dtype=torch.float32, device="cuda")
