@@ -327,6 +327,8 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
             const float* vg = v_s + g * U * CTB;
             float w[U];                            // the column's own values: what each token writes
             float x[DELTA ? NC * U : 1], y[NC * U];     // [column][token]
+            constexpr bool HOLD = DELTA && NR == 8;     // the keys stay in registers between the reading and the writing
+            float k_r[HOLD ? U * NR : 1];
 #pragma unroll
             for (int j = 0; j < NC * U; ++j) {
                 if (DELTA) x[j] = 0.f;
@@ -339,6 +341,10 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
                     float kk[4], qq[4];
                     if (DELTA) *reinterpret_cast<float4*>(kk) = *reinterpret_cast<const float4*>(kg + u * KS + qd * 4 * RG);
                     *reinterpret_cast<float4*>(qq) = *reinterpret_cast<const float4*>(qg + u * KS + qd * 4 * RG);
+                    if constexpr (HOLD) {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) k_r[u * NR + qd * 4 + e] = kk[e];
+                    }
 #pragma unroll
                     for (int e = 0; e < 4; ++e)
 #pragma unroll
@@ -348,21 +354,13 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
                         }
                 }
             if constexpr (DELTA) halve<NC * U / 2>(x, CG, b0);
-            halve<NC * U / 2>(y, CG, b0);
-            if constexpr (NC == 4) {
-                if constexpr (DELTA) halve<U>(x, 2 * CG, b1);
-                halve<U>(y, 2 * CG, b1);
-            }
+            if constexpr (DELTA && NC == 4) halve<U>(x, 2 * CG, b1);
             if constexpr (DELTA) {
 #pragma unroll
                 for (int o = NC * CG; o <= 16; o <<= 1)
 #pragma unroll
                     for (int u = 0; u < U; ++u) x[u] += __shfl_xor_sync(0xffffffffu, x[u], o);
             }
-            if (NREP >= 2) halve<4>(y, NC * CG, rep & 1);
-            if (NREP >= 4) halve<2>(y, 2 * NC * CG, rep & 2);
-            if (NREP >= 8) halve<1>(y, 4 * NC * CG, rep & 4);
-            if (NREP >= 16) y[0] += __shfl_xor_sync(0xffffffffu, y[0], 16);
             if constexpr (DELTA) {
 #pragma unroll
                 for (int t = 0; t < U; ++t) {
@@ -390,18 +388,6 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
 #pragma unroll
                 for (int t = 0; t < U; ++t) w[t] = vg[t * CTB + own_col];       // the step is in the table
             }
-#pragma unroll
-            for (int j = 0; j < N_OWN; ++j) {
-                const int t = t_own + j;
-                float p[U];
-                *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(tab + 64 + t * 8);
-                *reinterpret_cast<float4*>(p + 4) = *reinterpret_cast<const float4*>(tab + 64 + t * 8 + 4);
-                float o = tab[144 + t] * y[j];
-#pragma unroll
-                for (int s = 0; s < U; ++s) o = fmaf(p[s], w[s], o);
-                if (!DELTA) o = fmaf(d_skip, vg[t * CTB + own_col], o);
-                if (stores && g * U + t < n_tok) A.out[(size_t)(t0 + g * U + t) * A.H * dv + h * dv + c0 + own_col] = o;
-            }
             const float g_all = tab[160];
 #pragma unroll
             for (int j = 0; j < NR; ++j)
@@ -420,12 +406,36 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
 #pragma unroll
                 for (int qd = 0; qd < NQ; ++qd) {
                     float kk[4];
-                    *reinterpret_cast<float4*>(kk) = *reinterpret_cast<const float4*>(kg + u * KS + qd * 4 * RG);
+                    if constexpr (HOLD) {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) kk[e] = k_r[u * NR + qd * 4 + e];
+                    } else {
+                        *reinterpret_cast<float4*>(kk) = *reinterpret_cast<const float4*>(kg + u * KS + qd * 4 * RG);
+                    }
 #pragma unroll
                     for (int e = 0; e < 4; ++e)
 #pragma unroll
                         for (int c = 0; c < NC; ++c) S[qd * 4 + e][c] = fmaf(kk[e], ww[c], S[qd * 4 + e][c]);
                 }
+            }
+            // the read-outs, which nothing of the state waits for
+            halve<NC * U / 2>(y, CG, b0);
+            if constexpr (NC == 4) halve<U>(y, 2 * CG, b1);
+            if (NREP >= 2) halve<4>(y, NC * CG, rep & 1);
+            if (NREP >= 4) halve<2>(y, 2 * NC * CG, rep & 2);
+            if (NREP >= 8) halve<1>(y, 4 * NC * CG, rep & 4);
+            if (NREP >= 16) y[0] += __shfl_xor_sync(0xffffffffu, y[0], 16);
+#pragma unroll
+            for (int j = 0; j < N_OWN; ++j) {
+                const int t = t_own + j;
+                float p[U];
+                *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(tab + 64 + t * 8);
+                *reinterpret_cast<float4*>(p + 4) = *reinterpret_cast<const float4*>(tab + 64 + t * 8 + 4);
+                float o = tab[144 + t] * y[j];
+#pragma unroll
+                for (int s = 0; s < U; ++s) o = fmaf(p[s], w[s], o);
+                if (!DELTA) o = fmaf(d_skip, vg[t * CTB + own_col], o);
+                if (stores && g * U + t < n_tok) A.out[(size_t)(t0 + g * U + t) * A.H * dv + h * dv + c0 + own_col] = o;
             }
         }
     }

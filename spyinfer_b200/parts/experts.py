@@ -85,7 +85,7 @@ class ExpertMixture(FeedForward):
 
     def _grouped_from(self) -> int:
         spare = 2 * self.experts - 3 * self.top                    # half the dense form's rows must be enough and some over
-        return max(512, -(-3 * 128 * self.experts // spare)) if spare > 0 else 0
+        return max(1024, -(-3 * 128 * self.experts // spare)) if spare > 0 else 0     # fewer tokens: the form's further launches cost what it saves
 
     def weight_decls(self):
         p, W = self.prefix, self.hidden
