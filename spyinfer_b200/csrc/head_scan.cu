@@ -15,7 +15,7 @@
 //     S  <- g_7 S0 + sum_s D(7,s) k_s w_s^T
 // which is the token-by-token walk with its sums in another order.  Only products of decays occur, no quotients.  A column's own chain
 // of eight is walked by the lanes that hold it.  So a token costs three multiply-adds an element of the state (two without the delta
-// rule), the lanes' sums over the rows run for eight tokens together, and nothing waits for one token.
+// rule; packed two to an instruction), the lanes' sums over the rows run for eight tokens together, and nothing waits for one token.
 // The coefficients (dot products among the eight tokens' keys and queries, their decays) are the same for every column of a head:
 // a kernel ahead (head_table_kernel) makes them once, a warp for every eight tokens of a key head.
 //
@@ -30,6 +30,8 @@ SPY_MODULE(spy_head_scan)
 constexpr int U = 8;              // tokens taken together
 constexpr int WARPS = 4;          // of a block of the kernel for portions
 constexpr int THREADS = 32 * WARPS;
+// groups of eight in shared memory (keys of KS elements): one that is walked, the others on their way
+__host__ __device__ constexpr int ring_of(int KS) { return KS > 512 ? 2 : 4; }
 constexpr int TABLE = 64 + 64 + 5 * U;   // floats of a group's coefficients: among the tokens (removal, read-out), then per token
 
 struct HeadScanArgs {
@@ -64,7 +66,30 @@ __device__ __forceinline__ void cp_async4(float* smem_dst, const float* src)
 {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(src) : "memory");
 }
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// two 32-bit floats side by side: one instruction for both
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 pair2(float a, float b)
+{
+    f2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ void split2(f2 v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c)
+{
+    f2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b)
+{
+    f2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
 
 // v[0 .. 2M) of every lane -> v[0 .. M): lanes whose `bit` of `off` is 0 keep the first half, the others the second, each summed with
 // the partner's half
@@ -214,16 +239,15 @@ __global__ void __launch_bounds__(32 * TABLE_WARPS) head_table_kernel(HeadScanAr
 // A thread's rows: quads qd * 4 RG + 4 rg .. + 3 (qd < NR / 4) of RG * NR >= dk; its columns: NC neighbours.  RG row groups share a
 // warp's lanes (rg = lane / CG), so a warp owns (32 / RG) * NC columns and a block four times that.
 template <bool DELTA, int RG, int NR, int NC>
-__global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, int TC)
+__global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A)
 {
     constexpr int NQ = NR / 4, KS = RG * NR, CG = 32 / RG, WC = CG * NC, CTB = WARPS * WC, NREP = RG / NC;
     static_assert(RG >= NC && NC >= 2, "the columns of a thread are dealt out over its row groups");
     extern __shared__ __align__(16) float sm[];
     // in plain stream order (spy_launch_in_order): it runs long on about a block an SM
     pdl_wait();
-    const int groups = TC / U;
-    const size_t stage_floats = 2 * (size_t)TC * KS + (size_t)TC * CTB + (size_t)groups * TABLE;
-    float* w_s = sm + 2 * stage_floats;                          // [WARPS][U][WC]
+    constexpr int RING = ring_of(KS), STAGE = U * (2 * KS + CTB) + TABLE;            // floats of a group: keys, queries, values, coefficients
+    float* w_s = sm + RING * STAGE;                          // [WARPS][U][WC]
 
     const int seq = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * CTB, hk = h / A.share;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -238,67 +262,73 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
     const float* my_tables = A.tables + ((size_t)first_group(t_begin, seq) * A.H + h) * TABLE;
     const bool aligned = (dk & 3) == 0 && (A.ld & 3) == 0 && ((A.off_k | A.off_q) & 3) == 0 && (reinterpret_cast<uintptr_t>(A.proj) & 15) == 0;
     const bool v_aligned = (dv & 3) == 0 && (A.ld & 3) == 0 && (A.off_v & 3) == 0 && (reinterpret_cast<uintptr_t>(A.proj) & 15) == 0;
-    // brings a stage's rows (a warp a token) and coefficients into shared memory; zeros behind a row's end and the run's
-    auto request = [&](int t0, int stage) {
-        const int n_tok = min(TC, t_end - t0), n_pad = (n_tok + U - 1) / U * U;
-        float* k_s = sm + stage * stage_floats;
-        float* q_s = k_s + (size_t)TC * KS;
-        float* v_s = q_s + (size_t)TC * KS;
-        float* tab = v_s + TC * CTB;
-        for (int tt = warp; tt < n_pad; tt += WARPS) {
-            const float* row = A.proj + (size_t)(t0 + tt) * A.ld;
-            const bool in = tt < n_tok;
-            const float *ks = row + A.off_k + hk * dk, *qs = row + A.off_q + hk * dk, *vs = row + A.off_v + h * dv + c0;
-            if (aligned) {
+    const int n_groups = (t_end - t_begin + U - 1) / U;
+    // Requests a group's rows (a warp a token) and coefficients: a few copies a warp and group, so that the walk's own traffic with shared
+    // memory never waits behind many of them.  Zeros behind a row's end and the run's.
+    auto request = [&](int g) {
+        if (g < n_groups) {
+            const int t0 = t_begin + g * U, n_tok = min(U, t_end - t0);
+            float* k_s = sm + (g % RING) * STAGE;
+            float* q_s = k_s + U * KS;
+            float* v_s = q_s + U * KS;
 #pragma unroll
-                for (int e = 4 * lane; e < KS; e += 128) {
-                    if (in && e < dk) {
-                        cp_async16(k_s + tt * KS + e, ks + e);
-                        cp_async16(q_s + tt * KS + e, qs + e);
-                    } else {
-                        *reinterpret_cast<float4*>(k_s + tt * KS + e) = make_float4(0.f, 0.f, 0.f, 0.f);
-                        *reinterpret_cast<float4*>(q_s + tt * KS + e) = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int tt = warp; tt < U; tt += WARPS) {
+                const float* row = A.proj + (size_t)(t0 + tt) * A.ld;
+                const bool in = tt < n_tok;
+                const float *ks = row + A.off_k + hk * dk, *qs = row + A.off_q + hk * dk, *vs = row + A.off_v + h * dv + c0;
+                if (aligned) {
+#pragma unroll
+                    for (int e = 4 * lane; e < KS; e += 128) {
+                        if (in && e < dk) {
+                            cp_async16(k_s + tt * KS + e, ks + e);
+                            cp_async16(q_s + tt * KS + e, qs + e);
+                        } else {
+                            *reinterpret_cast<float4*>(k_s + tt * KS + e) = make_float4(0.f, 0.f, 0.f, 0.f);
+                            *reinterpret_cast<float4*>(q_s + tt * KS + e) = make_float4(0.f, 0.f, 0.f, 0.f);
+                        }
+                    }
+                } else {
+                    for (int e = lane; e < KS; e += 32) {
+                        if (in && e < dk) {
+                            cp_async4(k_s + tt * KS + e, ks + e);
+                            cp_async4(q_s + tt * KS + e, qs + e);
+                        } else {
+                            k_s[tt * KS + e] = q_s[tt * KS + e] = 0.f;
+                        }
                     }
                 }
-            } else {
-                for (int e = lane; e < KS; e += 32) {
-                    if (in && e < dk) {
-                        cp_async4(k_s + tt * KS + e, ks + e);
-                        cp_async4(q_s + tt * KS + e, qs + e);
-                    } else {
-                        k_s[tt * KS + e] = q_s[tt * KS + e] = 0.f;
+                if (v_aligned) {
+                    for (int c = 4 * lane; c < CTB; c += 128) {
+                        if (in && c0 + c < dv) cp_async16(v_s + tt * CTB + c, vs + c);
+                        else *reinterpret_cast<float4*>(v_s + tt * CTB + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+                    }
+                } else {
+                    for (int c = lane; c < CTB; c += 32) {
+                        if (in && c0 + c < dv) cp_async4(v_s + tt * CTB + c, vs + c);
+                        else v_s[tt * CTB + c] = 0.f;
                     }
                 }
             }
-            if (v_aligned) {
-                for (int c = 4 * lane; c < CTB; c += 128) {
-                    if (in && c0 + c < dv) cp_async16(v_s + tt * CTB + c, vs + c);
-                    else *reinterpret_cast<float4*>(v_s + tt * CTB + c) = make_float4(0.f, 0.f, 0.f, 0.f);
-                }
-            } else {
-                for (int c = lane; c < CTB; c += 32) {
-                    if (in && c0 + c < dv) cp_async4(v_s + tt * CTB + c, vs + c);
-                    else v_s[tt * CTB + c] = 0.f;
-                }
+            if (warp == (g & (WARPS - 1))) {
+                const float* src = my_tables + (size_t)g * A.H * TABLE;
+                for (int e = 4 * lane + (DELTA ? 0 : 64); e < TABLE; e += 128) cp_async16(v_s + U * CTB + e, src + e);
             }
         }
-        const int g0 = (t0 - t_begin) / U;
-        for (int g = warp; g < n_pad / U; g += WARPS) {
-            const float* src = my_tables + (size_t)(g0 + g) * A.H * TABLE;
-            for (int e = 4 * lane + (DELTA ? 0 : 64); e < TABLE; e += 128) cp_async16(tab + g * TABLE + e, src + e);
-        }
+        cp_async_commit();                         // one group of copies a call, empty behind the last
     };
-    request(t_begin, 0);
+#pragma unroll
+    for (int g = 0; g < RING - 1; ++g) request(g);
     const int rg = lane / CG, cg = lane % CG;
     const int col0 = c0 + warp * WC + cg * NC;                   // the thread's first column
     float* st = A.state + ((size_t)slot * A.H + h) * dk * dv;
-    float S[NR][NC];
+    f2 S[NR / 2][NC];                                            // rows 2 i and 2 i + 1 of the thread's, one column
 #pragma unroll
-    for (int i = 0; i < NR; ++i)
+    for (int i = 0; i < NR / 2; ++i)
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-            const int r = (i / 4) * 4 * RG + 4 * rg + i % 4;
-            S[i][c] = r < dk && col0 + c < dv ? st[(size_t)r * dv + col0 + c] : 0.f;
+            const int r = (i / 2) * 4 * RG + 4 * rg + 2 * (i % 2);
+            const bool in = col0 + c < dv;
+            S[i][c] = pair2(in && r < dk ? st[(size_t)r * dv + col0 + c] : 0.f, in && r + 1 < dk ? st[(size_t)(r + 1) * dv + col0 + c] : 0.f);
         }
     // which column of the thread's row groups this lane sums and walks, and (NREP lanes walk the same column) which copy it is
     const bool b0 = rg & 1, b1 = rg & 2;
@@ -310,49 +340,58 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
     const int t_own = NREP >= 8 ? (rep & 1) * 4 + (rep & 2) + ((rep & 4) >> 2) : NREP >= 4 ? (rep & 1) * 4 + (rep & 2) : NREP >= 2 ? (rep & 1) * 4 : 0;
     constexpr int N_OWN = NREP >= U ? 1 : U / NREP;
     const bool stores = c0 + own_col < dv && (NREP < 16 || rep < 8);
-    int stage = 0;
-    for (int t0 = t_begin; t0 < t_end; t0 += TC, stage ^= 1) {
-        const int n_tok = min(TC, t_end - t0), n_groups = (n_tok + U - 1) / U;
-        const float* k_s = sm + stage * stage_floats;
-        const float* q_s = k_s + (size_t)TC * KS;
-        const float* v_s = q_s + (size_t)TC * KS;
-        const float* tables = v_s + TC * CTB;
-        cp_async_wait_all();
-        __syncthreads();                           // this stage has landed; every warp is past the stage before, whose place is free
-        if (t0 + TC < t_end) request(t0 + TC, stage ^ 1);
-        for (int g = 0; g < n_groups; ++g) {
-            const float* tab = tables + g * TABLE;
-            const float* kg = k_s + g * U * KS + 4 * rg;
-            const float* qg = q_s + g * U * KS + 4 * rg;
-            const float* vg = v_s + g * U * CTB;
+    for (int g = 0; g < n_groups; ++g) {
+        cp_async_wait<RING - 2>();
+        __syncthreads();                           // this group has landed; every warp is past the one before, whose place is free
+        request(g + RING - 1);
+        {
+            const int t0 = t_begin + g * U, n_tok = t_end - t0;
+            const float* kg = sm + (g % RING) * STAGE + 4 * rg;
+            const float* qg = kg + U * KS;
+            const float* vg = sm + (g % RING) * STAGE + 2 * U * KS;
+            const float* tab = vg + U * CTB;
             float w[U];                            // the column's own values: what each token writes
             float x[DELTA ? NC * U : 1], y[NC * U];     // [column][token]
-            constexpr bool HOLD = DELTA && NR == 8;     // the keys stay in registers between the reading and the writing
-            float k_r[HOLD ? U * NR : 1];
+            constexpr int PART = NC == 4 ? 4 : U;      // tokens whose sums are under way together
 #pragma unroll
-            for (int j = 0; j < NC * U; ++j) {
-                if (DELTA) x[j] = 0.f;
-                y[j] = 0.f;
-            }
+            for (int u0 = 0; u0 < U; u0 += PART) {
+                f2 x2[DELTA ? NC * PART : 1], y2[NC * PART];
 #pragma unroll
-            for (int u = 0; u < U; ++u)
+                for (int j = 0; j < NC * PART; ++j) {
+                    if (DELTA) x2[j] = 0ull;
+                    y2[j] = 0ull;
+                }
 #pragma unroll
-                for (int qd = 0; qd < NQ; ++qd) {
-                    float kk[4], qq[4];
-                    if (DELTA) *reinterpret_cast<float4*>(kk) = *reinterpret_cast<const float4*>(kg + u * KS + qd * 4 * RG);
-                    *reinterpret_cast<float4*>(qq) = *reinterpret_cast<const float4*>(qg + u * KS + qd * 4 * RG);
-                    if constexpr (HOLD) {
+                for (int u = 0; u < PART; ++u)
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) k_r[u * NR + qd * 4 + e] = kk[e];
-                    }
-#pragma unroll
-                    for (int e = 0; e < 4; ++e)
+                    for (int qd = 0; qd < NQ; ++qd) {
+                        ulonglong2 kk, qq;
+                        if (DELTA) kk = *reinterpret_cast<const ulonglong2*>(kg + (u0 + u) * KS + qd * 4 * RG);
+                        qq = *reinterpret_cast<const ulonglong2*>(qg + (u0 + u) * KS + qd * 4 * RG);
 #pragma unroll
                         for (int c = 0; c < NC; ++c) {
-                            if (DELTA) x[c * U + u] = fmaf(kk[e], S[qd * 4 + e][c], x[c * U + u]);
-                            y[c * U + u] = fmaf(qq[e], S[qd * 4 + e][c], y[c * U + u]);
+                            if (DELTA) x2[c * PART + u] = fma2(kk.x, S[qd * 2][c], x2[c * PART + u]);
+                            y2[c * PART + u] = fma2(qq.x, S[qd * 2][c], y2[c * PART + u]);
                         }
-                }
+#pragma unroll
+                        for (int c = 0; c < NC; ++c) {
+                            if (DELTA) x2[c * PART + u] = fma2(kk.y, S[qd * 2 + 1][c], x2[c * PART + u]);
+                            y2[c * PART + u] = fma2(qq.y, S[qd * 2 + 1][c], y2[c * PART + u]);
+                        }
+                    }
+#pragma unroll
+                for (int c = 0; c < NC; ++c)
+#pragma unroll
+                    for (int u = 0; u < PART; ++u) {
+                        float p, q;
+                        if constexpr (DELTA) {
+                            split2(x2[c * PART + u], p, q);
+                            x[c * U + u0 + u] = p + q;
+                        }
+                        split2(y2[c * PART + u], p, q);
+                        y[c * U + u0 + u] = p + q;
+                    }
+            }
             if constexpr (DELTA) halve<NC * U / 2>(x, CG, b0);
             if constexpr (DELTA && NC == 4) halve<U>(x, 2 * CG, b1);
             if constexpr (DELTA) {
@@ -388,34 +427,31 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
 #pragma unroll
                 for (int t = 0; t < U; ++t) w[t] = vg[t * CTB + own_col];       // the step is in the table
             }
-            const float g_all = tab[160];
+            const f2 g_all = pair2(tab[160], tab[160]);
 #pragma unroll
-            for (int j = 0; j < NR; ++j)
+            for (int j = 0; j < NR / 2; ++j)
 #pragma unroll
-                for (int c = 0; c < NC; ++c) S[j][c] *= g_all;
+                for (int c = 0; c < NC; ++c) S[j][c] = mul2(S[j][c], g_all);
 #pragma unroll
             for (int u = 0; u < U; ++u) {
                 float ww[NC];
                 const float* src = DELTA ? wb + u * WC + cg * NC : vg + u * CTB + warp * WC + cg * NC;
                 if (NC == 4) *reinterpret_cast<float4*>(ww) = *reinterpret_cast<const float4*>(src);
                 else *reinterpret_cast<float2*>(ww) = *reinterpret_cast<const float2*>(src);
-                if (!DELTA) {
+                f2 w2[NC];
 #pragma unroll
-                    for (int c = 0; c < NC; ++c) ww[c] *= tab[152 + u];
+                for (int c = 0; c < NC; ++c) {
+                    const float v = DELTA ? ww[c] : ww[c] * tab[152 + u];
+                    w2[c] = pair2(v, v);
                 }
 #pragma unroll
                 for (int qd = 0; qd < NQ; ++qd) {
-                    float kk[4];
-                    if constexpr (HOLD) {
+                    const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(kg + u * KS + qd * 4 * RG);
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) kk[e] = k_r[u * NR + qd * 4 + e];
-                    } else {
-                        *reinterpret_cast<float4*>(kk) = *reinterpret_cast<const float4*>(kg + u * KS + qd * 4 * RG);
+                    for (int c = 0; c < NC; ++c) {
+                        S[qd * 2][c] = fma2(kk.x, w2[c], S[qd * 2][c]);
+                        S[qd * 2 + 1][c] = fma2(kk.y, w2[c], S[qd * 2 + 1][c]);
                     }
-#pragma unroll
-                    for (int e = 0; e < 4; ++e)
-#pragma unroll
-                        for (int c = 0; c < NC; ++c) S[qd * 4 + e][c] = fmaf(kk[e], ww[c], S[qd * 4 + e][c]);
                 }
             }
             // the read-outs, which nothing of the state waits for
@@ -435,16 +471,19 @@ __global__ void __launch_bounds__(THREADS, 2) head_scan_kernel(HeadScanArgs A, i
 #pragma unroll
                 for (int s = 0; s < U; ++s) o = fmaf(p[s], w[s], o);
                 if (!DELTA) o = fmaf(d_skip, vg[t * CTB + own_col], o);
-                if (stores && g * U + t < n_tok) A.out[(size_t)(t0 + g * U + t) * A.H * dv + h * dv + c0 + own_col] = o;
+                if (stores && t < n_tok) A.out[(size_t)(t0 + t) * A.H * dv + h * dv + c0 + own_col] = o;
             }
         }
     }
 #pragma unroll
-    for (int j = 0; j < NR; ++j)
+    for (int i = 0; i < NR / 2; ++i)
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-            const int r = (j / 4) * 4 * RG + 4 * rg + j % 4;
-            if (r < dk && col0 + c < dv) st[(size_t)r * dv + col0 + c] = S[j][c];
+            const int r = (i / 2) * 4 * RG + 4 * rg + 2 * (i % 2);
+            float p, q;
+            split2(S[i][c], p, q);
+            if (col0 + c < dv && r < dk) st[(size_t)r * dv + col0 + c] = p;
+            if (col0 + c < dv && r + 1 < dk) st[(size_t)(r + 1) * dv + col0 + c] = q;
         }
     pdl_launch_dependents();
 }
@@ -591,28 +630,22 @@ __global__ void __launch_bounds__(DT, NI * V <= 32 ? 3 : NI * V <= 64 ? 2 : 1) h
 }
 
 template <bool DELTA, int RG, int NR, int NC>
-static int launch_portions(const HeadScanArgs& A, int num_seqs, int longest, cudaStream_t stream)
+static int launch_portions(const HeadScanArgs& A, int num_seqs, cudaStream_t stream)
 {
     constexpr int KS = RG * NR, WC = 32 / RG * NC, CTB = WARPS * WC;
-    int tc = 32;
-    while (tc > U && tc / 2 >= longest) tc /= 2;
-    auto bytes = [&](int n) {
-        return (2 * (2 * (size_t)n * KS + (size_t)n * CTB + (size_t)(n / U) * TABLE) + (size_t)WARPS * U * WC) * sizeof(float);
-    };
-    while (tc > U && bytes(tc) > 112 * 1024) tc /= 2;            // two blocks an SM
-    const size_t smem = bytes(tc);
-    if (smem > 220 * 1024) SPY_FAIL("head scan: a key size of %d does not fit a block's shared memory", A.dk);
+    constexpr size_t smem = (ring_of(KS) * (U * (2 * (size_t)KS + CTB) + TABLE) + (size_t)WARPS * U * WC) * sizeof(float);
+    static_assert(smem <= 220 * 1024, "the ring fits a block's shared memory");
     const int tiles = (A.dv + CTB - 1) / CTB;
     if (tiles > 65535) SPY_FAIL("head scan: a value size of %d exceeds the grid limit", A.dv);
     auto kernel = head_scan_kernel<DELTA, RG, NR, NC>;
     if (smem > 48 * 1024) SPY_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    spy_launch_in_order(kernel, dim3(num_seqs, A.H, tiles), dim3(THREADS), smem, stream, A, tc);
+    spy_launch_in_order(kernel, dim3(num_seqs, A.H, tiles), dim3(THREADS), smem, stream, A);
     SPY_CHECK_LAUNCH("head scan");
     return 0;
 }
 
 template <bool DELTA, int RG, int NR>
-static int launch_portions_cols(const HeadScanArgs& A, int num_seqs, int longest, cudaStream_t stream)
+static int launch_portions_cols(const HeadScanArgs& A, int num_seqs, cudaStream_t stream)
 {
     // four columns a thread where that still gives the SMs enough blocks, else two
     static int forced = -1;                      // SPYINFER_HEAD_SCAN_COLUMNS = 2 or 4 in the environment fixes it (for measurements)
@@ -624,9 +657,9 @@ static int launch_portions_cols(const HeadScanArgs& A, int num_seqs, int longest
     const long long blocks = (long long)num_seqs * A.H * ((A.dv + wide - 1) / wide);
     const bool four = forced == 4 || (forced != 2 && 3 * blocks >= 2LL * spy_sm_count());      // measured: 128 blocks of four 441 us, 256 of two 471; 64 of four 436, 128 of two 371
     if constexpr (NR <= 16) {
-        if (four) return launch_portions<DELTA, RG, NR, 4>(A, num_seqs, longest, stream);
+        if (four) return launch_portions<DELTA, RG, NR, 4>(A, num_seqs, stream);
     }
-    return launch_portions<DELTA, RG, NR, 2>(A, num_seqs, longest, stream);
+    return launch_portions<DELTA, RG, NR, 2>(A, num_seqs, stream);
 }
 
 template <bool DELTA, int V>
@@ -666,12 +699,12 @@ template <bool DELTA> static int launch_head_scan(const HeadScanArgs& A, int num
     if (vec) spy_launch(head_table_kernel<DELTA, 4>, grid, block, 0, stream, A, num_seqs, num_groups);
     else spy_launch(head_table_kernel<DELTA, 1>, grid, block, 0, stream, A, num_seqs, num_groups);
     SPY_CHECK_LAUNCH("head scan (coefficients)");
-    if (A.dk <= 32) return launch_portions_cols<DELTA, 4, 8>(A, num_seqs, longest, stream);
-    if (A.dk <= 64) return launch_portions_cols<DELTA, 8, 8>(A, num_seqs, longest, stream);
-    if (A.dk <= 128) return launch_portions_cols<DELTA, 16, 8>(A, num_seqs, longest, stream);
-    if (A.dk <= 256) return launch_portions_cols<DELTA, 32, 8>(A, num_seqs, longest, stream);
-    if (A.dk <= 512) return launch_portions_cols<DELTA, 32, 16>(A, num_seqs, longest, stream);
-    return launch_portions_cols<DELTA, 32, 32>(A, num_seqs, longest, stream);
+    if (A.dk <= 32) return launch_portions_cols<DELTA, 4, 8>(A, num_seqs, stream);
+    if (A.dk <= 64) return launch_portions_cols<DELTA, 8, 8>(A, num_seqs, stream);
+    if (A.dk <= 128) return launch_portions_cols<DELTA, 16, 8>(A, num_seqs, stream);
+    if (A.dk <= 256) return launch_portions_cols<DELTA, 32, 8>(A, num_seqs, stream);
+    if (A.dk <= 512) return launch_portions_cols<DELTA, 32, 16>(A, num_seqs, stream);
+    return launch_portions_cols<DELTA, 32, 32>(A, num_seqs, stream);
 }
 
 // Floats of scratch that a step with prompt portions needs (`tables`; it may be null when every request brings one token).

@@ -517,7 +517,7 @@ def _scan_case(kind, heads, share, dk, dv, lens, seed, slow):
     return proj, gates, a_log, dt_bias, d_skip, S, want, last
 
 
-SCAN_SIZES = [(4, 2, 12, 20), (3, 3, 20, 9), (6, 1, 64, 32), (8, 4, 128, 64), (2, 1, 128, 128), (5, 1, 7, 11), (4, 4, 33, 50), (2, 2, 256, 40), (16, 8, 16, 64)]
+SCAN_SIZES = [(4, 2, 12, 20), (3, 3, 20, 9), (6, 1, 64, 32), (8, 4, 128, 64), (2, 1, 128, 128), (5, 1, 7, 11), (4, 4, 33, 50), (2, 2, 256, 40), (16, 8, 16, 64), (2, 1, 300, 24), (1, 1, 643, 16)]
 
 
 @gpu
