@@ -219,17 +219,19 @@ class DynamicTanh(Norm):
         return TanhDelta(y, self.norm, float(scale))
 
     def _pending(self, delta):
+        """What is to be added first, its norm, its multiplier, and this norm: one storage type for the two norms of a launch."""
         if delta is None:
-            return None, None, 1.0
+            return None, None, 1.0, self.norm
         if not isinstance(delta, TanhDelta):
             raise ValueError("dynamic_tanh: what is pending on the stream must be a sublayer output that a norm of this kind deferred")
-        # one storage type for the two norms of a launch
-        norm = delta.norm if self.norm is None or delta.norm[1].dtype == self.norm[1].dtype else tuple(t.to(self.norm[1].dtype) if t.numel() > 1 else t for t in delta.norm)
-        return delta.y, norm, delta.scale
+        theirs, own = delta.norm, self.norm
+        if own is not None and theirs[1].dtype != own[1].dtype:
+            theirs, own = tuple(t.float() for t in theirs), tuple(t.float() for t in own)
+        return delta.y, theirs, delta.scale, own
 
     def add_normed(self, residual, delta):
         """``residual += scale * dyt(y)`` for a ``TanhDelta`` (32-bit, in place)."""
-        y, norm, scale = self._pending(delta)
+        y, norm, scale, _ = self._pending(delta)
         if y is not None:
             kernels.dynamic_tanh(residual, y=y, y_norm=norm, y_scale=scale)
         return residual
@@ -239,7 +241,7 @@ class DynamicTanh(Norm):
         return kernels.dynamic_tanh(x, norm=self.norm, out=out)
 
     def forward_add(self, residual, delta, rows=None, out_dtype=None):
-        y, norm, scale = self._pending(delta)
+        y, norm, scale, own = self._pending(delta)
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.size), dtype=out_dtype or self.ctx.dtype, device=residual.device)
-        return kernels.dynamic_tanh(residual, y=y, y_norm=norm, y_scale=scale, norm=self.norm, out=out, rows=rows)
+        return kernels.dynamic_tanh(residual, y=y, y_norm=norm, y_scale=scale, norm=own, out=out, rows=rows)

@@ -341,6 +341,30 @@ def test_dynamic_tanh_adds_a_result_and_norms_the_stream(dtype):
 
 
 @gpu
+@pytest.mark.parametrize("theirs,own", [(torch.float32, torch.bfloat16), (torch.bfloat16, torch.float32), (torch.bfloat16, torch.bfloat16)])
+def test_two_norms_of_one_launch_may_be_stored_in_different_types(theirs, own):
+    """What a norm in the one type left behind is formed by one in the other, and neither's weights are rounded."""
+    from spyinfer_b200.config import PartSpec
+    from spyinfer_b200.parts import BuildContext, build_part
+
+    g = torch.Generator().manual_seed(6)
+    n, rows = 72, 5
+    ctx = BuildContext(device="cuda", dtype=torch.float32, max_model_len=8)
+    norms, plain = [], []
+    for dtype in (theirs, own):
+        w = {"n": (1.0 + 0.3 * torch.randn(n, generator=g)).to(dtype), "n.b": (0.3 * torch.randn(n, generator=g)).to(dtype), "n.alpha": torch.tensor(0.7).to(dtype)}
+        norms.append(build_part(PartSpec("dynamic_tanh", {"size": n, "weight": "n"}), ctx))
+        norms[-1].bind({k: v.cuda() for k, v in w.items()})
+        plain.append({k: v.double() for k, v in w.items()})
+    h, y = torch.randn(rows, n, generator=g), torch.randn(rows, n, generator=g)
+    hd = h.cuda()
+    out = norms[1].forward_add(hd, norms[0].defer(y.cuda(), 0.5))
+    want = h.double() + 0.5 * P.dynamic_tanh(y.double(), plain[0], "n")
+    assert torch.allclose(hd.cpu().double(), want, atol=3e-6)
+    assert torch.allclose(out.cpu().double(), P.dynamic_tanh(want, plain[1], "n"), atol=3e-6)
+
+
+@gpu
 @pytest.mark.parametrize("dims,base,yarn", [(12, 500.0, (3.0, 64, 8.0, 0.5)), (64, 10000.0, (4.0, 512, 32.0, 1.0)), (16, 100.0, (8.0, 2000, 1.0, 1.0)),
                                             (8, 1e6, (1.0, 4096, 32.0, 1.0)), (24, 10000.0, None), (2, 10.0, (2.0, 5, 64.0, 0.001))])
 def test_the_stretched_rotations_table(dims, base, yarn):
