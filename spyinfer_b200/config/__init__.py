@@ -9,6 +9,8 @@ from . import daronex as _daronex  # registers "Daronex"
 from . import naforax as _naforax  # registers "Naforax"
 from . import dogilorn as _dogilorn  # registers "Dogilorn"
 from . import zonevik as _zonevik  # registers "Zonevik"
+from . import bubalix as _bubalix  # registers "Bubalix"
+from .bubalix import BubalixConfig
 from .daronex import DaronexConfig
 from .dogilorn import DogilornConfig
 from .naforax import NaforaxConfig
@@ -18,5 +20,5 @@ from .zonevik import ZonevikConfig
 
 __all__ = ["EngineConfig", "ArchitectureConfig", "ConfigError", "config_from_json", "known_architectures",
            "load_model_config", "register_architecture", "LayerSpec", "ModelSpec", "PagedCacheNeed", "PartSpec",
-           "RunEntry", "StateCacheNeed", "CompositeCacheNeed", "Qwen3Config", "NezolornConfig", "DaronexConfig", "NaforaxConfig", "DogilornConfig", "ZonevikConfig", "StreamAdd",
+           "RunEntry", "StateCacheNeed", "CompositeCacheNeed", "Qwen3Config", "NezolornConfig", "DaronexConfig", "NaforaxConfig", "DogilornConfig", "ZonevikConfig", "BubalixConfig", "StreamAdd",
            "StreamProject"]

@@ -31,6 +31,8 @@
 // The three arrays must therefore have been written before any kernel that can still be
 // running when this one starts (the engine copies them at the start of the step); the queries
 // and the new token's page are read after the wait.
+// SpyScores (common.cuh): a cap and a distance bias are applied to a key's scores as they come out of tensor memory; learned
+// sinks and the result's scale enter where a head's result is written.
 // Every wait on an mbarrier is bounded; a wait that runs out raises the block's abort flag,
 // which ends all roles, and the status word reports it.
 //
@@ -76,6 +78,7 @@ constexpr int SMEM_TOTAL = BAR_OFF + NUM_BARS * 8 + 32 + 1024;   // then slack t
 constexpr int TMEM_COLS = 64;                                    // S^T: 2 x 16 columns; O^T: 16 columns from 32
 
 struct Params {
+    SpyScores scores;
     bf16* out;                 // [T, nh * hd]
     float* lse;                // null, or [T, nh]: the natural logarithm of every head's sum of exp(score) (for a caller that merges further keys in)
     const int* block_table;    // [S, table_width]
@@ -179,7 +182,20 @@ __device__ __forceinline__ int ordered(float f)
 }
 __device__ __forceinline__ float unordered(int i) { return __int_as_float(i ^ ((i >> 31) & 0x7fffffff)); }
 
-template <int HD, int GN>
+// what a head's denominator takes beside its keys, the maximum in use being m (log2 domain)
+__device__ __forceinline__ float sink_share(const Params& p, int head, float m)
+{
+    return p.scores.sinks != nullptr && m > -INFINITY ? fast_exp2(__ldg(p.scores.sinks + head) * LOG2E - m) : 0.f;
+}
+
+// what a head's result is multiplied by (the kernel ahead may have written it: read after the wait, past the L1)
+__device__ __forceinline__ float result_scale(const Params& p, int tok, int head)
+{
+    return p.scores.out_scale != nullptr ? __ldcg(p.scores.out_scale + (size_t)tok * p.nh + head) : 1.f;
+}
+
+// SCORES: a cap and/or a distance bias on the scores
+template <int HD, int GN, bool SCORES>
 __global__ void __maxnreg__(160)
 attention_decode_kernel(const __grid_constant__ CUtensorMap page_map, const __grid_constant__ CUtensorMap q_map, const Params p)
 {
@@ -313,7 +329,16 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap page_map, const __gr
                 float sc[GN];
 #pragma unroll
                 for (int n = 0; n < GN; ++n) {
-                    sc[n] = visible ? __uint_as_float(r[n]) * p.scale_log2 : -INFINITY;
+                    if constexpr (SCORES) {
+                        // tanh(x) = 1 - 2 / (exp(2 x) + 1), in 32-bit
+                        const float cap = p.scores.softcap;
+                        float v = __uint_as_float(r[n]) * p.scale_log2;
+                        if (cap > 0.f) v = cap * LOG2E * (1.f - 2.f * fast_rcp(fast_exp2(2.f * v / cap) + 1.f));
+                        if (p.scores.slopes != nullptr && n < p.G) v -= __ldg(p.scores.slopes + g.kvh * p.G + n) * LOG2E * (float)(pos - j);
+                        sc[n] = visible ? v : -INFINITY;
+                    } else {
+                        sc[n] = visible ? __uint_as_float(r[n]) * p.scale_log2 : -INFINITY;
+                    }
                     const int mx = __reduce_max_sync(0xffffffffu, ordered(sc[n]));
                     if (lane == n) red[(st * 4 + warp) * NCOLS + n] = unordered(mx);
                 }
@@ -385,11 +410,15 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap page_map, const __gr
             float sums[GN];
 #pragma unroll
             for (int n = 0; n < GN; ++n) sums[n] = (lred[n] + lred[NCOLS + n]) + (lred[2 * NCOLS + n] + lred[3 * NCOLS + n]);
+            if (p.scores.out_scale != nullptr) pdl_wait();
             if (direct) {
 #pragma unroll
                 for (int n = 0; n < GN; ++n) {
-                    if (n < p.G && tid < p.hd)
-                        p.out[((size_t)tok * p.nh + g.kvh * p.G + n) * p.hd + tid] = __float2bfloat16_rn(sums[n] > 0.f ? __uint_as_float(o[n]) / sums[n] : 0.f);
+                    if (n < p.G && tid < p.hd) {
+                        const int head = g.kvh * p.G + n;
+                        const float den = sums[n] + sink_share(p, head, m_used[n]);
+                        p.out[((size_t)tok * p.nh + head) * p.hd + tid] = __float2bfloat16_rn(den > 0.f ? __uint_as_float(o[n]) / den * result_scale(p, tok, head) : 0.f);
+                    }
                     if (p.lse != nullptr && n < p.G && tid == n)
                         p.lse[(size_t)tok * p.nh + g.kvh * p.G + n] = sums[n] > 0.f ? (m_used[n] + log2f(sums[n])) * 0.6931471805599453f : -INFINITY;
                 }
@@ -456,7 +485,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap page_map, const __gr
                             }
                         }
                         bf16* dst = p.out + ((size_t)tok * p.nh + g.kvh * p.G + n) * p.hd + col;
-                        const float inv = L > 0.f ? 1.f / L : 0.f;
+                        const float den = L + sink_share(p, g.kvh * p.G + n, M);
+                        const float inv = den > 0.f ? result_scale(p, tok, g.kvh * p.G + n) / den : 0.f;
                         if (p.lse != nullptr && col == 0) p.lse[(size_t)tok * p.nh + g.kvh * p.G + n] = L > 0.f ? (M + log2f(L)) * 0.6931471805599453f : -INFINITY;
 #pragma unroll
                         for (int i = 0; i < W; i += 8) {
@@ -610,15 +640,22 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap page_map, const __gr
 
 int sm_count() { return spy_sm_count(); }
 
+template <int HD, int GN, bool SCORES>
+int launch_as(const CUtensorMap& page_map, const CUtensorMap& q_map, const Params& p, cudaStream_t stream)
+{
+    SPY_ONCE_PER_DEVICE {
+        SPY_CUDA(cudaFuncSetAttribute(attention_decode_kernel<HD, GN, SCORES>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL));
+    }
+    spy_launch(attention_decode_kernel<HD, GN, SCORES>, dim3(p.blocks), dim3(NUM_THREADS), (size_t)SMEM_TOTAL, stream, page_map, q_map, p);
+    SPY_CHECK_LAUNCH("attention_decode");
+    return 0;
+}
+
 template <int HD, int GN>
 int launch(const CUtensorMap& page_map, const CUtensorMap& q_map, const Params& p, cudaStream_t stream)
 {
-    SPY_ONCE_PER_DEVICE {
-        SPY_CUDA(cudaFuncSetAttribute(attention_decode_kernel<HD, GN>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL));
-    }
-    spy_launch(attention_decode_kernel<HD, GN>, dim3(p.blocks), dim3(NUM_THREADS), (size_t)SMEM_TOTAL, stream, page_map, q_map, p);
-    SPY_CHECK_LAUNCH("attention_decode");
-    return 0;
+    return p.scores.softcap > 0.f || p.scores.slopes != nullptr ? launch_as<HD, GN, true>(page_map, q_map, p, stream)
+                                                                : launch_as<HD, GN, false>(page_map, q_map, p, stream);
 }
 
 }  // namespace
@@ -637,9 +674,10 @@ extern "C" long long spy_attention_decode_scratch_floats(int seqs, int nh, int n
 static int run_attention_decode(const void* q, long long q_row_stride, void* out, float* lse, const void* pages, const int* block_table, int table_width,
                                 int page_size, int num_pages, int nh, int nkv, int hd, const int* positions, const int* q_start, int tokens,
                                 int seqs, int window, float scale, int mode, float* scratch, long long scratch_floats, int* status,
-                                cudaStream_t stream, int planes)
+                                cudaStream_t stream, int planes, SpyScores scores = {0.f, nullptr, nullptr, nullptr})
 {
     if (tokens <= 0 || seqs <= 0) return 0;
+    if (scores.softcap < 0.f) SPY_FAIL("attention_decode: a cap of %g on the scores", scores.softcap);
     if (planes != 1 && planes != 2) SPY_FAIL("attention_decode: a cache of %d planes (1 or 2)", planes);
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) SPY_FAIL("attention_decode: %d query heads do not group over %d key/value heads", nh, nkv);
     const int G = nh / nkv;
@@ -665,6 +703,7 @@ static int run_attention_decode(const void* q, long long q_row_stride, void* out
     if (encode == nullptr) SPY_FAIL("attention_decode: cuTensorMapEncodeTiled is not available from the driver");
 
     Params p;
+    p.scores = scores;
     p.planes = planes;
     p.out = (bf16*)out; p.lse = lse; p.block_table = block_table; p.positions = positions; p.q_start = q_start; p.status = status;
     p.part_o = scratch; p.part_ml = scratch + ((size_t)seqs * nkv + sms) * G * hd_tile;
@@ -717,4 +756,15 @@ extern "C" int spy_attention_decode_lse(const void* q, long long q_row_stride, v
     if (lse == nullptr) SPY_FAIL("attention_decode: no place for the logarithms of the sums");
     return run_attention_decode(q, q_row_stride, out, lse, pages, block_table, table_width, page_size, num_pages, nh, nkv, hd, positions, q_start, tokens,
                                 seqs, window, scale, mode, scratch, scratch_floats, status, stream, planes);
+}
+
+// The same with what a layer does with its scores (SpyScores).
+extern "C" int spy_attention_decode_scores(const void* q, long long q_row_stride, void* out, const void* pages, const int* block_table, int table_width,
+                                           int page_size, int num_pages, int nh, int nkv, int hd, const int* positions, const int* q_start, int tokens,
+                                           int seqs, int window, float scale, int mode, float* scratch, long long scratch_floats, int* status,
+                                           cudaStream_t stream, int planes, float softcap, const float* slopes, const float* sinks, const float* out_scale)
+{
+    const SpyScores scores = {softcap, slopes, sinks, out_scale};
+    return run_attention_decode(q, q_row_stride, out, nullptr, pages, block_table, table_width, page_size, num_pages, nh, nkv, hd, positions, q_start, tokens,
+                                seqs, window, scale, mode, scratch, scratch_floats, status, stream, planes, scores);
 }

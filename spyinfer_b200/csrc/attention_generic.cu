@@ -15,6 +15,7 @@
 // Two options of the mask and the softmax: with a window, `keep_first` > 0 lets every query also see
 // the keys at the sequence's first keep_first positions (at their true positions); `sink` != 0 adds one
 // to the softmax's denominator (a key of score 0 that has no value): p = exp(score) / (1 + sum exp(score)).
+// SpyScores (common.cuh) caps the scores, takes a distance bias off, adds a learned sink a head, scales the result.
 #include "common.cuh"
 
 SPY_MODULE(spy_attention_generic)
@@ -45,7 +46,7 @@ __global__ void __launch_bounds__(CHUNK)
 attention_generic_kernel(const TA* __restrict__ q, long long q_row_stride, TA* __restrict__ out, const TC* __restrict__ pages,
                          const int* __restrict__ block_table, int table_width, int page_size, int num_pages, int nh, int nkv, int hd,
                          const int* __restrict__ positions, const int* __restrict__ seq_of_token, int window, float scale, int* status, int planes,
-                         int keep_first, int sink)
+                         int keep_first, int sink, SpyScores sc)
 {
     extern __shared__ float smem[];
     pdl_enter();
@@ -109,6 +110,8 @@ attention_generic_kernel(const TA* __restrict__ q, long long q_row_stride, TA* _
                 for (int d = 0; d < hd; ++d) dot = fmaf(q_s[d], to_f32(k[d]), dot);
             }
             s = dot * scale;
+            if (sc.softcap > 0.f) s = sc.softcap * tanhf(s / sc.softcap);
+            if (sc.slopes != nullptr) s -= sc.slopes[h] * (float)(pos - j);
         }
         const float chunk_max = block_max(s, scratch);
         const float m_new = fmaxf(m, chunk_max);
@@ -137,11 +140,13 @@ attention_generic_kernel(const TA* __restrict__ q, long long q_row_stride, TA* _
         __syncthreads();  // p_s and row_s are rewritten by the next chunk
     }
     if (sink) l += m == -INFINITY ? 1.f : expf(-m);      // the key of score 0 without a value
+    if (sc.sinks != nullptr) l += m == -INFINITY ? 1.f : expf(sc.sinks[h] - m);      // (too large for 32-bit: the result is 0, as it should be)
+    const float os = sc.out_scale != nullptr ? sc.out_scale[(size_t)t * nh + h] : 1.f;
     TA* o_row = out + ((size_t)t * nh + h) * hd;
 #pragma unroll
     for (int r = 0; r < ACC; ++r) {
         const int d = tid + r * CHUNK;
-        if (d < hd) o_row[d] = from_f32<TA>(l > 0.f ? acc[r] / l : 0.f);
+        if (d < hd) o_row[d] = from_f32<TA>(l > 0.f ? acc[r] / l * os : 0.f);
     }
 }
 
@@ -150,8 +155,11 @@ attention_generic_kernel(const TA* __restrict__ q, long long q_row_stride, TA* _
 extern "C" int spy_attention_generic(const void* q, long long q_row_stride, void* out, int act_dtype, const void* pages, int cache_dtype,
                                      const int* block_table, int table_width, int page_size, int num_pages, int nh, int nkv, int hd,
                                      const int* positions, const int* seq_of_token, int tokens, int window, float scale, int* status,
-                                     cudaStream_t stream, int planes, int keep_first, int sink)
+                                     cudaStream_t stream, int planes, int keep_first, int sink, float softcap, const float* slopes, const float* sinks,
+                                     const float* out_scale)
 {
+    if (softcap < 0.f) SPY_FAIL("attention: a cap of %g on the scores", softcap);
+    const SpyScores scores = {softcap, slopes, sinks, out_scale};
     if (keep_first < 0 || (keep_first > 0 && window <= 0)) SPY_FAIL("attention: kept first keys (%d) go with a window", keep_first);
     if (tokens <= 0) return 0;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) SPY_FAIL("attention: %d query heads do not group over %d key/value heads", nh, nkv);
@@ -165,7 +173,7 @@ extern "C" int spy_attention_generic(const void* q, long long q_row_stride, void
         SPY_DISPATCH_DTYPE(cache_dtype, TC, {
             spy_launch(attention_generic_kernel<TA, TC>, grid, dim3(CHUNK), smem, stream,
                 (const TA*)q, q_row_stride, (TA*)out, (const TC*)pages, block_table, table_width, page_size, num_pages, nh, nkv, hd,
-                positions, seq_of_token, window, scale, status, planes, keep_first, sink);
+                positions, seq_of_token, window, scale, status, planes, keep_first, sink, scores);
         })
     })
     SPY_CHECK_LAUNCH("attention_generic");

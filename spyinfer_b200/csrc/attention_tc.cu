@@ -35,6 +35,10 @@
 // such rows hold finite values that the masks then exclude.  A block whose sequence ends within
 // its first 128 rows (the end of a prompt, a single decoded token of a mixed batch) runs
 // query tile A alone; tile A also leaves out a last key tile that only tile B's tokens see.
+// SpyScores (common.cuh): a cap on the scores and a distance bias are applied to the scores as they are read from tensor
+// memory, in 32-bit.  A cap of at most CAP_AS_REFERENCE needs no running maximum: no score is above the cap, and a query
+// always sees itself, whose score is at least minus the cap, so the probabilities are taken against the cap itself and the
+// scores are read once.  Learned sinks and the result's scale enter where a row's result is stored.
 // Every wait on an mbarrier is bounded; a wait that runs out raises the block's abort flag,
 // which ends all roles, and the status word reports it.
 //
@@ -64,8 +68,11 @@ constexpr int GROUP_THREADS = 128;
 constexpr int NUM_THREADS = 352;     // warp 8: TMEM + MMA; warps 9, 10: TMA of K and of V
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float RESCALE_THRESHOLD = 8.0f;
+constexpr float CAP_AS_REFERENCE = 30.0f;     // 2^(-2 cap log2(e)), the least a query's own key can weigh, times 2^-24 is still a normal 32-bit number
+enum { PLAIN_SCORES = 0, CAPPED_SCORES = 1, BIASED_SCORES = 2 };   // 1: capped at no more than that, with or without a bias; 2: any bias, any cap
 
 struct Params {
+    SpyScores scores;
     const bf16* q;
     long long q_stride;
     bf16* out;                 // [T, nh * hd]
@@ -114,7 +121,7 @@ template <int HD> struct Smem {
 //   MMA thread:       Q_A.K(0), Q_B.K(0), then for every t:
 //                     wait P_A(t), V(t) | P_A.V(t) | wait K(t+1) | Q_A.K(t+1) | wait P_B(t) | P_B.V(t) | Q_B.K(t+1)
 // so the tensor cores work on query tile B while group A works on its probabilities, and the other way round.
-template <int HD>
+template <int HD, int SCORES>
 __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __grid_constant__ CUtensorMap page_map, const Params p)
 {
     using L = Smem<HD>;
@@ -262,7 +269,16 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
             mbar_arrive(bar_q);
             if (tid == 0) describe_next(j + 1);   // while the first scores are on their way
 
-            float m_used = -INFINITY, l = 0.f;   // the maximum the row's probabilities are taken against, and their sum
+            // The scores' transform, in the log2 domain: tanh(x) = 1 - 2 / (exp(2 x) + 1), and the bias of key0 + i is bias0 + i * slope2.
+            const float cap = SCORES != PLAIN_SCORES ? p.scores.softcap : 0.f, cap_log2 = cap * LOG2E;
+            const float cap_in = cap > 0.f ? 2.f * p.scale_log2 / cap : 0.f;
+            const float slope2 = (SCORES != PLAIN_SCORES && p.scores.slopes != nullptr && row_ok) ? __ldg(p.scores.slopes + head) * LOG2E : 0.f;
+            auto biased = [&](float s, int i, float bias0) {        // SCORES == BIASED_SCORES: the whole transform of one score
+                const float v = cap > 0.f ? cap_log2 - 2.f * cap_log2 * fast_rcp(fast_exp2(s * cap_in) + 1.f) : s * p.scale_log2;
+                return v + fmaf((float)i, slope2, bias0);
+            };
+
+            float m_used = SCORES == CAPPED_SCORES ? cap_log2 : -INFINITY, l = 0.f;   // the maximum the row's probabilities are taken against, and their sum
             for (int t = 0; t < my_tiles; ++t, ++count) {
                 const uint32_t ph = (uint32_t)count & 1;
                 alive = mbar_wait(bar_s + grp, ph, abort_flag);          // S_g(t) is complete
@@ -270,6 +286,44 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
                 fence_after_sync();
                 const int key0 = (tile_first + t) * TILE;
                 const bool whole = __all_sync(0xffffffffu, !row_ok || (key0 >= lo && key0 + TILE - 1 <= pos));
+                const float bias0 = slope2 * (float)(key0 - pos);
+                if constexpr (SCORES == CAPPED_SCORES) {
+                    float sums[2] = {0.f, 0.f};
+#pragma unroll
+                    for (int h = 0; h < 2; ++h) {
+                        uint32_t sc[HALF];
+#pragma unroll
+                        for (int c = 0; c < HALF; c += 32) tmem_load<32>(tmem_s + h * HALF + c, *reinterpret_cast<uint32_t(*)[32]>(&sc[c]));
+                        tmem_wait_ld();
+                        uint32_t packed[HALF / 2];
+#pragma unroll
+                        for (int i = 0; i < HALF; i += 2) {
+                            float pr[2];
+#pragma unroll
+                            for (int e = 0; e < 2; ++e) {
+                                // cap tanh(s scale / cap) - cap, with the bias: two units of exp2 and one reciprocal a score
+                                const float r = fast_rcp(fast_exp2(__uint_as_float(sc[i + e]) * cap_in) + 1.f);
+                                pr[e] = fast_exp2(fmaf(-2.f * cap_log2, r, fmaf((float)(h * HALF + i + e), slope2, bias0)));
+                            }
+                            if (!whole) {
+#pragma unroll
+                                for (int e = 0; e < 2; ++e) {
+                                    const int k = key0 + h * HALF + i + e;
+                                    if (!(k <= pos && k >= lo)) pr[e] = 0.f;
+                                }
+                            }
+                            sums[0] += pr[0];
+                            sums[1] += pr[1];
+                            packed[i / 2] = pack_bf16(pr[0], pr[1]);
+                        }
+                        tmem_store<32>(tmem_s + h * (HALF / 2), packed);
+                    }
+                    l += sums[0] + sums[1];
+                    tmem_wait_st();
+                    fence_before_sync();
+                    mbar_arrive(bar_p + grp);
+                    continue;
+                }
                 // First reading of the row's 128 raw scores: the maximum, by 3-input max in four independent chains
                 // (on the raw scores: the scale is positive).  Scores the row does not see count as -inf.
                 float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -279,6 +333,10 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
 #pragma unroll
                     for (int c = 0; c < HALF; c += 32) tmem_load<32>(tmem_s + h * HALF + c, *reinterpret_cast<uint32_t(*)[32]>(&sc[c]));
                     tmem_wait_ld();
+                    if constexpr (SCORES == BIASED_SCORES) {
+#pragma unroll
+                        for (int i = 0; i < HALF; ++i) sc[i] = __float_as_uint(biased(__uint_as_float(sc[i]), h * HALF + i, bias0));
+                    }
                     if (!whole) {
 #pragma unroll
                         for (int i = 0; i < HALF; ++i) {
@@ -292,7 +350,7 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
                         for (int c = 0; c < 4; ++c) mx4[c] = max3(mx4[c], __uint_as_float(sc[i + 2 * c]), __uint_as_float(sc[i + 2 * c + 1]));
                     }
                 }
-                const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
+                const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (SCORES == BIASED_SCORES ? 1.f : p.scale_log2);
                 // the maximum in use moves only when the row's maximum grew by more than the threshold (or from nothing)
                 const float m_new = fmaxf(m_used, mx);
                 const bool grow = m_new > m_used + RESCALE_THRESHOLD || (m_used == -INFINITY && m_new != -INFINITY);
@@ -322,7 +380,8 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
                 // exp2(s * scale - m), one packed FMA for two scores; the sum runs in two packed accumulators.  P goes
                 // over the first 64 columns of S, 64 keys at a time: the columns written have been read before.
                 const float neg_m = m_used == -INFINITY ? 0.f : -m_used;
-                const uint64_t scale2 = pack2(p.scale_log2, p.scale_log2), neg2 = pack2(neg_m, neg_m);
+                const float second_scale = SCORES == BIASED_SCORES ? 1.f : p.scale_log2;
+                const uint64_t scale2 = pack2(second_scale, second_scale), neg2 = pack2(neg_m, neg_m);
                 uint64_t sum2[2] = {0ull, 0ull};
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
@@ -330,6 +389,10 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
 #pragma unroll
                     for (int c = 0; c < HALF; c += 32) tmem_load<32>(tmem_s + h * HALF + c, *reinterpret_cast<uint32_t(*)[32]>(&sc[c]));
                     tmem_wait_ld();
+                    if constexpr (SCORES == BIASED_SCORES) {
+#pragma unroll
+                        for (int i = 0; i < HALF; ++i) sc[i] = __float_as_uint(biased(__uint_as_float(sc[i]), h * HALF + i, bias0));
+                    }
                     if (!whole) {
 #pragma unroll
                         for (int i = 0; i < HALF; ++i) {
@@ -371,7 +434,9 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
             if (q_requested) request_q(item_ring[(j + 1) & 1]);
             // ---- ... and this item's output is read and stored meanwhile: O_g / l
             if (my_tiles > 0) {
-                const float inv = l > 0.f ? 1.f / l : 0.f;
+                if (p.scores.sinks != nullptr && row_ok && m_used > -INFINITY) l += fast_exp2(__ldg(p.scores.sinks + head) * LOG2E - m_used);
+                float inv = l > 0.f ? 1.f / l : 0.f;
+                if (p.scores.out_scale != nullptr && row_ok) inv *= p.scores.out_scale[(size_t)tok * p.nh + head];
                 if (p.lse != nullptr && row_ok) p.lse[(size_t)tok * p.nh + head] = l > 0.f ? (m_used + log2f(l)) * 0.6931471805599453f : -INFINITY;
                 bf16* dst = p.out + ((size_t)(row_ok ? tok : 0) * p.nh + head) * p.hd;
 #pragma unroll 1
@@ -534,15 +599,25 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
     }
 }
 
+template <int HD, int SCORES>
+int launch(dim3 grid, const CUtensorMap& page_map, const Params& p, cudaStream_t stream)
+{
+    SPY_ONCE_PER_DEVICE { SPY_CUDA(cudaFuncSetAttribute(attention_tc_kernel<HD, SCORES>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<HD>::TOTAL)); }
+    spy_launch(attention_tc_kernel<HD, SCORES>, grid, dim3(NUM_THREADS), (size_t)Smem<HD>::TOTAL, stream, page_map, p);
+    SPY_CHECK_LAUNCH("attention_tc");
+    return 0;
+}
+
 }  // namespace
 
 
 // Attention of a batch over its pages: prompt portions, any mix, single tokens included.
 static int run_attention_tc(const void* q, long long q_row_stride, void* out, float* lse, const void* pages, const int* block_table, int table_width,
                             int page_size, int num_pages, int nh, int nkv, int hd, const int* positions, const int* q_start, int tokens,
-                            int seqs, int window, float scale, int* status, cudaStream_t stream, int planes)
+                            int seqs, int window, float scale, int* status, cudaStream_t stream, int planes, SpyScores scores = {0.f, nullptr, nullptr, nullptr})
 {
     if (tokens <= 0 || seqs <= 0) return 0;
+    if (scores.softcap < 0.f) SPY_FAIL("attention_tc: a cap of %g on the scores", scores.softcap);
     if (planes != 1 && planes != 2) SPY_FAIL("attention_tc: a cache of %d planes (1 or 2)", planes);
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) SPY_FAIL("attention_tc: %d query heads do not group over %d key/value heads", nh, nkv);
     const int G = nh / nkv;
@@ -554,6 +629,7 @@ static int run_attention_tc(const void* q, long long q_row_stride, void* out, fl
     if (page_size <= 0 || num_pages <= 0 || table_width <= 0) SPY_FAIL("attention_tc: page_size, num_pages and table_width must be positive");
     const int Gp = G;   // rows a token takes in a query tile: one per head of the group (128 / G tokens a tile, the remainder of the rows stays empty)
     Params p;
+    p.scores = scores;
     p.planes = planes;
     p.q = (const bf16*)q; p.q_stride = q_row_stride; p.out = (bf16*)out; p.lse = lse; p.block_table = block_table;
     p.positions = positions; p.q_start = q_start; p.status = status; p.table_width = table_width; p.page_size = page_size;
@@ -575,10 +651,6 @@ static int run_attention_tc(const void* q, long long q_row_stride, void* out, fl
                             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
         if (r != CUDA_SUCCESS) SPY_FAIL("attention_tc: cuTensorMapEncodeTiled failed with code %d", (int)r);
     }
-    SPY_ONCE_PER_DEVICE {
-        SPY_CUDA(cudaFuncSetAttribute(attention_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<64>::TOTAL));
-        SPY_CUDA(cudaFuncSetAttribute(attention_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Smem<128>::TOTAL));
-    }
     const int tokens_per_block = 2 * (BLOCK_ROWS / 2 / Gp);
     const long long blocks = (tokens + tokens_per_block - 1) / tokens_per_block + seqs;   // an upper bound without a host copy of q_start
     const long long items = blocks * nkv;
@@ -589,10 +661,10 @@ static int run_attention_tc(const void* q, long long q_row_stride, void* out, fl
     // last tiles of the one before are worked on)
     const int sms = spy_sm_count();
     dim3 grid((unsigned)(items < sms ? items : sms));
-    if (hd <= 64) spy_launch(attention_tc_kernel<64>, grid, dim3(NUM_THREADS), (size_t)Smem<64>::TOTAL, stream, page_map, p);
-    else spy_launch(attention_tc_kernel<128>, grid, dim3(NUM_THREADS), (size_t)Smem<128>::TOTAL, stream, page_map, p);
-    SPY_CHECK_LAUNCH("attention_tc");
-    return 0;
+    if (scores.softcap == 0.f && scores.slopes == nullptr) return hd <= 64 ? launch<64, PLAIN_SCORES>(grid, page_map, p, stream) : launch<128, PLAIN_SCORES>(grid, page_map, p, stream);
+    if (scores.softcap > 0.f && scores.softcap <= CAP_AS_REFERENCE)
+        return hd <= 64 ? launch<64, CAPPED_SCORES>(grid, page_map, p, stream) : launch<128, CAPPED_SCORES>(grid, page_map, p, stream);
+    return hd <= 64 ? launch<64, BIASED_SCORES>(grid, page_map, p, stream) : launch<128, BIASED_SCORES>(grid, page_map, p, stream);
 }
 
 extern "C" int spy_attention_tc(const void* q, long long q_row_stride, void* out, const void* pages, const int* block_table, int table_width,
@@ -612,4 +684,15 @@ extern "C" int spy_attention_tc_lse(const void* q, long long q_row_stride, void*
     if (lse == nullptr) SPY_FAIL("attention_tc: no place for the logarithms of the sums");
     return run_attention_tc(q, q_row_stride, out, lse, pages, block_table, table_width, page_size, num_pages, nh, nkv, hd, positions, q_start, tokens, seqs,
                             window, scale, status, stream, planes);
+}
+
+// The same with what a layer does with its scores (SpyScores).
+extern "C" int spy_attention_tc_scores(const void* q, long long q_row_stride, void* out, const void* pages, const int* block_table, int table_width,
+                                       int page_size, int num_pages, int nh, int nkv, int hd, const int* positions, const int* q_start, int tokens,
+                                       int seqs, int window, float scale, int* status, cudaStream_t stream, int planes, float softcap,
+                                       const float* slopes, const float* sinks, const float* out_scale)
+{
+    const SpyScores scores = {softcap, slopes, sinks, out_scale};
+    return run_attention_tc(q, q_row_stride, out, nullptr, pages, block_table, table_width, page_size, num_pages, nh, nkv, hd, positions, q_start, tokens, seqs,
+                            window, scale, status, stream, planes, scores);
 }

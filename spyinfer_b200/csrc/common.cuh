@@ -185,6 +185,18 @@ __device__ __forceinline__ int spy_first_key(int pos, int mask)
     return mask > 0 ? max(0, pos - mask + 1) : (mask < 0 ? pos - pos % (-mask) : 0);
 }
 
+// What a layer does with its scores and results beside scaling them (all off when zero or null); the attention kernels take it
+// by value.  For a query at position i and a key at position j under head h:
+//   score = softcap * tanh(q . k * scale / softcap)   (softcap 0: q . k * scale)      - slopes[h] * (i - j)
+// The softmax's denominator also holds exp(sinks[h]), a number without a key or a value that is neither scaled, capped nor
+// biased; the result is multiplied by out_scale[token, h].
+struct SpyScores {
+    float softcap;
+    const float* slopes;       // [heads]
+    const float* sinks;        // [heads]
+    const float* out_scale;    // [tokens, heads]
+};
+
 __device__ __forceinline__ void report_status(int* status, int code, int detail)
 {
     if (status != nullptr && atomicCAS(status, 0, code) == 0) status[1] = detail;

@@ -196,3 +196,44 @@ extern "C" int spy_stream_concat(const float* stream, const void* table, int tab
     SPY_CHECK_LAUNCH("stream_concat");
     return 0;
 }
+
+// out[t, j] = act(gate[t, j]) * table[ids[t], col + j] for j < dim: a token's own vector (a layer's share of a wider table row) let
+// through by a gate that was projected from the stream; gate [T, dim] or a stack of split-K partial sums.  act: 0 the tanh form of gelu.
+template <typename TG, typename TW, typename TO>
+__global__ void __launch_bounds__(128)
+token_gate_kernel(const TG* __restrict__ gate, int splits, long long split_stride, const TW* __restrict__ table, long long table_ld, int col,
+                  const int* __restrict__ ids, int vocab, TO* __restrict__ out, int dim, int* status)
+{
+    pdl_enter();
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    const bool ok = id >= 0 && id < vocab;
+    if (!ok && threadIdx.x == 0 && blockIdx.y == 0) report_status(status, SPY_STATUS_BAD_TOKEN, t);
+    const int j = blockIdx.y * blockDim.x + threadIdx.x;
+    if (j >= dim) return;
+    const float e = ok ? to_f32(table[(long long)id * table_ld + col + j]) : 0.f;
+    float z = to_f32(gate[(long long)t * dim + j]);
+#pragma unroll 4
+    for (int s = 1; s < splits; ++s) z += to_f32(gate[s * split_stride + (long long)t * dim + j]);
+    const float g = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    out[(long long)t * dim + j] = from_f32<TO>(g * e);
+}
+
+extern "C" int spy_token_gate(const void* gate, int gate_dtype, int splits, long long split_stride, const void* table, int table_dtype, long long table_ld,
+                              int col, const int* ids, int vocab, void* out, int out_dtype, int tokens, int dim, int act, int* status, cudaStream_t stream)
+{
+    if (tokens <= 0) return 0;
+    if (dim <= 0 || vocab <= 0 || splits < 1 || col < 0 || col + dim > table_ld) SPY_FAIL("token_gate: columns %d .. %d do not lie within a table row of %lld", col, col + dim, table_ld);
+    if (act != 0) SPY_FAIL("token_gate: activation code %d", act);
+    const dim3 grid(tokens, (dim + 127) / 128);
+    SPY_DISPATCH_DTYPE(gate_dtype, TG, {
+        SPY_DISPATCH_DTYPE(table_dtype, TW, {
+            SPY_DISPATCH_DTYPE(out_dtype, TO, {
+                spy_launch(token_gate_kernel<TG, TW, TO>, grid, dim3(128), 0, stream, (const TG*)gate, splits, split_stride, (const TW*)table, table_ld, col, ids,
+                           vocab, (TO*)out, dim, status);
+            })
+        })
+    })
+    SPY_CHECK_LAUNCH("token_gate");
+    return 0;
+}

@@ -119,7 +119,7 @@ constexpr int NC = 128;         // output columns a pass of a block takes: one a
 // shared memory too, KC rows of the block's 128 columns at a time, every thread's loads of a chunk under way together
 // (a thread that fetched its column's weights one after the other from L2 spent its time waiting for them).  A token's
 // sum runs over the inputs in their order whatever NT is.
-template <typename TA, typename TW, int NT>
+template <typename TI, typename TA, typename TW, int NT>
 __global__ void __launch_bounds__(128) head_product_kernel(HeadProductArgs A)
 {
     extern __shared__ __align__(16) float in_s[];        // [K + tail][NT + 4] (the pad spreads a column's stores over the banks), then the weights' chunk [KC][NC]
@@ -128,7 +128,7 @@ __global__ void __launch_bounds__(128) head_product_kernel(HeadProductArgs A)
     const int t0 = blockIdx.x * NT, h = blockIdx.y, tid = threadIdx.x;
     const int n_tok = min(NT, A.T - t0), KT = A.K + A.tail;
     float* w_s = in_s + (size_t)KT * LD;
-    const TA* in = (const TA*)A.in;
+    const TI* in = (const TI*)A.in;
     TA* out = (TA*)A.out;
     for (int first = tid; first < NT * KT; first += 8 * 128) {        // eight loads a thread under way at a time
         float v[8];
@@ -211,8 +211,9 @@ __global__ void __launch_bounds__(128) head_product_kernel(HeadProductArgs A)
 }
 
 // in [T, in_ld]: head h's K inputs (and `tail` more) start at column h * in_head_stride.  W [H][K][N] (w_dtype).
-// out [T, out_ld]: head h's N results (and the rotated tail) start at column h * out_head_stride.  in and out have act_dtype.
-extern "C" int spy_head_product(const void* in, long long in_ld, int in_head_stride, int K, const void* W, int w_dtype, int N, void* out, long long out_ld,
+// out [T, out_ld]: head h's N results (and the rotated tail) start at column h * out_head_stride.  `in` has in_dtype (act_dtype, or
+// float32: a part of a projection that was left in 32-bit), out act_dtype.
+extern "C" int spy_head_product(const void* in, int in_dtype, long long in_ld, int in_head_stride, int K, const void* W, int w_dtype, int N, void* out, long long out_ld,
                                 int out_head_stride, int act_dtype, int tail, const float* rope, int rot_half, int table_rows, int interleaved,
                                 const int* positions, const float* gate, long long gate_ld, int gate_off, int tokens, int heads, int* status,
                                 cudaStream_t stream)
@@ -226,11 +227,19 @@ extern "C" int spy_head_product(const void* in, long long in_ld, int in_head_str
     if (smem > 160 * 1024) SPY_FAIL("head_product: %d inputs a head do not fit a block's shared memory", K + tail);
     HeadProductArgs A = {in, in_ld, in_head_stride, K, W, N, out, out_ld, out_head_stride, tail, rope, rot_half, table_rows, interleaved, positions,
                          gate, gate_ld, gate_off, tokens, status};
+    if (in_dtype != act_dtype && in_dtype != SPY_F32) SPY_FAIL("head_product: inputs of dtype code %d for results of dtype code %d", in_dtype, act_dtype);
+    auto run = [&](auto kernel) -> cudaError_t {
+        if (smem > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (e != cudaSuccess) return e;
+        }
+        spy_launch(kernel, dim3((tokens + nt - 1) / nt, heads), dim3(128), smem, stream, A);
+        return cudaSuccess;
+    };
     SPY_DISPATCH_DTYPE(act_dtype, TA, {
         SPY_DISPATCH_DTYPE(w_dtype, TW, {
-            auto kernel = nt == 16 ? head_product_kernel<TA, TW, 16> : head_product_kernel<TA, TW, TOK>;
-            if (smem > 48 * 1024) SPY_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-            spy_launch(kernel, dim3((tokens + nt - 1) / nt, heads), dim3(128), smem, stream, A);
+            if (in_dtype == SPY_F32) SPY_CUDA(nt == 16 ? run(head_product_kernel<float, TA, TW, 16>) : run(head_product_kernel<float, TA, TW, TOK>));
+            else SPY_CUDA(nt == 16 ? run(head_product_kernel<TA, TA, TW, 16>) : run(head_product_kernel<TA, TA, TW, TOK>));
         })
     })
     SPY_CHECK_LAUNCH("head_product");

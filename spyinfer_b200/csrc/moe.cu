@@ -14,7 +14,9 @@
 // only (the weights stay the plain scores); the outputs form `group_count` equal groups of neighbours, a group's score is its
 // largest choice score (`group_score` 1: the sum of its two largest), and only the outputs of the `group_keep` best groups can be
 // chosen.  `act` 1: an expert is weight * silu(gate) * up, without clamps.  `score` 1: the scores are sigmoid(logit) instead of a
-// softmax over all outputs.
+// softmax over all outputs.  A `table` [vocab, top] of expert numbers takes the router's place altogether: a token's id gives its
+// experts, each with the weight 1 / top (an expert that a row names twice counts twice).  `shared_plain`: the shared expert has the
+// weight 1, there is no gate.
 #include "common.cuh"
 
 SPY_MODULE(spy_moe)
@@ -30,6 +32,10 @@ struct MoeRouting {
     float* shared_weight;          // null, or [T]: the shared expert's weight (sigmoid of its gate's logit)
     int score;                     // 0: softmax over all outputs; 1: sigmoid of each
     int group_score;               // 0: a group counts by its largest choice score; 1: by the sum of its two largest
+    const int* table;              // null, or [vocab, top]: the experts of every token id, in place of the router's logits
+    const int* ids;                // with a table: the step's token ids
+    int vocab;
+    int shared_plain;              // 1: the shared expert's weight is 1
 };
 
 template <typename TA, typename TO>
@@ -46,60 +52,73 @@ __global__ void moe_activation_kernel(const TA* __restrict__ gu, long long gu_ld
     float* kept_w = w_s + total + 1;               // kept_w[e]: the weight if chosen, else 0
     float* choice = kept_w + total;                // the score the choice goes by
     float* group_s = choice + total;
-    // softmax over all outputs, or the sigmoid of each
-    float m = -INFINITY, s = 0.f;
-    if (r.score == 0) {
-        for (int e = tid; e < total; e += blockDim.x) m = fmaxf(m, lg[e]);
-        m = block_max(m, scratch);
-        for (int e = tid; e < total; e += blockDim.x) s += expf(lg[e] - m);
-        s = block_sum(s, scratch);
-    }
-    for (int e = tid; e < total; e += blockDim.x) {
-        const float v = r.score == 0 ? expf(lg[e] - m) / s : 1.0f / (1.0f + expf(-lg[e]));
-        w_s[e] = v;
-        choice[e] = r.correction != nullptr ? v + r.correction[e] : v;
-    }
-    __syncthreads();
-    if (r.group_count > 0) {
-        // a group's score is its largest choice score, or the sum of its two largest; a group stays when fewer than group_keep groups beat it
-        const int per = total / r.group_count;
-        for (int g = tid; g < r.group_count; g += blockDim.x) {
-            float best = -INFINITY, next = -INFINITY;
-            for (int e = g * per; e < g * per + per; ++e) {
-                const float v = choice[e];
-                if (v > best) {
-                    next = best;
-                    best = v;
-                } else {
-                    next = fmaxf(next, v);
-                }
-            }
-            group_s[g] = r.group_score == 1 && per > 1 ? best + next : best;
-        }
+    if (r.table != nullptr) {
+        // no scores: the token id names its experts
+        for (int e = tid; e < total; e += blockDim.x) kept_w[e] = 0.f;
         __syncthreads();
+        const int id = r.ids[t];
+        if (id >= 0 && id < r.vocab) {
+            for (int k = tid; k < top; k += blockDim.x) {
+                const int e = r.table[(long long)id * top + k];
+                if (e >= 0 && e < experts) atomicAdd(kept_w + e, 1.0f / (float)top);
+            }
+        }
+    } else {
+        // softmax over all outputs, or the sigmoid of each
+        float m = -INFINITY, s = 0.f;
+        if (r.score == 0) {
+            for (int e = tid; e < total; e += blockDim.x) m = fmaxf(m, lg[e]);
+            m = block_max(m, scratch);
+            for (int e = tid; e < total; e += blockDim.x) s += expf(lg[e] - m);
+            s = block_sum(s, scratch);
+        }
         for (int e = tid; e < total; e += blockDim.x) {
-            const int g = e / per;
-            const float v = group_s[g];
-            int ahead = 0;
-            for (int o = 0; o < r.group_count; ++o) {
-                const float x = group_s[o];
-                ahead += (x > v || (x == v && o < g)) ? 1 : 0;
-            }
-            if (ahead >= r.group_keep) choice[e] = -INFINITY;
+            const float v = r.score == 0 ? expf(lg[e] - m) / s : 1.0f / (1.0f + expf(-lg[e]));
+            w_s[e] = v;
+            choice[e] = r.correction != nullptr ? v + r.correction[e] : v;
         }
         __syncthreads();
-    }
-    // the `top` largest stay: an output stays when fewer than `top` beat it (a larger choice score, or an equal one at a lower index)
-    for (int e = tid; e < total; e += blockDim.x) {
-        const float v = choice[e];
-        int ahead = 0;
-        for (int o = 0; o < total; ++o) {
-            const float x = choice[o];
-            ahead += (x > v || (x == v && o < e)) ? 1 : 0;
+        if (r.group_count > 0) {
+            // a group's score is its largest choice score, or the sum of its two largest; a group stays when fewer than group_keep groups beat it
+            const int per = total / r.group_count;
+            for (int g = tid; g < r.group_count; g += blockDim.x) {
+                float best = -INFINITY, next = -INFINITY;
+                for (int e = g * per; e < g * per + per; ++e) {
+                    const float v = choice[e];
+                    if (v > best) {
+                        next = best;
+                        best = v;
+                    } else {
+                        next = fmaxf(next, v);
+                    }
+                }
+                group_s[g] = r.group_score == 1 && per > 1 ? best + next : best;
+            }
+            __syncthreads();
+            for (int e = tid; e < total; e += blockDim.x) {
+                const int g = e / per;
+                const float v = group_s[g];
+                int ahead = 0;
+                for (int o = 0; o < r.group_count; ++o) {
+                    const float x = group_s[o];
+                    ahead += (x > v || (x == v && o < g)) ? 1 : 0;
+                }
+                if (ahead >= r.group_keep) choice[e] = -INFINITY;
+            }
+            __syncthreads();
         }
-        kept_w[e] = (ahead < top && v > -INFINITY) ? w_s[e] : 0.f;
+        // the `top` largest stay: an output stays when fewer than `top` beat it (a larger choice score, or an equal one at a lower index)
+        for (int e = tid; e < total; e += blockDim.x) {
+            const float v = choice[e];
+            int ahead = 0;
+            for (int o = 0; o < total; ++o) {
+                const float x = choice[o];
+                ahead += (x > v || (x == v && o < e)) ? 1 : 0;
+            }
+            kept_w[e] = (ahead < top && v > -INFINITY) ? w_s[e] : 0.f;
+        }
     }
-    if (tid == 0) w_s[total] = shared_ff > 0 ? 1.0f / (1.0f + expf(-lg[total])) : 0.f;
+    if (tid == 0) w_s[total] = shared_ff <= 0 ? 0.f : (r.shared_plain ? 1.0f : 1.0f / (1.0f + expf(-lg[total])));
     __syncthreads();
     if (r.id_weight != nullptr && tid == 0) {
         float idw = 0.f;
@@ -199,7 +218,7 @@ extern "C" int spy_moe_activation(const void* gu, int gu_dtype, long long gu_ld,
                                   long long y_ld, int tokens, int experts, int top, int ff, float limit, int shared_ff, float shared_limit, float alpha,
                                   float* weights_out, cudaStream_t stream)
 {
-    MoeRouting r = {0, nullptr, 0, 0, 0, nullptr, nullptr, 0, 0};
+    MoeRouting r = {0, nullptr, 0, 0, 0, nullptr, nullptr, 0, 0, nullptr, nullptr, 0, 0};
     return run_moe_activation(gu, gu_dtype, gu_ld, logits, logits_ld, y, y_dtype, y_ld, tokens, experts, top, ff, limit, shared_ff, shared_limit, alpha,
                               weights_out, r, stream);
 }
@@ -212,9 +231,21 @@ extern "C" int spy_moe_activation_routed(const void* gu, int gu_dtype, long long
                                          float* id_weight, float* shared_weight, cudaStream_t stream, int score, int group_score)
 {
     if (gu == nullptr && weights_out == nullptr) SPY_FAIL("moe_activation: neither activations nor weights are asked for");
-    MoeRouting r = {identity, correction, group_count, group_keep, act, id_weight, shared_weight, score, group_score};
+    MoeRouting r = {identity, correction, group_count, group_keep, act, id_weight, shared_weight, score, group_score, nullptr, nullptr, 0, 0};
     return run_moe_activation(gu, gu_dtype, gu_ld, logits, logits_ld, y, y_dtype, y_ld, tokens, experts, top, ff, limit, shared_ff, shared_limit, alpha,
                               weights_out, r, stream);
+}
+
+// The activations with the experts named by a table [vocab, top] of the step's token ids.  shared_gate: null, or [tokens, gate_ld]
+// float32 logits of the shared expert's gate (null with shared_ff > 0: its weight is 1).
+extern "C" int spy_moe_activation_table(const void* gu, int gu_dtype, long long gu_ld, const int* table, const int* ids, int vocab, const float* shared_gate,
+                                        long long gate_ld, void* y, int y_dtype, long long y_ld, int tokens, int experts, int top, int ff, float limit,
+                                        int shared_ff, float shared_limit, float alpha, int act, cudaStream_t stream)
+{
+    if (gu == nullptr || table == nullptr || ids == nullptr || vocab <= 0) SPY_FAIL("moe_activation: a table of experts needs token ids, a vocabulary and inputs");
+    MoeRouting r = {0, nullptr, 0, 0, act, nullptr, nullptr, 0, 0, table, ids, vocab, shared_gate == nullptr ? 1 : 0};
+    return run_moe_activation(gu, gu_dtype, gu_ld, shared_gate != nullptr ? shared_gate - experts : nullptr, gate_ld, y, y_dtype, y_ld, tokens, experts, top, ff,
+                              limit, shared_ff, shared_limit, alpha, nullptr, r, stream);
 }
 
 // out[t, :] += w[t] * x[t, :] in 32-bit (out float32): what the identity experts of a mixture contribute.
@@ -382,7 +413,7 @@ __global__ void expert_activation_kernel(const TA* __restrict__ gu, long long gu
 {
     pdl_enter();
     const long long r = blockIdx.x;
-    const float w = row_w[r];
+    const float w = row_w != nullptr ? row_w[r] : 1.f;
     const TA* src = gu + r * gu_ld;
     TO* dst = y + r * y_ld;
     if constexpr (sizeof(TA) == 2 && sizeof(TO) == 2) {
@@ -539,6 +570,49 @@ extern "C" int spy_moe_route_weights(const float* weights, long long ld, int tok
     spy_launch_in_order(moe_pairs_kernel, dim3(blocks), dim3(32 * warps), (size_t)experts * sizeof(int), stream, weights, ld, tokens, experts, top, choice,
                         choice_w, slot, counts);
     SPY_CHECK_LAUNCH("moe_pairs");
+    spy_launch(moe_slots_kernel, dim3(experts), dim3(1024), 0, stream, (const int*)choice, (const float*)choice_w, (const int*)counts,
+               tokens * top, top, experts, offsets, slot, row_token, row_w, pad < 1 ? 1 : pad, tile_expert, pad > 1 ? num_rows / pad : 0);
+    SPY_CHECK_LAUNCH("moe_slots");
+    return 0;
+}
+
+// The pairs of a step whose experts a table [vocab, top] names by token id, all with the weight 1 / top, in the table's order.
+__global__ void moe_table_kernel(const int* __restrict__ table, const int* __restrict__ ids, int vocab, long long pairs, int experts, int top,
+                                 int* __restrict__ choice, float* __restrict__ choice_w, int* __restrict__ slot, int* __restrict__ counts)
+{
+    extern __shared__ int hist_s[];
+    pdl_enter();
+    for (int e = threadIdx.x; e < experts; e += blockDim.x) hist_s[e] = 0;
+    __syncthreads();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < pairs; i += (long long)gridDim.x * blockDim.x) {
+        const long long t = i / top;
+        const int id = ids[t];
+        int e = id >= 0 && id < vocab ? table[(long long)id * top + (i - t * top)] : -1;
+        if (e < 0 || e >= experts) e = -1;
+        choice[i] = e;
+        choice_w[i] = e >= 0 ? 1.0f / (float)top : 0.f;
+        slot[i] = -1;
+        if (e >= 0) atomicAdd(hist_s + e, 1);
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < experts; e += blockDim.x)
+        if (hist_s[e] != 0) atomicAdd(counts + e, hist_s[e]);
+}
+
+// The other arrays as for spy_moe_route.
+extern "C" int spy_moe_route_table(const int* table, const int* ids, int vocab, int tokens, int experts, int top, int* choice, float* choice_w, int* counts,
+                                   int* offsets, int* slot, int* row_token, float* row_w, cudaStream_t stream, int pad, int* tile_expert, int num_rows)
+{
+    if (tokens <= 0) return 0;
+    if (int rc = prepare_rows(tokens, experts, top, pad, tile_expert, num_rows, row_token, stream)) return rc;
+    if (table == nullptr || ids == nullptr || vocab <= 0) SPY_FAIL("moe_route_table: a table of experts needs token ids and a vocabulary");
+    if (experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0) SPY_FAIL("moe_route_table: %d experts (at most %d), top %d", experts, MOE_MAX_EXPERTS, top);
+    SPY_CUDA(cudaMemsetAsync(counts, 0, sizeof(int) * experts, stream));
+    const long long pairs = (long long)tokens * top;
+    const int blocks = (int)min((pairs + 255) / 256, (long long)4 * 148);
+    spy_launch_in_order(moe_table_kernel, dim3(blocks), dim3(256), (size_t)experts * sizeof(int), stream, table, ids, vocab, pairs, experts, top, choice, choice_w,
+                        slot, counts);
+    SPY_CHECK_LAUNCH("moe_table");
     spy_launch(moe_slots_kernel, dim3(experts), dim3(1024), 0, stream, (const int*)choice, (const float*)choice_w, (const int*)counts,
                tokens * top, top, experts, offsets, slot, row_token, row_w, pad < 1 ? 1 : pad, tile_expert, pad > 1 ? num_rows / pad : 0);
     SPY_CHECK_LAUNCH("moe_slots");

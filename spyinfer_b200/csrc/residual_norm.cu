@@ -252,3 +252,81 @@ extern "C" int spy_normed_sum(float* out, const void* a, int a_dtype, int a_spli
     SPY_CHECK_LAUNCH("normed_sum");
     return 0;
 }
+
+template <int V, typename T>
+__device__ __forceinline__ void sum_load(const T* p, float (&v)[V])
+{
+    if constexpr (V == 4) Quad<T>::load(p, v);
+    else v[0] = to_f32(*p);
+}
+template <int V, typename T>
+__device__ __forceinline__ void sum_store(T* p, const float (&v)[V])
+{
+    if constexpr (V == 4) Quad<T>::store(p, v);
+    else *p = from_f32<T>(v[0]);
+}
+
+// hidden += a (+ b), each a result [rows, len] or a stack of split-K partial sums, and (optionally) the sum's copy in the type the
+// next product reads: what a block does whose two sublayers read one norm.  V elements a thread.
+template <typename TA, typename TB, typename TC, int V>
+__global__ void __launch_bounds__(256)
+stream_sum_kernel(float* __restrict__ hidden, const TA* __restrict__ a, int a_splits, long long a_stride, const TB* __restrict__ b, int b_splits,
+                  long long b_stride, TC* __restrict__ copy, long long n)
+{
+    pdl_enter();
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= n) return;
+    float h[V];
+    sum_load<V>(hidden + i, h);
+    float t[V], u[V];
+    sum_load<V>(a + i, t);
+#pragma unroll 4
+    for (int s = 1; s < a_splits; ++s) {
+        sum_load<V>(a + s * a_stride + i, u);
+#pragma unroll
+        for (int e = 0; e < V; ++e) t[e] += u[e];
+    }
+    if (b != nullptr) {
+        float w[V];
+        sum_load<V>(b + i, w);
+#pragma unroll 4
+        for (int s = 1; s < b_splits; ++s) {
+            sum_load<V>(b + s * b_stride + i, u);
+#pragma unroll
+            for (int e = 0; e < V; ++e) w[e] += u[e];
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) t[e] += w[e];
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) h[e] += t[e];
+    sum_store<V>(hidden + i, h);
+    if (copy != nullptr) sum_store<V>(copy + i, h);
+}
+
+extern "C" int spy_stream_sum(float* hidden, const void* a, int a_dtype, int a_splits, long long a_stride, const void* b, int b_dtype, int b_splits,
+                              long long b_stride, void* copy, int copy_dtype, long long n, cudaStream_t stream)
+{
+    if (n <= 0) return 0;
+    if (hidden == nullptr || a == nullptr || a_splits < 1 || (b != nullptr && b_splits < 1)) SPY_FAIL("stream_sum: a stream and a result are needed");
+    if (b == nullptr) b_dtype = SPY_F32;
+    if (copy == nullptr) copy_dtype = SPY_BF16;
+    auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const bool vec = n % 4 == 0 && a_stride % 4 == 0 && b_stride % 4 == 0 && aligned(hidden) && aligned(a) && aligned(b) && aligned(copy);
+    const long long blocks = (n / (vec ? 4 : 1) + 255) / 256;
+    if (blocks > 0x7fffffffLL) SPY_FAIL("stream_sum: %lld elements exceed the grid", n);
+    SPY_DISPATCH_DTYPE(a_dtype, TA, {
+        SPY_DISPATCH_DTYPE(b_dtype, TB, {
+            SPY_DISPATCH_DTYPE(copy_dtype, TC, {
+                if (vec)
+                    spy_launch(stream_sum_kernel<TA, TB, TC, 4>, dim3((unsigned)blocks), dim3(256), 0, stream, hidden, (const TA*)a, a_splits, a_stride, (const TB*)b,
+                               b_splits, b_stride, (TC*)copy, n);
+                else
+                    spy_launch(stream_sum_kernel<TA, TB, TC, 1>, dim3((unsigned)blocks), dim3(256), 0, stream, hidden, (const TA*)a, a_splits, a_stride, (const TB*)b,
+                               b_splits, b_stride, (TC*)copy, n);
+            })
+        })
+    })
+    SPY_CHECK_LAUNCH("stream_sum");
+    return 0;
+}

@@ -59,6 +59,15 @@ class Model:
         self.stream_products: Dict[str, Optional[Linear]] = {e.before.tensor: None for e in spec.run_order if isinstance(e.before, StreamProject)}
         if self.stream_products and getattr(self.embedding, "pairs", None) is not None:
             raise ValueError("run order: a projection of the stream and the embedding output needs an embedding that is a table's row")
+        # tensors that several parts read, declared and bound once
+        self.shared: Dict[str, WeightDecl] = {}
+        for part in self.parts():
+            for d in part.shared_decls():
+                if self.shared.setdefault(d.name, d) != d:
+                    raise ValueError(f"the parts that share the tensor {d.name!r} do not agree on its shape")
+
+    def parts(self) -> List:
+        return [self.embedding, self.final_norm, self.head] + [p for l in self.layers for p in l.parts()]
 
     # ---- weights ---------------------------------------------------------------------------
     def weight_decls(self) -> List[WeightDecl]:
@@ -66,6 +75,7 @@ class Model:
         for layer in self.layers:
             for part in layer.parts():
                 decls += _prefixed(part, layer.prefix)
+        decls += list(self.shared.values())
         decls += [WeightDecl(name, (rows, self.spec.hidden_size)) for name, rows in self.stream_rows.items()]
         decls += [WeightDecl(name, (self.spec.hidden_size, 2 * self.spec.hidden_size)) for name in self.stream_products]
         decls += _prefixed(self.final_norm, "") + _prefixed(self.head, "")
@@ -87,6 +97,11 @@ class Model:
         for layer in self.layers:
             for part in layer.parts():
                 part.bind(sub(part, layer.prefix))
+        shared = {name: tensors[name] for name in self.shared}
+        for part in self.parts():
+            wanted = part.shared_decls()
+            if wanted:
+                part.bind_shared({d.name: shared[d.name] for d in wanted})
         self.stream_tensors = {name: tensors[name] for name in self.stream_rows}
         for name in self.stream_products:
             self.stream_products[name] = Linear(tensors[name], self.ctx.dtype)
@@ -125,7 +140,7 @@ class Model:
 
     def kernel_modules(self) -> List[str]:
         mods: List[str] = []
-        for part in [self.embedding, self.final_norm, self.head] + [p for l in self.layers for p in l.parts()]:
+        for part in self.parts():
             mods += part.modules()
         for layer in self.layers:
             mods += list(getattr(layer.block, "kernel_modules", ()))
@@ -137,7 +152,7 @@ class Model:
 
     def graph_safe(self) -> bool:
         """Every part and every block arrangement says that its launches do not depend on a batch's content."""
-        parts = [self.embedding, self.final_norm, self.head] + [p for l in self.layers for p in l.parts()]
+        parts = self.parts()
         nested = [p.position for p in parts if getattr(p, "position", None) is not None]
         return all(p.graph_safe for p in parts + nested) and all(l.block.graph_safe for l in self.layers)
 

@@ -348,13 +348,28 @@ def qk_rope_store(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim
     return q_out
 
 
+def _score_args(tokens: int, num_heads: int, softcap: float, slopes: Optional[torch.Tensor], sinks: Optional[torch.Tensor], out_scale: Optional[torch.Tensor]):
+    """What the attention kernels do with a layer's scores and results beside scaling them (all optional, float32):
+    ``softcap``: ``s = cap * tanh(s / cap)``; then ``slopes [heads]``: ``s -= slopes[h] * (i - j)`` for a query at ``i`` and a key at ``j``;
+    ``sinks [heads]``: the softmax's denominator also holds ``exp(sinks[h])``; ``out_scale [T, heads]``: a factor on every head's result."""
+    if softcap < 0.0:
+        raise KernelError(f"attention: the cap on the scores {softcap} must not be negative")
+    for t, what, shape in ((slopes, "distance slopes", (num_heads,)), (sinks, "sinks", (num_heads,)), (out_scale, "result scale", (tokens, num_heads))):
+        if t is not None:
+            _check(t, what, torch.float32, len(shape))
+            if tuple(t.shape) != shape:
+                raise KernelError(f"attention: {what} {tuple(t.shape)} do not fit {shape}")
+    return ctypes.c_float(softcap), _ptr(slopes), _ptr(sinks), _ptr(out_scale)
+
+
 def attention_generic(q: torch.Tensor, num_heads: int, head_dim: int, out: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor,
                       positions: torch.Tensor, seq_of_token: torch.Tensor, scale: float, window: Optional[int] = None,
-                      status: Optional[torch.Tensor] = None, keep_first: int = 0, sink: bool = False) -> torch.Tensor:
+                      status: Optional[torch.Tensor] = None, keep_first: int = 0, sink: bool = False, softcap: float = 0.0,
+                      slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, out_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of every token of the batch over its sequence's pages (any mix of prompt
     portions and single tokens).  ``q [T, >= nh*hd]`` (only the first nh*hd columns are read),
     ``out [T, nh*hd]``.  ``keep_first`` (with a window): the sequence's first so many keys stay visible;
-    ``sink``: one is added to the softmax's denominator."""
+    ``sink``: one is added to the softmax's denominator.  ``softcap``, ``slopes``, ``sinks``, ``out_scale``: see ``_score_args``."""
     _check(q, "attention queries", ndim=2)
     _check(out, "attention output", q.dtype, 2)
     _check(pages, "cache pages", ndim=5)
@@ -372,7 +387,7 @@ def attention_generic(q: torch.Tensor, num_heads: int, head_dim: int, out: torch
     _call("attention_generic", "spy_attention_generic", _ptr(q), ctypes.c_longlong(q.shape[1]), _ptr(out), _code(q, "attention queries"),
           _ptr(pages), _code(pages, "cache pages"), _ptr(block_table), block_table.shape[1], page_size, num_pages, num_heads, nkv, head_dim,
           _ptr(positions), _ptr(seq_of_token), T, int(window or 0), ctypes.c_float(scale), _ptr(status), _stream(), planes, int(keep_first),
-          int(bool(sink)))
+          int(bool(sink)), *_score_args(T, num_heads, softcap, slopes, sinks, out_scale))
     return out
 
 
@@ -700,11 +715,14 @@ def attention_mma(q: torch.Tensor, num_heads: int, head_dim: int, out: torch.Ten
 
 def attention_tc(q: torch.Tensor, num_heads: int, head_dim: int, out: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor,
                  positions: torch.Tensor, q_start: torch.Tensor, num_seqs: int, scale: float, window: Optional[int] = None,
-                 status: Optional[torch.Tensor] = None, lse: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 status: Optional[torch.Tensor] = None, lse: Optional[torch.Tensor] = None,
+                 softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
+                 out_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of a batch over its pages on tcgen05 (blocks of two 128-row query tiles that share
     every key and value tile, scores and output in tensor memory, pages brought in by TMA): prompt
     portions, any mix.  Page sizes 8 .. 128.  ``lse [T, nh]`` (float32, optional) receives the natural
-    logarithm of every row's sum of ``exp(score * scale)``, with which further keys can be merged in."""
+    logarithm of every row's sum of ``exp(score * scale)``, with which further keys can be merged in (not
+    together with the options of ``_score_args``: ``softcap``, ``slopes``, ``sinks``, ``out_scale``)."""
     _check(q, "attention queries", torch.bfloat16, 2)
     _check(out, "attention output", torch.bfloat16, 2)
     _check(pages, "cache pages", torch.bfloat16, 5)
@@ -722,12 +740,20 @@ def attention_tc(q: torch.Tensor, num_heads: int, head_dim: int, out: torch.Tens
     if status is None:
         status = status_word(q.device)
     if lse is not None:
+        if softcap or slopes is not None or sinks is not None or out_scale is not None:
+            raise KernelError("attention: no logarithms of the sums for scores with a cap, a bias, sinks or a scale of the result")
         _check(lse, "logarithms of the sums", torch.float32, 2)
         if tuple(lse.shape) != (T, num_heads):
             raise KernelError(f"attention: lse {tuple(lse.shape)} does not fit {T} tokens of {num_heads} heads")
         _call("attention_tc", "spy_attention_tc_lse", _ptr(q), ctypes.c_longlong(q.shape[1]), _ptr(out), _ptr(lse), _ptr(pages), _ptr(block_table),
               block_table.shape[1], page_size, num_pages, num_heads, nkv, head_dim, _ptr(positions), _ptr(q_start), T, num_seqs,
               int(window or 0), ctypes.c_float(scale), _ptr(status), _stream(), planes)
+        return out
+    if softcap or slopes is not None or sinks is not None or out_scale is not None:
+        _call("attention_tc", "spy_attention_tc_scores", _ptr(q), ctypes.c_longlong(q.shape[1]), _ptr(out), _ptr(pages), _ptr(block_table),
+              block_table.shape[1], page_size, num_pages, num_heads, nkv, head_dim, _ptr(positions), _ptr(q_start), T, num_seqs,
+              int(window or 0), ctypes.c_float(scale), _ptr(status), _stream(), planes,
+              *_score_args(T, num_heads, softcap, slopes, sinks, out_scale))
         return out
     _call("attention_tc", "spy_attention_tc", _ptr(q), ctypes.c_longlong(q.shape[1]), _ptr(out), _ptr(pages), _ptr(block_table),
           block_table.shape[1], page_size, num_pages, num_heads, nkv, head_dim, _ptr(positions), _ptr(q_start), T, num_seqs,
@@ -759,7 +785,9 @@ def attention_decode_takes(num_heads: int, num_kv_heads: int, head_dim: int, pag
 
 def attention_decode(q: torch.Tensor, num_heads: int, head_dim: int, out: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor,
                      positions: torch.Tensor, q_start: torch.Tensor, num_seqs: int, scale: float, window: Optional[int] = None,
-                     status: Optional[torch.Tensor] = None, share: str = "auto", lse: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     status: Optional[torch.Tensor] = None, share: str = "auto", lse: Optional[torch.Tensor] = None,
+                     softcap: float = 0.0, slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
+                     out_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of a decoding batch (one token per sequence) over its pages: one persistent block
     per SM, keys in the rows of tcgen05 tiles, pages brought in by TMA, the batch's tiles shared out
     evenly over the blocks and merged through scratch memory.  At most 1024 sequences.  ``positions``,
@@ -768,7 +796,8 @@ def attention_decode(q: torch.Tensor, num_heads: int, head_dim: int, out: torch.
     on different streams must not overlap (they share the counters of the merge).  ``share``: how
     the work is dealt out, "auto" (the kernel decides), "split" (tiles split evenly, merged) or
     "whole" ((sequence, kv head) pairs whole).  ``lse [T, nh]`` (float32, optional) receives, at every sequence's token, the
-    natural logarithm of each head's sum of ``exp(score * scale)``, with which further keys can be merged in."""
+    natural logarithm of each head's sum of ``exp(score * scale)``, with which further keys can be merged in (not
+    together with the options of ``_score_args``: ``softcap``, ``slopes``, ``sinks``, ``out_scale``)."""
     if share not in ("auto", "split", "whole"):
         raise KernelError(f"attention_decode: share {share!r} is not 'auto', 'split' or 'whole'")
     _check(q, "attention queries", torch.bfloat16, 2)
@@ -792,6 +821,8 @@ def attention_decode(q: torch.Tensor, num_heads: int, head_dim: int, out: torch.
     if status is None:
         status = status_word(q.device)
     if lse is not None:
+        if softcap or slopes is not None or sinks is not None or out_scale is not None:
+            raise KernelError("attention: no logarithms of the sums for scores with a cap, a bias, sinks or a scale of the result")
         _check(lse, "logarithms of the sums", torch.float32, 2)
         if tuple(lse.shape) != (T, num_heads):
             raise KernelError(f"attention: lse {tuple(lse.shape)} does not fit {T} tokens of {num_heads} heads")
@@ -799,6 +830,13 @@ def attention_decode(q: torch.Tensor, num_heads: int, head_dim: int, out: torch.
               block_table.shape[1], page_size, num_pages, num_heads, nkv, head_dim, _ptr(positions), _ptr(q_start), T, num_seqs,
               int(window or 0), ctypes.c_float(scale), ("auto", "split", "whole").index(share), _ptr(scratch), ctypes.c_longlong(scratch.numel()),
               _ptr(status), _stream(), planes)
+        return out
+    if softcap or slopes is not None or sinks is not None or out_scale is not None:
+        _call("attention_decode", "spy_attention_decode_scores", _ptr(q), ctypes.c_longlong(q.shape[1]), _ptr(out), _ptr(pages), _ptr(block_table),
+              block_table.shape[1], page_size, num_pages, num_heads, nkv, head_dim, _ptr(positions), _ptr(q_start), T, num_seqs,
+              int(window or 0), ctypes.c_float(scale), ("auto", "split", "whole").index(share), _ptr(scratch), ctypes.c_longlong(scratch.numel()),
+              _ptr(status), _stream(), planes,
+              *_score_args(T, num_heads, softcap, slopes, sinks, out_scale))
         return out
     _call("attention_decode", "spy_attention_decode", _ptr(q), ctypes.c_longlong(q.shape[1]), _ptr(out), _ptr(pages), _ptr(block_table),
           block_table.shape[1], page_size, num_pages, num_heads, nkv, head_dim, _ptr(positions), _ptr(q_start), T, num_seqs,
@@ -933,11 +971,11 @@ def head_product(x: torch.Tensor, in_head_stride: int, weight: torch.Tensor, out
                  rope_table: Optional[torch.Tensor] = None, interleaved: bool = False, positions: Optional[torch.Tensor] = None,
                  gate: Optional[torch.Tensor] = None, gate_offset: int = 0, status: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``out[t, h * out_head_stride + n] = sum_k weight[h, k, n] * x[t, h * in_head_stride + k]`` (32-bit sums) for a weight
-    ``[heads, K, N]``; x and out ``[T, >= heads * stride]`` of one dtype.  ``tail`` elements that follow each head's K inputs go,
+    ``[heads, K, N]``; x and out ``[T, >= heads * stride]`` of one dtype, or x float32.  ``tail`` elements that follow each head's K inputs go,
     rotated by ``rope_table`` at the token's position (pairs as in ``latent_prep``), to the columns after its N results.
     ``gate`` (float32 ``[T, ld]``): the results are multiplied by ``sigmoid(gate[t, gate_offset + h * N + n])``."""
     _check(x, "head_product input", ndim=2)
-    _check(out, "head_product output", x.dtype, 2)
+    _check(out, "head_product output", x.dtype if x.dtype != torch.float32 else None, 2)
     _check(weight, "head_product weight", ndim=3)
     H, K, N = weight.shape
     T = x.shape[0]
@@ -960,8 +998,8 @@ def head_product(x: torch.Tensor, in_head_stride: int, weight: torch.Tensor, out
         gate_ld = gate.shape[1]
         if gate.shape[0] != T or gate_offset < 0 or gate_offset + H * N > gate_ld:
             raise KernelError("head_product: the gate's columns do not fit")
-    _call("latent", "spy_head_product", _ptr(x), ctypes.c_longlong(x.shape[1]), int(in_head_stride), K, _ptr(weight), _code(weight, "head_product weight"), N,
-          _ptr(out), ctypes.c_longlong(out.shape[1]), int(out_head_stride), _code(x, "head_product input"), int(tail), _ptr(rope_table), rot_half, table_rows,
+    _call("latent", "spy_head_product", _ptr(x), _code(x, "head_product input"), ctypes.c_longlong(x.shape[1]), int(in_head_stride), K, _ptr(weight),
+          _code(weight, "head_product weight"), N, _ptr(out), ctypes.c_longlong(out.shape[1]), int(out_head_stride), _code(out, "head_product output"), int(tail), _ptr(rope_table), rot_half, table_rows,
           int(bool(interleaved)), _ptr(positions), _ptr(gate), ctypes.c_longlong(gate_ld), int(gate_offset), T, H, _ptr(status), _stream())
     return out
 
@@ -1703,6 +1741,133 @@ def moe_route(logits: torch.Tensor, experts: int, top: int, has_shared: bool, pa
     return out if pad == 1 else out + (tile_expert,)
 
 
+def _check_table(table: torch.Tensor, ids: torch.Tensor, tokens: int) -> None:
+    _check(table, "table of experts", torch.int32, 2)
+    _check(ids, "token ids", torch.int32, 1)
+    if ids.shape[0] != tokens:
+        raise KernelError(f"table of experts: {ids.shape[0]} token ids for {tokens} tokens")
+
+
+def moe_activation_table(gate_up: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, experts: int, ff: int, limit: float = 0.0,
+                         shared_ff: int = 0, shared_limit: float = 0.0, alpha: float = 1.702, activation: str = "silu",
+                         shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """As ``moe_activation`` with the experts of every token named by ``table [vocab, top]`` (int32) of its id, each with the weight
+    ``1 / top``.  The shared expert's weight is one, or the sigmoid of ``shared_gate [T, 1]`` (float32)."""
+    _check(gate_up, "expert gate|up", ndim=2)
+    _check(out, "expert activations", ndim=2)
+    T, cols, top = gate_up.shape[0], experts * ff + shared_ff, table.shape[1]
+    _check_table(table, ids, T)
+    if activation not in ("clamped_swish", "silu"):
+        raise KernelError(f"moe_activation: unknown activation {activation!r}")
+    if gate_up.shape[1] != 2 * cols or tuple(out.shape) != (T, cols):
+        raise KernelError(f"moe_activation: gate|up {tuple(gate_up.shape)}, output {tuple(out.shape)} do not fit {experts} experts of {ff} and {shared_ff}")
+    if shared_gate is not None:
+        _check(shared_gate, "shared gate", torch.float32, 2)
+        if shared_gate.shape[0] != T:
+            raise KernelError("moe_activation: one shared gate a token")
+    _call("moe", "spy_moe_activation_table", _ptr(gate_up), _code(gate_up, "expert gate|up"), ctypes.c_longlong(gate_up.shape[1]), _ptr(table), _ptr(ids),
+          table.shape[0], _ptr(shared_gate), ctypes.c_longlong(shared_gate.shape[1] if shared_gate is not None else 0), _ptr(out),
+          _code(out, "expert activations"), ctypes.c_longlong(out.shape[1]), T, int(experts), int(top), int(ff), ctypes.c_float(limit), int(shared_ff),
+          ctypes.c_float(shared_limit), ctypes.c_float(alpha), 1 if activation == "silu" else 0, _stream())
+    return out
+
+
+def moe_route_table(table: torch.Tensor, ids: torch.Tensor, experts: int, pad: int = 1):
+    """As ``moe_route`` with the experts named by ``table [vocab, top]`` of the token ids, all weights ``1 / top``: ``offsets, slot,
+    row_token, row_w`` (and ``tile_expert`` with ``pad`` above 1)."""
+    _check_table(table, ids, ids.shape[0])
+    T, top = ids.shape[0], table.shape[1]
+    choice, choice_w, counts, offsets, slot, row_token, row_w, tile_expert, R = _route_buffers(T, experts, top, pad, ids.device)
+    _call("moe", "spy_moe_route_table", _ptr(table), _ptr(ids), table.shape[0], T, int(experts), int(top), _ptr(choice), _ptr(choice_w), _ptr(counts),
+          _ptr(offsets), _ptr(slot), _ptr(row_token), _ptr(row_w), _stream(), int(pad), _ptr(tile_expert), R)
+    out = (offsets, slot.view(T, top), row_token, row_w)
+    return out if pad == 1 else out + (tile_expert,)
+
+
+def stream_sum(hidden: torch.Tensor, a: torch.Tensor, b: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``hidden += a (+ b)`` in 32-bit and in place, each of hidden's shape or a stack ``[splits, T, len]`` of float32 partial sums;
+    ``copy`` (of hidden's shape) receives the sum in its own type."""
+    _check(hidden, "residual stream", torch.float32, 2)
+    pa, sa, stride_a = _stack_of(a, hidden, "first result")
+    pb, sb, stride_b = _stack_of(b, hidden, "second result")
+    if copy is not None:
+        _check(copy, "copy of the stream", ndim=2)
+        if tuple(copy.shape) != tuple(hidden.shape):
+            raise KernelError("stream_sum: the copy has another shape than the stream")
+    _call("residual_norm", "spy_stream_sum", _ptr(hidden), _ptr(pa), _code(pa, "first result"), sa, ctypes.c_longlong(stride_a if sa > 1 else 0), _ptr(pb),
+          _code(pb, "second result") if pb is not None else 0, max(sb, 1), ctypes.c_longlong(stride_b if sb > 1 else 0), _ptr(copy),
+          _code(copy, "copy of the stream") if copy is not None else 0, ctypes.c_longlong(hidden.numel()), _stream())
+    return hidden
+
+
+def token_gate(gate: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor, out: torch.Tensor, status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[t, j] = gelu_tanh(gate[t, j]) * table[ids[t], col + j]``; ``gate [T, dim]`` or a stack ``[splits, T, dim]`` of float32 partial
+    sums, ``table [vocab, >= col + dim]``, ``out [T, dim]``."""
+    _check(out, "gated token rows", ndim=2)
+    T, dim = out.shape
+    if gate.dim() == 3:
+        _check(gate, "gate parts", torch.float32, 3)
+        splits, stride = gate.shape[0], gate.shape[1] * gate.shape[2]
+    else:
+        _check(gate, "gate", ndim=2)
+        splits, stride = 1, 0
+    _check(table, "token table", ndim=2)
+    _check(ids, "token ids", torch.int32, 1)
+    if tuple(gate.shape[-2:]) != (T, dim) or ids.shape[0] != T or not 0 <= col <= table.shape[1] - dim:
+        raise KernelError(f"token_gate: gate {tuple(gate.shape)}, output {tuple(out.shape)}, column {col} of a table {tuple(table.shape)} do not fit")
+    _call("embedding", "spy_token_gate", _ptr(gate), _code(gate, "gate"), splits, ctypes.c_longlong(stride), _ptr(table), _code(table, "token table"),
+          ctypes.c_longlong(table.shape[1]), int(col), _ptr(ids), table.shape[0], _ptr(out), _code(out, "gated token rows"), T, dim, 0, _ptr(status), _stream())
+    return out
+
+
+def conv_qkv_store(proj: torch.Tensor, kernel: torch.Tensor, state: Optional[torch.Tensor], q_start: torch.Tensor, state_slot: torch.Tensor, num_seqs: int,
+                   longest: int, positions: torch.Tensor, seq_of_token: torch.Tensor, q_out: torch.Tensor, block_table: torch.Tensor, pages: torch.Tensor,
+                   heads: int, kv_heads: int, dim: int, vdim: int, temp: Optional[tuple] = None, gate_col: int = -1, gate_out: Optional[torch.Tensor] = None,
+                   status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The step ahead of the attention kernel for queries, keys and values behind a causal convolution over time.  ``proj [T, ld]`` (or a
+    stack ``[splits, T, ld]`` of float32 partial products) holds from column 0 the queries (``heads`` x ``dim``), keys (``kv_heads`` x ``dim``) and
+    values (``kv_heads`` x ``vdim``); ``kernel [taps, channels]`` float32 (its last row meets the current token); ``state [slots, (taps - 1)
+    channels]`` float32 holds the inputs ahead of each request's run and receives the run's last ones.  ``temp = (coef, every)``: queries
+    times ``1 + coef ln(floor((p + 1) / every) + 1)``.  ``gate_out [T, heads]`` float32 receives the sigmoid of ``heads`` columns from
+    ``gate_col``.  ``q_out [T, heads hd]`` and ``pages [num_pages, 2, kv_heads, page_size, hd]`` get rows of ``hd`` with zeros behind their
+    content.  ``longest``: no request brings more tokens than this."""
+    if proj.dim() == 3:
+        _check(proj, "projection parts", torch.float32, 3)
+        splits, stride = proj.shape[0], proj.shape[1] * proj.shape[2]
+    else:
+        _check(proj, "projection", ndim=2)
+        splits, stride = 1, 0
+    T, ld = proj.shape[-2:]
+    _check(kernel, "convolution kernel", torch.float32, 2)
+    _check(q_out, "queries", ndim=2)
+    _check(pages, "cache pages", q_out.dtype, 5)
+    _check(block_table, "block table", torch.int32, 2)
+    for t, what in ((positions, "positions"), (seq_of_token, "seq_of_token"), (q_start, "q_start"), (state_slot, "state_slot")):
+        _check(t, what, torch.int32, 1)
+    taps, channels = kernel.shape
+    num_pages, two, nkv, page_size, hd = pages.shape
+    if two != 2 or nkv != kv_heads or tuple(q_out.shape) != (T, heads * hd) or positions.shape[0] != T or seq_of_token.shape[0] != T:
+        raise KernelError(f"conv_qkv_store: pages {tuple(pages.shape)} / queries {tuple(q_out.shape)} do not fit {heads} heads over {kv_heads} of rows {hd}")
+    if channels != heads * dim + kv_heads * (dim + vdim) or channels > ld:
+        raise KernelError(f"conv_qkv_store: {channels} channels and {ld} columns do not fit {heads} heads over {kv_heads} of {dim} and {vdim}")
+    if q_start.shape[0] < num_seqs + 1 or state_slot.shape[0] < num_seqs or block_table.shape[0] < num_seqs:
+        raise KernelError("conv_qkv_store: q_start needs one entry per request plus one, state_slot and the block table one per request")
+    if taps > 1:
+        _check(state, "convolution state", torch.float32, 2)
+        if state.shape[1] != (taps - 1) * channels:
+            raise KernelError(f"conv_qkv_store: state {tuple(state.shape)} does not fit {taps - 1} inputs of {channels} channels")
+    if gate_out is not None:
+        _check(gate_out, "head gates", torch.float32, 2)
+        if tuple(gate_out.shape) != (T, heads) or gate_col < channels or gate_col + heads > ld:
+            raise KernelError("conv_qkv_store: the gate's columns or its output do not fit")
+    coef, every = (float(temp[0]), float(temp[1])) if temp is not None else (0.0, 0.0)
+    _call("conv_qkv", "spy_conv_qkv_store", _ptr(proj), _code(proj, "projection"), ctypes.c_longlong(ld), splits, ctypes.c_longlong(stride), _ptr(kernel), taps,
+          _ptr(state if taps > 1 else None), _ptr(q_start), _ptr(state_slot), int(num_seqs), int(longest), ctypes.c_float(coef), ctypes.c_float(every),
+          int(gate_col), _ptr(gate_out), _ptr(positions), _ptr(seq_of_token), _ptr(q_out), _code(q_out, "queries"), _ptr(block_table), block_table.shape[1],
+          _ptr(pages), page_size, num_pages, int(heads), int(kv_heads), int(dim), int(vdim), hd, _ptr(status), _stream())
+    return q_out
+
+
 def grouped_tile_rows() -> int:
     """The rows of a tile of ``gemm_grouped``: what an expert's run of rows is padded to."""
     return int(build.load("gemm_grouped").spy_gemm_grouped_tile_rows())
@@ -1738,15 +1903,16 @@ def gather_rows(x: torch.Tensor, row_token: torch.Tensor, out: torch.Tensor) -> 
     return out
 
 
-def expert_activation(gate_up: torch.Tensor, row_w: torch.Tensor, out: torch.Tensor, limit: float, alpha: float = 1.702,
+def expert_activation(gate_up: torch.Tensor, row_w: Optional[torch.Tensor], out: torch.Tensor, limit: float, alpha: float = 1.702,
                       activation: str = "clamped_swish") -> torch.Tensor:
     """``out[r] = row_w[r] * g * sigmoid(alpha g) * (u + 1)`` over rows ``[gate | up]`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``;
-    ``activation="silu"``: ``row_w[r] * silu(gate) * up`` without clamps."""
+    ``activation="silu"``: ``row_w[r] * silu(gate) * up`` without clamps.  ``row_w`` None: every row's weight is one."""
     _check(gate_up, "expert gate|up", ndim=2)
     _check(out, "expert activations", ndim=2)
-    _check(row_w, "row weights", torch.float32, 1)
+    if row_w is not None:
+        _check(row_w, "row weights", torch.float32, 1)
     R, two = gate_up.shape
-    if two % 2 or tuple(out.shape) != (R, two // 2) or row_w.shape[0] < R:
+    if two % 2 or tuple(out.shape) != (R, two // 2) or (row_w is not None and row_w.shape[0] < R):
         raise KernelError("expert_activation: shapes do not fit")
     _call("moe", "spy_expert_activation", _ptr(gate_up), _code(gate_up, "expert gate|up"), ctypes.c_longlong(two), _ptr(row_w), _ptr(out),
           _code(out, "expert activations"), ctypes.c_longlong(two // 2), R, two // 2, ctypes.c_float(limit), ctypes.c_float(alpha), _stream(),

@@ -15,7 +15,7 @@ import math
 import torch
 
 from .. import kernels
-from ..config.spec import CompositeCacheNeed, PagedCacheNeed
+from ..config.spec import CompositeCacheNeed, PagedCacheNeed, StateCacheNeed
 from ..weights.loader import WeightDecl
 from .base import Mixer
 from .linear import Linear
@@ -28,7 +28,12 @@ class Attention(Mixer):
     (None: no q/k norm), ``position`` (a PartSpec or None), ``window`` (None: all keys),
     ``chunk`` (None, or a size: a query sees the earlier keys of its own block of that many positions only, blocks counted
     from position 0 of the sequence; not together with a window), ``scale`` (None: 1/sqrt(head_dim)), ``prefix``,
-    ``qkv_bias`` and ``o_bias`` (default false: the projections have bias tensors ``{q,k,v}_proj.bias`` / ``o_proj.bias``)."""
+    ``qkv_bias`` and ``o_bias`` (default false: the projections have bias tensors ``{q,k,v}_proj.bias`` / ``o_proj.bias``).
+
+    What a layer may do with its scores, inside the attention kernels and in 32-bit: ``softcap`` (0 or None: none; else
+    ``s = cap * tanh(s / cap)``), ``distance_bias`` (default false; else ``s -= 2^(-8 (h + 1) / heads) * (i - j)`` behind the cap) and
+    ``learned_sink`` (default false; else the tensor ``sink [heads]``: the softmax's denominator also holds ``exp(sink)``, which is
+    neither scaled, capped nor biased)."""
 
     graph_safe = True
     #: False: the head size must be a multiple of 4 (the kernel that rotates and stores q, k and v reads quads)
@@ -55,6 +60,11 @@ class Attention(Mixer):
         pos = params.get("position")
         self.position = build_part(pos, ctx) if pos is not None else None
         self.qkv = self.o = self.q_norm = self.k_norm = self.rope_table = None
+        self.softcap = float(params.get("softcap") or 0.0)
+        if self.softcap < 0.0:
+            raise ValueError(f"attention: the cap on the scores {self.softcap} must not be negative")
+        self.distance_bias, self.learned_sink = bool(params.get("distance_bias", False)), bool(params.get("learned_sink", False))
+        self.slopes = self.sinks = None
         # which attention kernels take these sizes (the page size, known at the first step, decides between them)
         self.tc = kernels.attention_tc_takes(self.nh, self.nkv, self.hd, ctx.dtype)        # tcgen05, pages that are one TMA box
         self.mma = kernels.attention_mma_takes(self.nh, self.nkv, self.hd, ctx.dtype)      # mma.sync, any page size
@@ -71,7 +81,7 @@ class Attention(Mixer):
             decls += [WeightDecl(p + "q_proj.bias", (nh * hd,)), WeightDecl(p + "k_proj.bias", (nkv * hd,)), WeightDecl(p + "v_proj.bias", (nkv * hd,))]
         if self.o_bias:
             decls += [WeightDecl(p + "o_proj.bias", (H,))]
-        return decls
+        return decls + self.sink_decls()
 
     def bind(self, tensors):
         p = self.prefix
@@ -87,6 +97,7 @@ class Attention(Mixer):
             self.q_norm, self.k_norm = tensors[p + "q_norm.weight"], tensors[p + "k_norm.weight"]
             if self.q_norm.dtype != self.k_norm.dtype:
                 self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
+        self.bind_scores(tensors)
 
     def modules(self):
         mods = ["qk_rope_store"] + (["attention_tc", "attention_decode"] if self.tc else []) + (["attention_mma"] if self.mma else ["attention_generic"]) + self.qkv.modules() + self.o.modules()
@@ -104,6 +115,22 @@ class Attention(Mixer):
     def key_mask(self):
         """What the attention kernels take as ``window``: None (every earlier key), the window, or minus the chunk size."""
         return -int(self.chunk) if self.chunk is not None else self.window
+
+    def sink_decls(self):
+        return [WeightDecl(self.prefix + "sink", (self.nh,))] if self.learned_sink else []
+
+    def bind_scores(self, tensors):
+        """The slopes and sinks that the kernels read (float32)."""
+        if self.distance_bias:
+            self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / self.nh) for h in range(self.nh)], dtype=torch.float64).to(torch.float32).to(self.ctx.device)
+        if self.learned_sink:
+            self.sinks = tensors[self.prefix + "sink"].float().contiguous()
+
+    def score_options(self, out_scale=None):
+        """What the attention kernels are told beside the scale; ``out_scale [T, heads]`` float32: a factor on every head's result."""
+        if not self.softcap and self.slopes is None and self.sinks is None and out_scale is None:
+            return {}
+        return {"softcap": self.softcap, "slopes": self.slopes, "sinks": self.sinks, "out_scale": out_scale}
 
     def split_plan(self, num_seqs: int):
         """(split_keys, max_splits) for decoding ``num_seqs`` requests: the keys of every request
@@ -143,18 +170,20 @@ class Attention(Mixer):
         self.attend(q, out, batch, cache)
         return self.o(out, defer=self.defer_output)
 
-    def attend(self, q, out, batch, cache):
+    def attend(self, q, out, batch, cache, out_scale=None):
         """The attention itself, ``q [T, >= nh hd]`` over the cache into ``out [T, nh hd]``, on the kernel that the sizes, the
         page size and the kind of batch call for."""
         x = q
+        options = self.score_options(out_scale)
+        mma = self.mma and not options
         decoding = batch.one_token_each         # every request brings one token
         boxes = self.tc and cache.page_size in kernels.ATTENTION_TMA_PAGE_SIZES        # a page is one TMA box
         if (boxes and decoding and batch.num_seqs <= kernels.ATTENTION_DECODE_MAX_SEQS and batch.num_seqs * self.nkv <= kernels.ATTENTION_DECODE_MAX_PAIRS
                 and kernels.attention_decode_takes(self.nh, self.nkv, self.hd, cache.page_size, x.dtype)):
             # memory-bound: one persistent block per SM, the batch's key tiles shared out evenly, pages by TMA
             kernels.attention_decode(q, self.nh, self.hd, out, cache.pages, cache.block_table, batch.positions, batch.q_start,
-                                     batch.num_seqs, self.scale, window=self.key_mask, status=batch.status)
-        elif decoding and self.mma:
+                                     batch.num_seqs, self.scale, window=self.key_mask, status=batch.status, **options)
+        elif decoding and mma:
             # page sizes that are no TMA box, or very many requests: keys split across blocks by a plan per batch size
             split_keys, max_splits = self.split_plan(batch.num_seqs)
             kernels.attention_mma(q, self.nh, self.hd, out, cache.pages, cache.block_table, batch.positions, batch.q_start,
@@ -169,16 +198,16 @@ class Attention(Mixer):
                 head = 0
             if head:
                 kernels.attention_decode(q, self.nh, self.hd, out, cache.pages, cache.block_table[:head], batch.positions, batch.q_start[:head + 1],
-                                         head, self.scale, window=self.key_mask, status=batch.status)
+                                         head, self.scale, window=self.key_mask, status=batch.status, **options)
             kernels.attention_tc(q, self.nh, self.hd, out, cache.pages, cache.block_table[head:], batch.positions, batch.q_start[head:],
-                                 batch.num_seqs - head, self.scale, window=self.key_mask, status=batch.status)
-        elif self.mma:
+                                 batch.num_seqs - head, self.scale, window=self.key_mask, status=batch.status, **options)
+        elif mma:
             kernels.attention_mma(q, self.nh, self.hd, out, cache.pages, cache.block_table, batch.positions, batch.q_start,
                                   batch.num_seqs, self.scale, window=self.key_mask, status=batch.status)
         else:
             # the float32 path, head sizes above 128 or no multiple of 8, more than 16 query heads a key/value head
             kernels.attention_generic(q, self.nh, self.hd, out, cache.pages, cache.block_table, batch.positions, batch.seq_of_token,
-                                      self.scale, window=self.key_mask, status=batch.status)
+                                      self.scale, window=self.key_mask, status=batch.status, **options)
         return out
 
 
@@ -289,28 +318,29 @@ class PooledWindowAttention(Attention):
 @register_part("latent_attention")
 class LatentAttention(Attention):
     """Softmax attention whose keys and values are per-head projections of one small latent per token, which is all the
-    cache keeps beside one rotated key part that the heads share; the queries go through a latent of their own.
+    cache keeps beside one rotated key part that the heads share; the queries go through a latent of their own, or are projected
+    from the input.
 
-    With ``h`` the input: ``c_q = rms_norm(W_dq h)``, ``q = W_uq c_q`` laid out head by head as ``[dim | rot_dim]``;
+    With ``h`` the input: ``c_q = rms_norm(W_dq h)``, ``q = W_uq c_q`` (or ``q = W_q h``) laid out head by head as ``[dim | rot_dim]``;
     ``W_dkv h = [kv_rank | rot_dim]``, ``c = rms_norm`` of the first part, ``k_r`` the rotated second part; per head
     ``score = (q_n . U_k c + rot(q_r) . k_r) * scale``, ``o = U_v (sum p c)``; optionally ``o * sigmoid(W_g h)``; then ``W_o``.
     It is computed in the absorbed form, ``(U_k^T q_n) . c``, so the attention runs over one key/value head of size
     ``kv_rank + rot_dim`` on a cache of one plane (the value is the key row's first ``kv_rank`` elements) with the kernels
     of ``attention``; see ``csrc/latent.cu``.
 
-    params: ``hidden_size``, ``num_heads``, ``head_dim`` (the unrotated part), ``rot_dim``, ``v_head_dim``, ``q_rank``,
-    ``kv_rank``, ``eps`` (of the two latent norms), ``scale``, ``window`` (None: every earlier key), ``position`` (a rotary
+    params: ``hidden_size``, ``num_heads``, ``head_dim`` (the unrotated part), ``rot_dim``, ``v_head_dim``, ``q_rank`` (None: no
+    query latent), ``kv_rank``, ``eps`` (of the two latent norms), ``scale``, ``window`` (None: every earlier key), ``position`` (a rotary
     part whose ``rotary_dim`` is at most ``rot_dim``, or None), ``gate`` (default false), ``shares_cache`` (true: the layer
-    has no ``W_dkv`` and reads the cache of the run-order entry that its ``RunEntry.cache_of`` names), ``prefix``.  Tensors:
-    ``dq``, ``dq.norm``, ``uq``, ``dkv``, ``dkv.norm``, ``uk``, ``uv``, ``g``, ``o``."""
+    has no ``W_dkv`` and reads the cache of the run-order entry that its ``RunEntry.cache_of`` names), ``learned_sink`` (as
+    ``attention``), ``prefix``.  Tensors: ``dq``, ``dq.norm``, ``uq`` (or ``q``), ``dkv``, ``dkv.norm``, ``uk``, ``uv``, ``g``, ``o``."""
 
     graph_safe = True
     any_head_dim = True
 
     def __init__(self, params, ctx):
         self.d, self.rd, self.vd = int(params["head_dim"]), int(params["rot_dim"]), int(params["v_head_dim"])
-        self.q_rank, self.kv_rank = int(params["q_rank"]), int(params["kv_rank"])
-        if min(self.d, self.vd, self.q_rank, self.kv_rank) <= 0 or self.rd < 0:
+        self.q_rank, self.kv_rank = int(params["q_rank"]) if params.get("q_rank") is not None else None, int(params["kv_rank"])
+        if min(self.d, self.vd, self.kv_rank) <= 0 or self.rd < 0 or (self.q_rank is not None and self.q_rank <= 0):
             raise ValueError("latent_attention: sizes must be positive")
         base = dict(params)
         base.update(num_kv_heads=1, head_dim=self.kv_rank + self.rd, qk_norm_eps=None)
@@ -325,43 +355,51 @@ class LatentAttention(Attention):
         if self.position is not None and 2 * (self.position.rotary_dim // 2) > self.rd:
             raise ValueError(f"latent_attention: a rotation of {self.position.rotary_dim} elements exceeds the rotated part of {self.rd}")
         self.width = self.kv_rank + self.rd      # a cache row, and a head of the absorbed query
-        self.c_offset = self.q_rank
-        self.gate_offset = self.q_rank + (0 if self.shares_cache else self.width)
+        # the columns of the fused projection: the query latent, or the queries themselves; the key/value latent; the gate
+        self.c_offset = self.q_rank if self.q_rank is not None else self.nh * (self.d + self.rd)
+        self.gate_offset = self.c_offset + (0 if self.shares_cache else self.width)
         self.fused = self.uq = self.uk = self.uv = self.q_norm_w = self.c_norm_w = None
 
     def weight_decls(self):
         p, H, W = self.prefix, self.nh, self.hidden
-        decls = [WeightDecl(p + "dq", (self.q_rank, W)), WeightDecl(p + "dq.norm", (self.q_rank,), init="one_plus_normal"),
-                 WeightDecl(p + "uq", (H * (self.d + self.rd), self.q_rank))]
+        if self.q_rank is None:
+            decls = [WeightDecl(p + "q", (H * (self.d + self.rd), W))]
+        else:
+            decls = [WeightDecl(p + "dq", (self.q_rank, W)), WeightDecl(p + "dq.norm", (self.q_rank,), init="one_plus_normal"),
+                     WeightDecl(p + "uq", (H * (self.d + self.rd), self.q_rank))]
         if not self.shares_cache:
             decls += [WeightDecl(p + "dkv", (self.width, W)), WeightDecl(p + "dkv.norm", (self.kv_rank,), init="one_plus_normal")]
         decls += [WeightDecl(p + "uk", (H * self.d, self.kv_rank)), WeightDecl(p + "uv", (H * self.vd, self.kv_rank))]
         if self.gated:
             decls.append(WeightDecl(p + "g", (H * self.vd, W)))
-        return decls + [WeightDecl(p + "o", (W, H * self.vd))]
+        return decls + self.sink_decls() + [WeightDecl(p + "o", (W, H * self.vd))]
 
     def bind(self, tensors):
         p, H = self.prefix, self.nh
-        rows = [tensors[p + "dq"]] + ([] if self.shares_cache else [tensors[p + "dkv"]]) + ([tensors[p + "g"]] if self.gated else [])
+        rows = [tensors[p + ("dq" if self.q_rank is not None else "q")]] + ([] if self.shares_cache else [tensors[p + "dkv"]]) + ([tensors[p + "g"]] if self.gated else [])
         if len({t.dtype for t in rows}) > 1:
             rows = [t.float() for t in rows]
         self.fused = Linear(torch.cat(rows, dim=0).contiguous(), self.ctx.dtype)
-        self.uq = Linear(tensors[p + "uq"], self.ctx.dtype)
+        if self.q_rank is not None:
+            self.uq = Linear(tensors[p + "uq"], self.ctx.dtype)
+            self.q_norm_w = tensors[p + "dq.norm"].float().contiguous()
+        self.bind_scores(tensors)
         self.o = Linear(tensors[p + "o"], self.ctx.dtype)
         self.uk = tensors[p + "uk"].reshape(H, self.d, self.kv_rank).contiguous()                      # [head][unrotated element][latent]: as stored
         self.uv = tensors[p + "uv"].reshape(H, self.vd, self.kv_rank).transpose(1, 2).contiguous()     # [head][latent][value element]
-        self.q_norm_w = tensors[p + "dq.norm"].float().contiguous()
         if not self.shares_cache:
             self.c_norm_w = tensors[p + "dkv.norm"].float().contiguous()
 
     def modules(self):
-        mods = ["latent"] + (["attention_tc", "attention_decode"] if self.tc else []) + ["attention_generic"] + self.fused.modules() + self.uq.modules() + self.o.modules()
+        mods = ["latent"] + (["attention_tc", "attention_decode"] if self.tc else []) + ["attention_generic"]
+        for lin in self.linears():
+            mods += lin.modules()
         if self.position is not None:
             mods += self.position.modules()
         return mods
 
     def linears(self):
-        return [self.fused, self.uq, self.o]
+        return [self.fused] + ([self.uq] if self.uq is not None else []) + [self.o]
 
     def cache_need(self):
         return PagedCacheNeed(1, self.width, int(self.window) if self.window is not None else None, planes=1)
@@ -374,10 +412,11 @@ class LatentAttention(Attention):
         T, H = x.shape[0], self.nh
         interleaved = self.position is not None and self.position.pairing == "interleaved"
         fused = self.fused(x, out_dtype=torch.float32)
-        cq = torch.empty((T, self.q_rank), dtype=x.dtype, device=x.device)
-        kernels.latent_prep(fused, 0, self.q_rank, self.q_norm_w, cq, self.c_offset if cache.writes else -1, self.kv_rank, self.c_norm_w, self.rd,
-                            self.rope_table, interleaved, batch.positions, batch.seq_of_token, cache.block_table, cache.pages, self.eps, status=batch.status)
-        q = self.uq(cq)
+        cq = torch.empty((T, self.q_rank), dtype=x.dtype, device=x.device) if self.q_rank is not None else None
+        if cq is not None or cache.writes:
+            kernels.latent_prep(fused, 0, self.q_rank or 0, self.q_norm_w, cq, self.c_offset if cache.writes else -1, self.kv_rank, self.c_norm_w, self.rd,
+                                self.rope_table, interleaved, batch.positions, batch.seq_of_token, cache.block_table, cache.pages, self.eps, status=batch.status)
+        q = self.uq(cq) if cq is not None else fused          # without a query latent the queries are the projection's first columns
         q_abs = torch.empty((T, H * self.width), dtype=x.dtype, device=x.device)
         kernels.head_product(q, self.d + self.rd, self.uk, q_abs, self.width, tail=self.rd, rope_table=self.rope_table, interleaved=interleaved,
                              positions=batch.positions, status=batch.status)
@@ -485,7 +524,7 @@ class KeptWindowAttention(Attention):
     denominator).  The attention kernels see rows of ``max(dim, vdim)`` rounded up to 8 (zeros behind a row's content).  On the
     bfloat16 path the window's keys run on the tensor-core kernels of ``attention``, which leave each row's logarithm of its sum of
     exponentials where something is to be merged in, and ``sink_merge`` adds the kept first keys and the sink; the plain kernel
-    does all of it in one pass.
+    does all of it in one pass (and is the one that takes kept keys together with ``softcap``, ``distance_bias`` or ``learned_sink``).
 
     params: ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale`` (None: ``dim^(-1/2)``), ``window``, ``keep_first`` (default 0), ``sink``,
     ``position`` and what ``attention`` takes beside them."""
@@ -519,23 +558,23 @@ class KeptWindowAttention(Attention):
     def attention_modules(self):
         return ["attention_generic"] + (["attention_tc", "attention_decode"] if self.tc else []) + (["sink_attention"] if self.sink or self.keep_first else [])
 
-    def attend(self, q, out, batch, cache):
-        if not (self.tc and cache.page_size in kernels.ATTENTION_TMA_PAGE_SIZES):
+    def attend(self, q, out, batch, cache, out_scale=None):
+        options, merges = self.score_options(out_scale), self.sink or self.keep_first > 0
+        if not (self.tc and cache.page_size in kernels.ATTENTION_TMA_PAGE_SIZES) or (options and merges):
             # the float32 path, and sizes or pages that the tensor-core kernels do not take: everything in one plain kernel
             return kernels.attention_generic(q, self.nh, self.hd, out, cache.pages, cache.block_table, batch.positions, batch.seq_of_token, self.scale,
-                                             window=self.window, status=batch.status, keep_first=self.keep_first, sink=self.sink)
+                                             window=self.window, status=batch.status, keep_first=self.keep_first, sink=self.sink, **options)
         head = batch.num_seqs if batch.one_token_each else batch.one_token_head
         if not (0 < head <= kernels.ATTENTION_DECODE_MAX_SEQS and head * self.nkv <= kernels.ATTENTION_DECODE_MAX_PAIRS
                 and kernels.attention_decode_takes(self.nh, self.nkv, self.hd, cache.page_size, q.dtype)):
             head = 0
-        merges = self.sink or self.keep_first > 0
         lse = torch.empty((q.shape[0], self.nh), dtype=torch.float32, device=q.device) if merges else None
         if head:
             kernels.attention_decode(q, self.nh, self.hd, out, cache.pages, cache.block_table[:head], batch.positions, batch.q_start[:head + 1], head,
-                                     self.scale, window=self.window, status=batch.status, lse=lse)
+                                     self.scale, window=self.window, status=batch.status, lse=lse, **options)
         if head < batch.num_seqs:
             kernels.attention_tc(q, self.nh, self.hd, out, cache.pages, cache.block_table[head:], batch.positions, batch.q_start[head:],
-                                 batch.num_seqs - head, self.scale, window=self.window, status=batch.status, lse=lse)
+                                 batch.num_seqs - head, self.scale, window=self.window, status=batch.status, lse=lse, **options)
         if merges:
             kernels.sink_merge(q, self.nh, self.hd, out, lse, cache.pages, cache.block_table, batch.positions, batch.seq_of_token, self.scale,
                                self.window, self.keep_first, self.sink, status=batch.status)
@@ -693,4 +732,80 @@ class GatedWindowAttention(KeptWindowAttention):
         if self.gated:
             rows = out if self.hd == self.vd else torch.empty((T, self.heads * self.vd), dtype=x.dtype, device=x.device)
             out = kernels.gate_heads(out, self.hd, proj, self.cols[3], rows, self.heads, self.vd)
+        return self.o(out, defer=self.defer_output, out_dtype=self.output_dtype)
+
+
+@register_part("conv_window_attention")
+class ConvWindowAttention(KeptWindowAttention):
+    """Grouped-query attention whose queries, keys and values go through a short causal convolution over time, channel by channel,
+    right behind their projections, without norms, biases or rotation: where a key stands shows through ``distance_bias`` alone.
+    Optionally a query is multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)`` at its position ``p``, and every head's result by the
+    sigmoid of one number, ``(W_g h)[head]``, ahead of the output projection.  All projections of the input are one product; one
+    kernel (``conv_qkv_store``) sums its split-K parts, convolves, applies the temperature and stores; the attention kernels
+    cap, bias, add the sinks and scale each head's result by its gate.  The ``taps - 1`` projected values ahead of a step's tokens are
+    a request's state, in 32-bit.
+
+    params: ``hidden_size``, ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``taps`` (1 to 16), ``scale`` (None: ``dim^(-1/2)``), ``window`` (None: every
+    earlier key), ``keep_first`` (default 0), ``softcap``, ``distance_bias``, ``learned_sink`` (as ``attention``), ``query_temperature``
+    (None or ``(coef, every)``), ``head_gate`` (default false), ``prefix``.  Tensors: ``q [heads dim, hidden]``, ``k [kv_heads dim, hidden]``,
+    ``v [kv_heads vdim, hidden]``, ``{q,k,v}.conv [rows, taps]``, with ``learned_sink`` ``sink [heads]``, with ``head_gate`` ``g [heads, hidden]``,
+    ``o [hidden, heads vdim]``."""
+
+    graph_safe = True
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        if self.position is not None:
+            raise ValueError("conv_window_attention: queries and keys are not rotated")
+        self.taps, self.channels = int(params["taps"]), self.n_q + self.n_k + self.n_v
+        if not 1 <= self.taps <= 16:
+            raise ValueError(f"conv_window_attention: {self.taps} taps (1 to 16) are not served")
+        t = params.get("query_temperature")
+        self.temperature = (float(t[0]), float(t[1])) if t is not None else None
+        if self.temperature is not None and not self.temperature[1] > 0.0:
+            raise ValueError(f"conv_window_attention: a query temperature every {self.temperature[1]} positions")
+        self.head_gate = bool(params.get("head_gate", False))
+        self.kernel = None
+
+    def weight_decls(self):
+        p, W = self.prefix, self.hidden
+        decls = []
+        for name, rows in (("q", self.n_q), ("k", self.n_k), ("v", self.n_v)):
+            decls += [WeightDecl(p + name, (rows, W)), WeightDecl(p + name + ".conv", (rows, self.taps))]
+        if self.head_gate:
+            decls.append(WeightDecl(p + "g", (self.heads, W)))
+        return decls + self.sink_decls() + [WeightDecl(p + "o", (W, self.heads * self.vd))]
+
+    def bind(self, tensors):
+        p = self.prefix
+        rows = [tensors[p + n] for n in ("q", "k", "v") + (("g",) if self.head_gate else ())]
+        if len({t.dtype for t in rows}) > 1:
+            rows = [t.float() for t in rows]
+        self.qkv = Linear(torch.cat(rows, dim=0).contiguous(), self.ctx.dtype)
+        self.kernel = torch.cat([tensors[p + n + ".conv"].float() for n in ("q", "k", "v")], dim=0).t().contiguous()     # [taps, channels]
+        self.bind_scores(tensors)
+        self.o = Linear(self.padded_output_weight(tensors[p + "o"]), self.ctx.dtype)
+
+    def modules(self):
+        return ["conv_qkv"] + self.attention_modules() + self.qkv.modules() + self.o.modules()
+
+    def linears(self):
+        return [self.qkv, self.o]
+
+    def cache_need(self):
+        window = int(self.window) if self.window is not None else None
+        paged = PagedCacheNeed(self.groups, self.hd, window, keep_first=self.keep_first)
+        return paged if self.taps == 1 else CompositeCacheNeed((paged, StateCacheNeed(((self.taps - 1) * self.channels,), "float32")))
+
+    def forward(self, x, batch, cache):
+        tokens, state = (cache, None) if self.taps == 1 else (cache.parts[0], cache.parts[1].state)
+        T = x.shape[0]
+        proj = self.qkv(x, defer=True)
+        q = torch.empty((T, self.nh * self.hd), dtype=x.dtype, device=x.device)
+        gate = torch.empty((T, self.nh), dtype=torch.float32, device=x.device) if self.head_gate else None
+        kernels.conv_qkv_store(proj, self.kernel, state, batch.q_start, batch.state_slot, batch.num_seqs, 1 if batch.one_token_each else batch.num_tokens,
+                               batch.positions, batch.seq_of_token, q, tokens.block_table, tokens.pages, self.heads, self.groups, self.d, self.vd,
+                               temp=self.temperature, gate_col=self.channels, gate_out=gate, status=batch.status)
+        out = torch.empty((T, self.nh * self.hd), dtype=x.dtype, device=x.device)
+        self.attend(q, out, batch, tokens, out_scale=gate)
         return self.o(out, defer=self.defer_output, out_dtype=self.output_dtype)

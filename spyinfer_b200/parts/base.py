@@ -100,6 +100,14 @@ class Part:
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         """Receives the declared tensors (same relative names), already on the device."""
 
+    def shared_decls(self) -> List[WeightDecl]:
+        """Tensors that several parts of a model read, by their full names (a table with a share for every layer): the model
+        binds each once and hands it to every part that names it (``bind_shared``)."""
+        return []
+
+    def bind_shared(self, tensors: Dict[str, torch.Tensor]) -> None:
+        """Receives the tensors of ``shared_decls`` (full names)."""
+
     def modules(self) -> List[str]:
         return list(self.kernel_modules)
 
@@ -114,6 +122,8 @@ class Norm(Part):
     takes_scaled_parts: bool = False
     #: True: ``forward_add`` also takes a ``ChannelScaled`` as ``delta``
     takes_channel_scale: bool = False
+    #: True: ``forward_add`` also takes a ``NormedDelta`` as ``delta`` (of its own size, groups and eps)
+    takes_normed_delta: bool = False
 
     def forward(self, x: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
         raise NotImplementedError
@@ -168,6 +178,8 @@ class FeedForward(Part):
     #: set with ``leave_output_bias``: a feed-forward whose result has a term ``w[t] * x[t]`` (a weight a row times its input) may
     #: leave that to the consumer as well and offers it, after every ``forward``, as ``output_rows = (x, w)`` (else None)
     output_rows: Optional[Tuple[torch.Tensor, torch.Tensor]] = None
+    #: True: ``forward`` takes the step's batch as a second argument (a feed-forward that looks at the token ids)
+    takes_batch: bool = False
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
@@ -202,6 +214,9 @@ class Block:
         """``hidden`` is the 32-bit residual stream; ``delta`` the previous block's output
         that is still to be added to it (None for the first).  Returns the same pair."""
         raise NotImplementedError
+
+    def run_feed_forward(self, x: torch.Tensor, batch) -> torch.Tensor:
+        return self.feed_forward.forward(x, batch) if self.feed_forward.takes_batch else self.feed_forward.forward(x)
 
     def cache_need(self):
         """What the layer keeps between steps: its mixer's need, unless the arrangement keeps something of its own beside

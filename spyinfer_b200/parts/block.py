@@ -41,7 +41,7 @@ class PreNormBlock(Block):
         x = self.mixer_norm.forward_add(hidden, delta)
         a = self.mixer.forward(x, batch, cache)
         x = self.ffn_norm.forward_add(hidden, a)
-        return hidden, self.feed_forward.forward(x)
+        return hidden, self.run_feed_forward(x, batch)
 
 
 @register_block("post_norm")
@@ -79,7 +79,7 @@ class PostNormBlock(Block):
             kernels.residual_norm(hidden, None, None, 0.0, copy=x)
         x = self.mixer_norm.add_normed(hidden, self.mixer.forward(x, batch, cache))
         if self.feed_forward is not None:
-            x = self.ffn_norm.add_normed(hidden, self.feed_forward.forward(x))
+            x = self.ffn_norm.add_normed(hidden, self.run_feed_forward(x, batch))
         batch.extras["stream_copy"] = (hidden, x)
         return hidden, None
 
@@ -144,7 +144,7 @@ class ScaledPreNormBlock(Block):
         if self.feed_forward is None:
             return hidden, a
         x = self.ffn_norm.forward_add(hidden, a, scale=self.residual_scale)
-        f = self.feed_forward.forward(x)
+        f = self.run_feed_forward(x, batch)
         return hidden, self.ffn_scale.defer(f, self.feed_forward.output_bias, self.feed_forward.output_rows) if self.ffn_scale is not None else f
 
 
@@ -200,7 +200,39 @@ class SandwichNormBlock(Block):
         x = self.ffn_norm.forward_add(hidden, delta)
         if self.ffn_conv is not None:
             x = self.ffn_conv.forward(x, batch, self._view(cache, "ffn_conv"))
-        return hidden, self.ffn_out_norm.defer(self.feed_forward.forward(x), self.mult)
+        return hidden, self.ffn_out_norm.defer(self.run_feed_forward(x, batch), self.mult)
 
     def settle(self, hidden, delta):
         return self.mixer_out_norm.add_normed(hidden, delta) if delta is not None else hidden
+
+
+@register_block("parallel_sublayers")
+class ParallelSublayersBlock(Block):
+    """``x = norm(h); h += mixer(x) + ffn(x)``: one norm, whose output both sublayers read; a layer may do without the
+    feed-forward.  Optionally ``side`` (a part with ``forward(stream, batch)`` and ``defer(y)``, such as ``token_input``): what
+    it makes of the finished sum is added to the stream behind the two, normed; it is handed on as a ``NormedDelta`` that the next
+    norm of the stream forms in its own launch (it must say ``takes_normed_delta``).  The sum of the two results, which may be
+    split-K partial products, and the copy of the stream that the side input's product reads are one launch."""
+
+    graph_safe = True
+    required = ("mixer_norm", "mixer")
+    optional = ("feed_forward", "side")
+    kernel_modules = ("residual_norm",)
+
+    def __init__(self, parts, params=None):
+        super().__init__(parts, params)
+        if self.side is not None and not self.mixer_norm.takes_normed_delta:
+            raise ValueError(f"block arrangement 'parallel_sublayers': the norm {self.mixer_norm.kind!r} takes no normed result of a side input")
+
+    def forward(self, hidden, delta, batch, cache):
+        x = self.mixer_norm.forward_add(hidden, delta)
+        a = self.mixer.forward(x, batch, cache)
+        f = self.run_feed_forward(x, batch) if self.feed_forward is not None else None
+        if self.side is None:
+            return kernels.stream_sum(hidden, a, f), None
+        copy = None if x.dtype == hidden.dtype else torch.empty(hidden.shape, dtype=x.dtype, device=hidden.device)
+        kernels.stream_sum(hidden, a, f, copy)
+        return hidden, self.side.defer(self.side.forward(hidden if copy is None else copy, batch))
+
+    def settle(self, hidden, delta):
+        return self.mixer_norm.add_normed(hidden, delta) if delta is not None else hidden

@@ -16,7 +16,8 @@ fused weights, nothing stored twice), and every token's ``top`` results and the 
 32-bit.  On the bfloat16 path the products of all experts are one launch each (``gemm_grouped``: the runs are padded to whole tiles, a
 tile finds its expert on the device, nothing is read back); with sizes that launch does not take, and in 32-bit, the experts' row
 counts are read back once a layer to size a product for each.  Weights and arithmetic are the same, so the two forms differ by the
-order of sums only.  Both forms serve the options of the choice (a correction for the choice only, groups
+order of sums only.  The router may be absent: with a table of experts by token id a token's choice is fixed and its experts weigh the
+same, so nothing is scored.  Both forms serve the options of the choice (a correction for the choice only, groups
 of router outputs, identity experts, whose pairs take no rows) and both activations.
 """
 from __future__ import annotations
@@ -42,7 +43,9 @@ class ExpertMixture(FeedForward):
     only), ``groups`` (None or ``(count, keep)``: the router's outputs form ``count`` equal groups of neighbours, a group counts
     by its best choice score, and only the ``keep`` best groups' outputs can be chosen), ``scoring`` (``softmax`` over all outputs, the
     default, or ``sigmoid`` of each output's logit) and ``group_score`` (``best``, the default, or ``best_two``: the sum of a group's two
-    largest choice scores).  Tensors: ``router [experts +
+    largest choice scores); or ``scoring="table"`` with ``vocab_size``: no router, the integer tensor ``table [vocab_size, top]`` gives every
+    token id its experts, each with the weight ``1 / top`` (none of the other options of the choice then).  ``shared_gate`` (default
+    true): the shared expert's result is weighted by the sigmoid of ``shared.sg``'s logit; false: it is added as it is.  Tensors: ``router [experts +
     identity, hidden]``, ``e<i>.{gate,up} [ff, hidden]``, ``e<i>.down [hidden, ff]``, and with a shared expert
     ``shared.{gate,up,down}`` and ``shared.sg [1, hidden]``."""
 
@@ -59,8 +62,18 @@ class ExpertMixture(FeedForward):
         self.groups = tuple(int(v) for v in params["groups"]) if params.get("groups") else None
         self.outputs = self.experts + self.identity                 # the router's outputs
         self.scoring, self.group_score = params.get("scoring", "softmax"), params.get("group_score", "best")
-        if self.scoring not in ("softmax", "sigmoid") or self.group_score not in ("best", "best_two"):
-            raise ValueError(f"expert_mixture: scoring {self.scoring!r} (softmax, sigmoid), group score {self.group_score!r} (best, best_two)")
+        self.shared_gate = bool(params.get("shared_gate", True))
+        self.by_table = self.scoring == "table"
+        if self.by_table and (self.identity or self.has_correction or self.groups is not None or int(params.get("vocab_size") or 0) <= 0
+                              or (self.shared_ff and self.shared_gate)):
+            raise ValueError("expert_mixture: a table of experts needs vocab_size, takes no options of the choice and no gate on the shared expert")
+        if not self.by_table and self.shared_ff and not self.shared_gate:
+            raise ValueError("expert_mixture: a shared expert beside a router has a gate")
+        self.vocab = int(params.get("vocab_size") or 0)
+        self.takes_batch = self.by_table
+        self.table = None
+        if self.scoring not in ("softmax", "sigmoid", "table") or self.group_score not in ("best", "best_two"):
+            raise ValueError(f"expert_mixture: scoring {self.scoring!r} (softmax, sigmoid, table), group score {self.group_score!r} (best, best_two)")
         if min(self.hidden, self.experts, self.top, self.ff) <= 0 or self.top > self.outputs or self.shared_ff < 0 or self.identity < 0:
             raise ValueError(f"expert_mixture: {self.experts} experts of {self.ff}, top {self.top}, shared {self.shared_ff} are not served")
         if self.activation not in ("clamped_swish", "silu") or (self.activation == "clamped_swish" and not self.limit > 0.0):
@@ -89,12 +102,15 @@ class ExpertMixture(FeedForward):
 
     def weight_decls(self):
         p, W = self.prefix, self.hidden
-        decls = [WeightDecl(p + "router", (self.outputs, W))] + ([WeightDecl(p + "correction", (self.outputs,))] if self.has_correction else [])
+        if self.by_table:
+            decls = [WeightDecl(p + "table", (self.vocab, self.top), init=f"choice:{self.experts}", integer=True)]
+        else:
+            decls = [WeightDecl(p + "router", (self.outputs, W))] + ([WeightDecl(p + "correction", (self.outputs,))] if self.has_correction else [])
         for e in range(self.experts):
             decls += [WeightDecl(f"{p}e{e}.gate", (self.ff, W)), WeightDecl(f"{p}e{e}.up", (self.ff, W)), WeightDecl(f"{p}e{e}.down", (W, self.ff))]
         if self.shared_ff:
             decls += [WeightDecl(p + "shared.gate", (self.shared_ff, W)), WeightDecl(p + "shared.up", (self.shared_ff, W)),
-                      WeightDecl(p + "shared.down", (W, self.shared_ff)), WeightDecl(p + "shared.sg", (1, W))]
+                      WeightDecl(p + "shared.down", (W, self.shared_ff))] + ([WeightDecl(p + "shared.sg", (1, W))] if self.shared_gate else [])
         return decls
 
     def bind(self, tensors):
@@ -106,6 +122,11 @@ class ExpertMixture(FeedForward):
             rows, downs = [t.float() for t in rows], [t.float() for t in downs]
         self.gate_up = Linear(torch.cat(rows, dim=0).contiguous(), self.ctx.dtype)
         self.down = Linear(torch.cat(downs, dim=1).contiguous(), self.ctx.dtype)
+        if self.by_table:
+            self.table = tensors[p + "table"].contiguous()
+            if int(self.table.min()) < 0 or int(self.table.max()) >= self.experts:
+                raise ValueError(f"expert_mixture: the table {p + 'table'!r} names experts outside 0 .. {self.experts - 1}")
+            return
         # the router (and the shared expert's gate behind it) in 32-bit
         routes = [tensors[p + "router"].float()] + ([tensors[p + "shared.sg"].float()] if self.shared_ff else [])
         self.router = Linear(torch.cat(routes, dim=0).contiguous(), self.ctx.dtype)
@@ -113,20 +134,24 @@ class ExpertMixture(FeedForward):
             self.correction = tensors[p + "correction"].float().contiguous()
 
     def modules(self):
-        return ["moe"] + (["gemm_grouped"] if self._one_launch() else []) + self.router.modules() + self.gate_up.modules() + self.down.modules()
+        return ["moe"] + (["gemm_grouped"] if self._one_launch() else []) + (self.router.modules() if self.router is not None else []) + self.gate_up.modules() + self.down.modules()
 
     def linears(self):
-        return [self.router, self.gate_up, self.down]
+        return ([self.router] if self.router is not None else []) + [self.gate_up, self.down]
 
     def _one_launch(self) -> bool:
         return self.grouped and self.gate_up is not None and self.gate_up.fast and self.down.fast
 
-    def forward(self, x):
+    def forward(self, x, batch=None):
         if 0 < self.routed_from <= x.shape[0] and self.top < self.outputs and not torch.cuda.is_current_stream_capturing():
-            return self._routed(x)
-        logits = self.router(x, out_dtype=torch.float32)
+            return self._routed(x, batch)
+        logits = self.router(x, out_dtype=torch.float32) if not self.by_table else None
         gu = self.gate_up(x)
         y = torch.empty((x.shape[0], self.cols), dtype=self.ctx.dtype, device=x.device)
+        if self.by_table:
+            kernels.moe_activation_table(gu, self.table, batch.token_ids, y, self.experts, self.ff, self.limit, self.shared_ff, self.shared_limit, self.slope,
+                                         activation=self.activation)
+            return self.down(y, defer=self.defer_output)
         if self.plain_choice:
             kernels.moe_activation(gu, logits, y, self.experts, self.top, self.ff, self.limit, self.shared_ff, self.shared_limit, self.slope)
             return self.down(y, defer=self.defer_output)
@@ -162,13 +187,15 @@ class ExpertMixture(FeedForward):
                     self.down.part(y[a:b], cols=(ff * e, ff * (e + 1)), out=results[a:b])
         return results
 
-    def _routed(self, x):
+    def _routed(self, x, batch):
         T, E, top, ff, sff, dev = x.shape[0], self.experts, self.top, self.ff, self.shared_ff, x.device
-        logits = self.router(x, out_dtype=torch.float32)
-        idw = None
+        logits = self.router(x, out_dtype=torch.float32) if not self.by_table else None
+        idw = shared_w = None
         grouped = self._one_launch()
         pad = kernels.grouped_tile_rows() if grouped else 1
-        if self.plain_choice:
+        if self.by_table:
+            offsets, slot, row_token, row_w, *tiles = kernels.moe_route_table(self.table, batch.token_ids, E, pad=pad)
+        elif self.plain_choice:
             offsets, slot, row_token, row_w, shared_w, *tiles = kernels.moe_route(logits, E, top, bool(sff), pad=pad)
         else:
             offsets, slot, row_token, row_w, shared_w, idw, *tiles = kernels.moe_route_general(

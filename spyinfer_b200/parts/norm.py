@@ -134,8 +134,8 @@ class ChannelScale(Norm):
 @register_part("group_rms_norm")
 class GroupRMSNorm(Norm):
     """RMS norm in groups: the row is cut into ``groups`` equal consecutive parts, each divided by its own
-    ``sqrt(mean(part^2) + eps)``, and the whole multiplied by a plain weight.  params: ``size``, ``groups``, ``eps``,
-    ``weight`` (the tensor's relative name).
+    ``sqrt(mean(part^2) + eps)``, and the whole multiplied by a plain weight.  params: ``size``, ``groups`` (default 1), ``eps``,
+    ``weight`` (the tensor's relative name), ``weight_offset`` (default 0; with 1 the stored tensor is the gain's distance from one).
 
     It serves on both sides of a sublayer.  Ahead of one, ``forward_add(residual, delta)`` norms the stream; ``delta`` may
     be a ``NormedDelta`` that a norm of this kind (same size, groups and eps) left behind a sublayer (``defer``), and the
@@ -143,21 +143,25 @@ class GroupRMSNorm(Norm):
     record, and ``add_normed`` adds it at once."""
 
     graph_safe = True
+    takes_normed_delta = True
     kernel_modules = ("group_norm",)
 
     def __init__(self, params, ctx):
         super().__init__(params, ctx)
         self.size, self.groups, self.eps = int(params["size"]), int(params.get("groups", 1)), float(params["eps"])
+        self.weight_offset = float(params.get("weight_offset", 0.0))
         if self.groups <= 0 or self.size % self.groups:
             raise ValueError(f"group_rms_norm: rows of {self.size} cannot be cut into {self.groups} equal groups")
         self.weight_name = params.get("weight", "weight")
         self.weight = None
 
     def weight_decls(self):
-        return [WeightDecl(self.weight_name, (self.size,), init="one_plus_normal")]
+        return [WeightDecl(self.weight_name, (self.size,), init="normal" if self.weight_offset else "one_plus_normal")]
 
     def bind(self, tensors):
         self.weight = tensors[self.weight_name].contiguous()
+        if self.weight_offset:
+            self.weight = (self.weight.float() + self.weight_offset).contiguous()     # the gain itself, in 32-bit
 
     def defer(self, y, scale=1.0):
         return NormedDelta(y, self.weight, float(scale))
@@ -167,7 +171,10 @@ class GroupRMSNorm(Norm):
             return None, None, 1.0
         if not isinstance(delta, NormedDelta):
             raise ValueError("group_rms_norm: what is pending on the stream must be a sublayer output that a norm of this kind deferred")
-        return delta.y, delta.weight, delta.scale
+        weight = delta.weight
+        if self.weight is not None and weight.dtype != self.weight.dtype:      # one storage type for the two norms of a launch
+            weight, self.weight = weight.float(), self.weight.float()
+        return delta.y, weight, delta.scale
 
     def add_normed(self, residual, delta):
         """``residual += scale * norm(y) * weight`` for a ``NormedDelta`` (32-bit, in place)."""

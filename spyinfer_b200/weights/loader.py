@@ -26,7 +26,8 @@ from .safetensors_io import SafetensorsError, SafetensorsFile, shard_paths
 class WeightDecl:
     """One tensor a model needs.  ``init`` says how a random model fills it: ``"normal"``
     (zero mean), ``"one_plus_normal"`` (norm gains) or ``"zeros"``.  ``integer`` marks an
-    index table, kept as int32."""
+    index table, kept as int32 (``init`` then ``"choice:<n>"``: every row holds different numbers
+    below n)."""
 
     name: str
     shape: Tuple[int, ...]

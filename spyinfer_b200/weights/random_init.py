@@ -26,9 +26,14 @@ def _tensor_seed(seed: int, name: str) -> int:
 
 
 def random_tensor(decl: WeightDecl, seed: int, std: float, norm_std: float, device) -> torch.Tensor:
-    if decl.integer:
+    if decl.integer and not decl.init.startswith("choice:"):
         raise ValueError(f"{decl.name}: no rule for a random integer table")
     g = torch.Generator(device=device).manual_seed(_tensor_seed(seed, decl.name))
+    if decl.integer:                  # "choice:<n>": every row holds different numbers below n
+        n, (rows, k) = int(decl.init.split(":")[1]), decl.shape
+        if k > n:
+            raise ValueError(f"{decl.name}: no {k} different numbers below {n}")
+        return torch.cat([torch.rand((min(rows - r, 65536), n), generator=g, device=device).argsort(1)[:, :k] for r in range(0, rows, 65536)]).to(torch.int32).contiguous()
     if decl.init == "zeros":
         return torch.zeros(decl.shape, dtype=torch.bfloat16, device=device)
     x = torch.randn(decl.shape, generator=g, device=device, dtype=torch.float32)
@@ -62,7 +67,7 @@ def write_model_folder(model_dir: str, config, seed: int, std: float = 0.02, nor
     decls = declared_weights(config.to_spec())
 
     def nbytes(d):
-        n = 2
+        n = 4 if d.integer else 2
         for k in d.shape:
             n *= int(k)
         return n
@@ -83,5 +88,5 @@ def write_model_folder(model_dir: str, config, seed: int, std: float = 0.02, nor
         with open(os.path.join(model_dir, "model.safetensors.index.json"), "w") as f:
             json.dump(index, f, indent=1)
     for name, part in zip(names, shards):
-        layout = [(d.name, torch.bfloat16, tuple(d.shape)) for d in part]
+        layout = [(d.name, torch.int32 if d.integer else torch.bfloat16, tuple(d.shape)) for d in part]
         write_safetensors(os.path.join(model_dir, name), layout, random_tensors(part, seed, std, norm_std, device))
