@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--shape 8b|14b|32b] [--batch B] [--context C] [--impl ours|reference]
     python bench.py --workload mixed [--shape 14b] [--requests 64] [--budget 2048]     (a continuous batch through LLMEngine; its own line)
-    python bench.py --workload nezolorn | daronex | naforax | dogilorn | zonevik [--layers 6] [--prefill-tokens 2048]   (another design beside Qwen3 at equal layer sizes; its own line)
+    python bench.py --workload nezolorn | daronex | naforax | dogilorn | zonevik | bubalix [--layers 6] [--prefill-tokens 2048]   (another design beside Qwen3 at equal layer sizes; its own line)
 
 The model has the layer sizes of Qwen3-8B (36 layers, hidden 4096, 32 query heads, 8 key/value
 heads, head size 128, intermediate 12288, vocabulary 151936, untied head) with seeded random
@@ -363,10 +363,11 @@ def mixed_workload(args, model_config, layers, full_layers, page) -> int:
     return 0
 
 
-def _measure_design(args, cfg_json, vocab, page, T, ctx, annotate):
+def _measure_design(args, cfg_json, vocab, page, T, ctx, annotate, tell_apart=None):
     """One model of ``--workload nezolorn`` / ``daronex``: a prompt of ``T`` tokens in one step, decoding at batch 8 and 64 from ``ctx``
     tokens, and every kernel's time inside one prompt step and one decode step of batch 64 launched one by one;
-    ``annotate(res, rate)`` adds achieved rates (``rate(block, kernel function, flops=, nbytes=)``)."""
+    ``annotate(res, rate)`` adds achieved rates (``rate(block, kernel function, flops=, nbytes=)``); ``tell_apart(fn, n)`` may name the ``n``-th
+    launch of a function within a step (one function that layers of several kinds launch)."""
     import torch
 
     from spyinfer_b200 import config_from_json, kernels
@@ -437,8 +438,11 @@ def _measure_design(args, cfg_json, vocab, page, T, ctx, annotate):
         finally:
             kernels.time_calls(None)
             runner._use_graphs = graphs
-        out = {}
+        out, seen = {}, {}
         for fn, a, b in sink:
+            seen[fn] = seen.get(fn, 0) + 1
+            if tell_apart is not None:
+                fn = tell_apart(fn, seen[fn] - 1)
             us, n = out.get(fn, (0.0, 0))
             out[fn] = (us + a.elapsed_time(b) * 1e3, n + 1)
         return {fn: {"us": round(us, 1), "launches": n} for fn, (us, n) in sorted(out.items(), key=lambda kv: -kv[1][0])}
@@ -909,6 +913,111 @@ def zonevik_workload(args) -> int:
     return 0
 
 
+def bubalix_workload(args) -> int:
+    """``--workload bubalix``: prefill and decode throughput of the Bubalix design (attention through a latent with sinks, and attention over
+    a window behind convolutions with capped, distance-biased scores, sinks, a query temperature and a gate a head, in turns; an
+    expert mixture by a table of token ids with a shared expert beside every mixer on one norm; a per-layer token input) at two layer
+    sizes that resemble real models, beside the engine's Qwen3 model with the same width, heads, head size, vocabulary, number of layers, the
+    same sliding window on every layer and a feed-forward of a token's experts' size, and beside its Daronex model with layers of
+    attention through a latent of the same sizes, all with seeded random weights in bfloat16.  Measured as ``--workload nezolorn`` is:
+    one prompt of ``--prefill-tokens`` tokens, decoding at batch 8 and 64 from ``--context`` tokens through the decode graphs, and each
+    kernel's time inside one prompt step and one decode step of batch 64."""
+    hbm_gbs, bf16_tflops, _, peak_src = peaks()
+    layers, vocab, page = args.layers or 6, 32000, 16
+    T, ctx = args.prefill_tokens, min(args.context, 4096)
+    window = 1024
+    sizes = {"width2048": dict(width=2048, heads=16, kv=4, hd=128, experts=8, top=2, expert_ff=2048, shared_ff=4096, side=256,
+                               l_heads=16, dim=64, rot=32, vdim=64, kv_rank=96),
+             "width4096": dict(width=4096, heads=32, kv=8, hd=128, experts=8, top=2, expert_ff=3072, shared_ff=6144, side=256,
+                               l_heads=16, dim=128, rot=32, vdim=128, kv_rank=96)}
+
+    def configs(z):
+        moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["expert_ff"]}, "shared": {"ff": z["shared_ff"]}}
+        rot = {"base": 500000.0, "dims": z["rot"], "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+        latent = {"heads": z["l_heads"], "dim": z["dim"], "rot_dim": z["rot"], "vdim": z["vdim"], "kv_rank": z["kv_rank"],
+                  "scale": (z["dim"] + z["rot"]) ** -0.5}
+        attn = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["hd"], "vdim": z["hd"], "scale": z["hd"] ** -0.5, "softcap": 20.0, "conv": 4,
+                "q_temp": {"coef": 0.1, "every": 2048}, "mask": {"size": window}}
+        kinds = [{"type": "latent_attention", "mixer": dict(latent, rot=rot), "mlp": moe}, {"type": "attention", "mixer": attn, "mlp": moe}]
+        active = z["top"] * z["expert_ff"] + z["shared_ff"]
+        bx = {"architecture": "Bubalix", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 2.0},
+              "token_side": {"dim": z["side"]}, "layers": [kinds[i % 2] for i in range(layers)]}
+        qw = dict(QWEN3_8B)
+        qw.update({"num_hidden_layers": layers, "hidden_size": z["width"], "num_attention_heads": z["heads"], "num_key_value_heads": z["kv"],
+                   "head_dim": z["hd"], "intermediate_size": active, "vocab_size": vocab, "use_sliding_window": True, "sliding_window": window,
+                   "max_window_layers": 0})
+        dx = {"architecture": "Daronex", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+              "layers": [{"type": "latent_attention", "mlp": {"kind": "dense", "ff": active},
+                          "mixer": dict(latent, q_rank=3 * z["width"] // 8, rot={"base": 500000.0, "dims": z["rot"]})}] * layers}
+        return {"bubalix": bx, "qwen3": qw, "daronex": dx}
+
+    def tell_apart(fn, n):
+        return fn + (":latent" if n % 2 == 0 else ":window") if fn in ("attention_tc.spy_attention_tc_scores", "attention_decode.spy_attention_decode_scores") else fn
+
+    def measure(cfg_json, z, name):
+        def annotate(res, rate):
+            W, H, kv, hd, row = z["width"], z["heads"], z["kv"], z["hd"], z["kv_rank"] + z["rot"]
+            n_lat = (layers + 1) // 2 if name == "bubalix" else layers
+            n_win = layers - n_lat if name == "bubalix" else layers
+            full, windowed = T * (T + 1) / 2, sum(min(p + 1, window) for p in range(T))
+            lat_flops, lat_bytes = 2.0 * full * n_lat * z["l_heads"] * (row + z["kv_rank"]), 64.0 * (ctx + 1) * n_lat * row * 2
+            win_flops, win_bytes = 4.0 * windowed * n_win * H * hd, 64.0 * kv * min(ctx + 1, window) * hd * 2 * 2 * n_win
+            product = 2.0 * n_lat * z["l_heads"] * (z["dim"] * z["kv_rank"] + z["kv_rank"] * z["vdim"])
+            tc, dec = "attention_tc.spy_attention_tc", "attention_decode.spy_attention_decode"
+            for block, rows in (("kernels_prefill", T), ("kernels_decode_b64", 64)):
+                if name == "bubalix":
+                    rate(block, tc + "_scores:latent", flops=lat_flops)
+                    rate(block, tc + "_scores:window", flops=win_flops)
+                    rate(block, dec + "_scores:latent", nbytes=lat_bytes)
+                    rate(block, dec + "_scores:window", nbytes=win_bytes)
+                    routed = "moe.spy_moe_combine" in res[block]
+                    f_bytes = 4 if routed else 2
+                    # the pending token input and the stream are read, the stream and the normed row written; the two results and the stream
+                    # are read, the stream and its 16-bit copy written
+                    rate(block, "group_norm.spy_group_norm", nbytes=float(layers) * rows * W * (2 + 4 + 4 + 2))
+                    rate(block, "residual_norm.spy_stream_sum", nbytes=float(layers) * rows * W * (2 + f_bytes + 4 + 4 + 2))
+                    rate(block, "conv_qkv.spy_conv_qkv_store", nbytes=float(rows) * n_win * (H + 2 * kv) * hd * 4)
+                    rate(block, "embedding.spy_token_gate", nbytes=float(rows) * layers * z["side"] * 6)
+                    if routed:
+                        pairs = float(layers) * rows * z["top"]
+                        rate(block, "gemm_grouped.spy_gemm_grouped", flops=pairs * 3 * W * z["expert_ff"] * 2)
+                        rate(block, "moe.spy_gather_rows", nbytes=pairs * W * 4)
+                        rate(block, "moe.spy_expert_activation", nbytes=(pairs * z["expert_ff"] + float(layers) * rows * z["shared_ff"]) * 6)
+                        rate(block, "moe.spy_moe_combine", nbytes=(pairs + 2 * layers * rows) * W * 4)
+                    else:
+                        cols = z["experts"] * z["expert_ff"] + z["shared_ff"]
+                        rate(block, "moe.spy_moe_activation_table", nbytes=float(layers) * rows * ((z["top"] * z["expert_ff"] + z["shared_ff"]) * 4 + cols * 2))
+                elif name == "qwen3":
+                    rate(block, tc, flops=win_flops)
+                    rate(block, dec, nbytes=win_bytes)
+                    rate(block, "rmsnorm.spy_rmsnorm", nbytes=float(2 * layers) * rows * W * (4 + 4 + 4 + 2))
+                    rate(block, "qk_rope_store.spy_qk_rope_store", nbytes=float(layers) * rows * (H + 2 * kv) * hd * 4)
+                else:
+                    rate(block, tc, flops=lat_flops)
+                    rate(block, dec, nbytes=lat_bytes)
+                    rate(block, "residual_norm.spy_residual_norm", nbytes=float(2 * layers) * rows * W * (4 + 4 + 4 + 2))
+                if name != "qwen3":
+                    rate(block, "latent.spy_head_product", flops=product * rows)
+                    rate(block, "latent.spy_latent_prep", nbytes=float(rows) * n_lat * row * 6)
+
+        return _measure_design(args, cfg_json, vocab, page, T, ctx, annotate, tell_apart if name == "bubalix" else None)
+
+    out_sizes = {}
+    with ClockSampler() as clocks:
+        for tag, z in sizes.items():
+            out_sizes[tag] = {"layer_sizes": z, "layers": layers}
+            for name, cfg_json in configs(z).items():
+                out_sizes[tag][name] = measure(cfg_json, z, name)
+    print(json.dumps({"metric": "prefill and decode tokens/s of the Bubalix design beside Qwen3 and Daronex at equal layer sizes (bf16, random weights)",
+                      "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": 3, "dtype": "bf16",
+                      "data": "synthetic: seeded random weights and random token ids",
+                      "config": {"layers": layers, "vocab": vocab, "prefill_tokens": T, "decode_context": ctx, "window": window, "page_size": page,
+                                 "pattern": "attention through a latent, attention over a window behind convolutions; in turns, an expert mixture beside each",
+                                 "timing": "CUDA events; inputs (weights, caches and states of 64 requests) exceed L2"},
+                      "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": bf16_tflops, "source": peak_src}, "sizes": out_sizes, "clocks": clocks.summary()}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -923,7 +1032,7 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1/64 and short-context points")
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-kernels", action="store_true", help="skip the per-kernel rooflines")
-    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "nezolorn", "daronex", "naforax", "dogilorn", "zonevik"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "nezolorn", "daronex", "naforax", "dogilorn", "zonevik", "bubalix"],
                     help="decode: the contract's line (default); mixed: a continuous batch of --requests requests with prompts of 64 to 2,048 "
                          "tokens and 128 generated tokens each through LLMEngine, its own line; nezolorn, daronex, naforax, dogilorn, zonevik: prefill and decode of that design "
                          "beside Qwen3 at equal layer sizes, its own line")
@@ -952,6 +1061,8 @@ def main() -> int:
         return dogilorn_workload(args)
     if args.workload == "zonevik":
         return zonevik_workload(args)
+    if args.workload == "bubalix":
+        return bubalix_workload(args)
     hbm_gbs, bf16_tflops, bf16_sustained, peak_src = peaks()
     cfg_json = dict(QWEN3_8B)
     cfg_json.update(SHAPES[args.shape])

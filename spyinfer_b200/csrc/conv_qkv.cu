@@ -9,7 +9,7 @@
 // group of columns, a gate a head, becomes gate_out[t, h] = sigmoid(u[gate_col + h]) (gate_out null: none).
 //
 // The `taps - 1` projected values ahead of a step's run of tokens lie in state[slot] (float32 [taps - 1, channels], oldest first,
-// zero for a new request) and the run's last ones go there.  Grid: x = request x piece of PIECE tokens, y = elements of a token's
+// zero for a new request) and the run's last ones go there.  Grid: x = request x piece of `PIECE` tokens, y = elements of a token's
 // rows; a thread owns V neighbouring channels of one piece and walks its tokens with the last inputs in registers.  Only the thread
 // of a run's first piece reads and writes the state of its (request, channels), so no thread reads what another writes.  All
 // arithmetic in 32-bit.
@@ -17,7 +17,8 @@
 
 SPY_MODULE(spy_conv_qkv)
 
-constexpr int PIECE = 16;          // tokens a thread walks; at least taps - 1, so that only a run's first piece needs the state
+// tokens a thread walks: at least taps - 1, so that only a run's first piece needs the state
+constexpr int piece_of(int max_taps) { return max_taps <= 4 ? 8 : 16; }
 
 template <int V, typename T>
 __device__ __forceinline__ void take(const T* p, float (&v)[V])
@@ -54,7 +55,6 @@ struct ConvArgs {
     const int* q_start;
     const int* state_slot;
     const int* positions;
-    const int* seq_of_token;
     const int* block_table;
     int table_width, page_size, num_pages, heads, kv_heads, dim, vdim, hd, taps, pieces;
     float temp_coef, temp_every;
@@ -81,6 +81,7 @@ template <typename TP, typename TQ, int V, int MAXT>
 __global__ void __launch_bounds__(128)
 conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restrict__ pages, ConvArgs A)
 {
+    constexpr int PIECE = piece_of(MAXT);
     pdl_enter();
     const int seq = blockIdx.x / A.pieces, piece = blockIdx.x % A.pieces;
     const int start = A.q_start[seq], end = A.q_start[seq + 1];
@@ -147,15 +148,19 @@ conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restr
                 if (i < hist_n) columns<V>(in + (long long)(t0 - hist_n + i) * A.ld, A.splits, A.split_stride, hist[i]);
         }
     }
-    // four tokens' inputs are requested together, then used in order
-    constexpr int AHEAD = 4;
+    // eight (or four) tokens' inputs are requested together, then used in order
+    constexpr int AHEAD = MAXT <= 4 ? 8 : 4;
     for (int tb = t0; tb < t1; tb += AHEAD) {
         float xs[AHEAD][V];
+        int pos_of[AHEAD], page_of[AHEAD];
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
 #pragma unroll
             for (int e = 0; e < V; ++e) xs[u][e] = 0.f;
             if (content && tb + u < t1) columns<V>(in + (long long)(tb + u) * A.ld, A.splits, A.split_stride, xs[u]);
+            pos_of[u] = tb + u < t1 ? A.positions[tb + u] : 0;
+            const int lp = pos_of[u] >= 0 ? pos_of[u] / A.page_size : -1;
+            page_of[u] = (kind != 0 && tb + u < t1 && lp >= 0 && lp < A.table_width) ? A.block_table[(long long)seq * A.table_width + lp] : -1;
         }
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
@@ -176,7 +181,7 @@ conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restr
 #pragma unroll
                     for (int e = 0; e < V; ++e) acc[e] = fmaf(k[j][e], xs[u][e], acc[e]);
                 }
-            const int pos = A.positions[t];
+            const int pos = pos_of[u];
             TQ* dst = nullptr;
             if (kind == 0) {
                 if (A.temp_every > 0.f) {
@@ -186,8 +191,7 @@ conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restr
                 }
                 dst = q_out + ((long long)t * A.heads + head) * A.hd + e0;
             } else {
-                const int lp = pos >= 0 ? pos / A.page_size : -1;
-                const int page = (lp >= 0 && lp < A.table_width) ? A.block_table[(long long)A.seq_of_token[t] * A.table_width + lp] : -1;
+                const int page = page_of[u];
                 if (page >= 0 && page < A.num_pages)
                     dst = pages + ((((long long)page * 2 + (kind - 1)) * A.kv_heads + head) * A.page_size + pos % A.page_size) * A.hd + e0;
                 else if (kind == 1 && head == 0 && e0 == 0) report_status(A.status, SPY_STATUS_BAD_PAGE, t);
@@ -209,7 +213,7 @@ conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restr
 // q_out [T, heads * hd]; pages [num_pages][2][kv_heads][page_size][hd] of the queries' type.  `longest`: no request brings more tokens.
 extern "C" int spy_conv_qkv_store(const void* proj, int proj_dtype, long long ld, int splits, long long split_stride, const float* kernel, int taps,
                                   float* state, const int* q_start, const int* state_slot, int seqs, int longest, float temp_coef, float temp_every,
-                                  int gate_col, float* gate_out, const int* positions, const int* seq_of_token, void* q_out, int q_dtype,
+                                  int gate_col, float* gate_out, const int* positions, void* q_out, int q_dtype,
                                   const int* block_table, int table_width, void* pages, int page_size, int num_pages, int heads, int kv_heads, int dim,
                                   int vdim, int hd, int* status, cudaStream_t stream)
 {
@@ -220,8 +224,8 @@ extern "C" int spy_conv_qkv_store(const void* proj, int proj_dtype, long long ld
     if (page_size <= 0 || num_pages <= 0 || table_width <= 0 || block_table == nullptr || pages == nullptr)
         SPY_FAIL("conv_qkv: page_size, num_pages and table_width must be positive");
     if (temp_every < 0.f) SPY_FAIL("conv_qkv: a query temperature every %g positions", temp_every);
-    const int pieces = (longest + PIECE - 1) / PIECE;
-    const ConvArgs A = {ld, split_stride, splits, kernel, state, q_start, state_slot, positions, seq_of_token, block_table, table_width, page_size, num_pages,
+    const int piece = taps <= 4 ? piece_of(4) : piece_of(16), pieces = (longest + piece - 1) / piece;
+    const ConvArgs A = {ld, split_stride, splits, kernel, state, q_start, state_slot, positions, block_table, table_width, page_size, num_pages,
                         heads, kv_heads, dim, vdim, hd, taps, pieces, temp_coef, temp_every, gate_col, gate_out, status};
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     const bool vec = dim % 4 == 0 && vdim % 4 == 0 && hd % 4 == 0 && ld % 4 == 0 && split_stride % 4 == 0 && aligned(proj) && aligned(kernel) && aligned(state)

@@ -1821,7 +1821,7 @@ def token_gate(gate: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Ten
 
 
 def conv_qkv_store(proj: torch.Tensor, kernel: torch.Tensor, state: Optional[torch.Tensor], q_start: torch.Tensor, state_slot: torch.Tensor, num_seqs: int,
-                   longest: int, positions: torch.Tensor, seq_of_token: torch.Tensor, q_out: torch.Tensor, block_table: torch.Tensor, pages: torch.Tensor,
+                   longest: int, positions: torch.Tensor, q_out: torch.Tensor, block_table: torch.Tensor, pages: torch.Tensor,
                    heads: int, kv_heads: int, dim: int, vdim: int, temp: Optional[tuple] = None, gate_col: int = -1, gate_out: Optional[torch.Tensor] = None,
                    status: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The step ahead of the attention kernel for queries, keys and values behind a causal convolution over time.  ``proj [T, ld]`` (or a
@@ -1842,11 +1842,11 @@ def conv_qkv_store(proj: torch.Tensor, kernel: torch.Tensor, state: Optional[tor
     _check(q_out, "queries", ndim=2)
     _check(pages, "cache pages", q_out.dtype, 5)
     _check(block_table, "block table", torch.int32, 2)
-    for t, what in ((positions, "positions"), (seq_of_token, "seq_of_token"), (q_start, "q_start"), (state_slot, "state_slot")):
+    for t, what in ((positions, "positions"), (q_start, "q_start"), (state_slot, "state_slot")):
         _check(t, what, torch.int32, 1)
     taps, channels = kernel.shape
     num_pages, two, nkv, page_size, hd = pages.shape
-    if two != 2 or nkv != kv_heads or tuple(q_out.shape) != (T, heads * hd) or positions.shape[0] != T or seq_of_token.shape[0] != T:
+    if two != 2 or nkv != kv_heads or tuple(q_out.shape) != (T, heads * hd) or positions.shape[0] != T:
         raise KernelError(f"conv_qkv_store: pages {tuple(pages.shape)} / queries {tuple(q_out.shape)} do not fit {heads} heads over {kv_heads} of rows {hd}")
     if channels != heads * dim + kv_heads * (dim + vdim) or channels > ld:
         raise KernelError(f"conv_qkv_store: {channels} channels and {ld} columns do not fit {heads} heads over {kv_heads} of {dim} and {vdim}")
@@ -1863,7 +1863,7 @@ def conv_qkv_store(proj: torch.Tensor, kernel: torch.Tensor, state: Optional[tor
     coef, every = (float(temp[0]), float(temp[1])) if temp is not None else (0.0, 0.0)
     _call("conv_qkv", "spy_conv_qkv_store", _ptr(proj), _code(proj, "projection"), ctypes.c_longlong(ld), splits, ctypes.c_longlong(stride), _ptr(kernel), taps,
           _ptr(state if taps > 1 else None), _ptr(q_start), _ptr(state_slot), int(num_seqs), int(longest), ctypes.c_float(coef), ctypes.c_float(every),
-          int(gate_col), _ptr(gate_out), _ptr(positions), _ptr(seq_of_token), _ptr(q_out), _code(q_out, "queries"), _ptr(block_table), block_table.shape[1],
+          int(gate_col), _ptr(gate_out), _ptr(positions), _ptr(q_out), _code(q_out, "queries"), _ptr(block_table), block_table.shape[1],
           _ptr(pages), page_size, num_pages, int(heads), int(kv_heads), int(dim), int(vdim), hd, _ptr(status), _stream())
     return q_out
 

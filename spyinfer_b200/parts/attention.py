@@ -804,7 +804,7 @@ class ConvWindowAttention(KeptWindowAttention):
         q = torch.empty((T, self.nh * self.hd), dtype=x.dtype, device=x.device)
         gate = torch.empty((T, self.nh), dtype=torch.float32, device=x.device) if self.head_gate else None
         kernels.conv_qkv_store(proj, self.kernel, state, batch.q_start, batch.state_slot, batch.num_seqs, 1 if batch.one_token_each else batch.num_tokens,
-                               batch.positions, batch.seq_of_token, q, tokens.block_table, tokens.pages, self.heads, self.groups, self.d, self.vd,
+                               batch.positions, q, tokens.block_table, tokens.pages, self.heads, self.groups, self.d, self.vd,
                                temp=self.temperature, gate_col=self.channels, gate_out=gate, status=batch.status)
         out = torch.empty((T, self.nh * self.hd), dtype=x.dtype, device=x.device)
         self.attend(q, out, batch, tokens, out_scale=gate)
