@@ -297,27 +297,24 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
                         tmem_wait_ld();
                         uint32_t packed[HALF / 2];
 #pragma unroll
-                        for (int i = 0; i < HALF; i += 4) {
-                            // cap tanh(s scale / cap) - cap = -2 cap / (exp(2 s scale / cap) + 1), and the bias: four scores share one
-                            // reciprocal, that of their denominators' product (each below 2^30.1: beyond that tanh is 1 in 32-bit)
-                            float a[4], pr[4];
+                        for (int i = 0; i < HALF; i += 2) {
+                            float pr[2];
 #pragma unroll
-                            for (int e = 0; e < 4; ++e) a[e] = fast_exp2(fminf(__uint_as_float(sc[i + e]) * cap_in, 30.f)) + 1.f;
-                            const float ab = a[0] * a[1], cd = a[2] * a[3], r = fast_rcp(ab * cd) * (-2.f * cap_log2), rcd = r * cd, rab = r * ab;
-                            const float inv4[4] = {rcd * a[1], rcd * a[0], rab * a[3], rab * a[2]};
-#pragma unroll
-                            for (int e = 0; e < 4; ++e) pr[e] = fast_exp2(inv4[e] + fmaf((float)(h * HALF + i + e), slope2, bias0));
+                            for (int e = 0; e < 2; ++e) {
+                                // cap tanh(s scale / cap) - cap = -2 cap / (exp(2 s scale / cap) + 1), and the bias
+                                const float r = fast_rcp(fast_exp2(__uint_as_float(sc[i + e]) * cap_in) + 1.f);
+                                pr[e] = fast_exp2(fmaf(-2.f * cap_log2, r, fmaf((float)(h * HALF + i + e), slope2, bias0)));
+                            }
                             if (!whole) {
 #pragma unroll
-                                for (int e = 0; e < 4; ++e) {
+                                for (int e = 0; e < 2; ++e) {
                                     const int k = key0 + h * HALF + i + e;
                                     if (!(k <= pos && k >= lo)) pr[e] = 0.f;
                                 }
                             }
-                            sums[0] += pr[0] + pr[1];
-                            sums[1] += pr[2] + pr[3];
+                            sums[0] += pr[0];
+                            sums[1] += pr[1];
                             packed[i / 2] = pack_bf16(pr[0], pr[1]);
-                            packed[i / 2 + 1] = pack_bf16(pr[2], pr[3]);
                         }
                         tmem_store<32>(tmem_s + h * (HALF / 2), packed);
                     }

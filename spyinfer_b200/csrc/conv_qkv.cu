@@ -82,11 +82,23 @@ __global__ void __launch_bounds__(128)
 conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restrict__ pages, ConvArgs A)
 {
     constexpr int PIECE = piece_of(MAXT);
+    __shared__ float temp_s[PIECE];          // what a token's queries are multiplied by
+    __shared__ long long page_s[PIECE];      // its place in the pages: page * 2 * kv_heads * page_size + slot, or below zero
     pdl_enter();
     const int seq = blockIdx.x / A.pieces, piece = blockIdx.x % A.pieces;
     const int start = A.q_start[seq], end = A.q_start[seq + 1];
     const int t0 = start + piece * PIECE, t1 = min(end, t0 + PIECE);
     if (t0 >= end) return;
+    if (threadIdx.x < PIECE && t0 + (int)threadIdx.x < t1) {
+        const int t = t0 + threadIdx.x, pos = A.positions[t];
+        const int lp = pos >= 0 ? pos / A.page_size : -1;
+        const int page = (lp >= 0 && lp < A.table_width) ? A.block_table[(long long)seq * A.table_width + lp] : -1;
+        const bool ok = page >= 0 && page < A.num_pages;
+        if (!ok && blockIdx.y == 0) report_status(A.status, SPY_STATUS_BAD_PAGE, t);
+        page_s[threadIdx.x] = ok ? (long long)page * 2 * A.kv_heads * A.page_size + (pos - lp * A.page_size) : -1;
+        temp_s[threadIdx.x] = A.temp_every > 0.f ? 1.0f + A.temp_coef * logf(floorf((float)(pos + 1) / A.temp_every) + 1.0f) : 1.0f;
+    }
+    __syncthreads();
     const int per_head = A.hd / V, rows = A.heads + 2 * A.kv_heads;
     int item = blockIdx.y * blockDim.x + threadIdx.x;
     if (item >= rows * per_head) {
@@ -148,19 +160,16 @@ conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restr
                 if (i < hist_n) columns<V>(in + (long long)(t0 - hist_n + i) * A.ld, A.splits, A.split_stride, hist[i]);
         }
     }
-    // eight (or four) tokens' inputs are requested together, then used in order
-    constexpr int AHEAD = MAXT <= 4 ? 8 : 4;
+    const long long row_at = (long long)(kind == 2 ? A.kv_heads + head : head) * A.page_size;      // a key or value head's rows within a page
+    // four tokens' inputs are requested together, then used in order
+    constexpr int AHEAD = 4;
     for (int tb = t0; tb < t1; tb += AHEAD) {
         float xs[AHEAD][V];
-        int pos_of[AHEAD], page_of[AHEAD];
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
 #pragma unroll
             for (int e = 0; e < V; ++e) xs[u][e] = 0.f;
             if (content && tb + u < t1) columns<V>(in + (long long)(tb + u) * A.ld, A.splits, A.split_stride, xs[u]);
-            pos_of[u] = tb + u < t1 ? A.positions[tb + u] : 0;
-            const int lp = pos_of[u] >= 0 ? pos_of[u] / A.page_size : -1;
-            page_of[u] = (kind != 0 && tb + u < t1 && lp >= 0 && lp < A.table_width) ? A.block_table[(long long)seq * A.table_width + lp] : -1;
         }
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
@@ -181,20 +190,14 @@ conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restr
 #pragma unroll
                     for (int e = 0; e < V; ++e) acc[e] = fmaf(k[j][e], xs[u][e], acc[e]);
                 }
-            const int pos = pos_of[u];
             TQ* dst = nullptr;
             if (kind == 0) {
-                if (A.temp_every > 0.f) {
-                    const float f = 1.0f + A.temp_coef * logf(floorf((float)(pos + 1) / A.temp_every) + 1.0f);
+                const float f = temp_s[t - t0];
 #pragma unroll
-                    for (int e = 0; e < V; ++e) acc[e] *= f;
-                }
+                for (int e = 0; e < V; ++e) acc[e] *= f;
                 dst = q_out + ((long long)t * A.heads + head) * A.hd + e0;
-            } else {
-                const int page = page_of[u];
-                if (page >= 0 && page < A.num_pages)
-                    dst = pages + ((((long long)page * 2 + (kind - 1)) * A.kv_heads + head) * A.page_size + pos % A.page_size) * A.hd + e0;
-                else if (kind == 1 && head == 0 && e0 == 0) report_status(A.status, SPY_STATUS_BAD_PAGE, t);
+            } else if (page_s[t - t0] >= 0) {
+                dst = pages + (page_s[t - t0] + row_at) * A.hd + e0;
             }
             if (dst != nullptr) put<V>(dst, acc);
 #pragma unroll
