@@ -38,7 +38,8 @@
 // SpyScores (common.cuh): a cap on the scores and a distance bias are applied to the scores as they are read from tensor
 // memory, in 32-bit.  A cap of at most CAP_AS_REFERENCE needs no running maximum: no score is above the cap, and a query
 // always sees itself, whose score is at least minus the cap, so the probabilities are taken against the cap itself and the
-// scores are read once.  Learned sinks and the result's scale enter where a row's result is stored.
+// scores are read once; tanh is a polynomial where all scores that a warp reads together stay below NEAR times the cap (packed
+// multiply-adds, no special-function unit), else 1 - 2 / (exp(2 x) + 1).  Learned sinks and the result's scale enter where a row's result is stored.
 // Every wait on an mbarrier is bounded; a wait that runs out raises the block's abort flag,
 // which ends all roles, and the status word reports it.
 //
@@ -69,6 +70,12 @@ constexpr int NUM_THREADS = 352;     // warp 8: TMEM + MMA; warps 9, 10: TMA of 
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float RESCALE_THRESHOLD = 8.0f;
 constexpr float CAP_AS_REFERENCE = 30.0f;     // 2^(-2 cap log2(e)), the least a query's own key can weigh, times 2^-24 is still a normal 32-bit number
+// tanh(u) / u as a polynomial in u^2 for |u| <= NEAR, fitted by reweighted least squares at Chebyshev nodes: 1.6e-7 of the value in 32-bit
+constexpr float NEAR = 0.8f;
+__device__ __forceinline__ constexpr float tanh_c(int k)
+{
+    return k == 0 ? 0.99999994f : k == 1 ? -0.33332676f : k == 2 ? 0.13321048f : k == 3 ? -0.05311431f : k == 4 ? 0.0190933f : -0.004355299f;
+}
 enum { PLAIN_SCORES = 0, CAPPED_SCORES = 1, BIASED_SCORES = 2 };   // 1: capped at no more than that, with or without a bias; 2: any bias, any cap
 
 struct Params {
@@ -288,37 +295,66 @@ __global__ void __launch_bounds__(NUM_THREADS, 1) attention_tc_kernel(const __gr
                 const bool whole = __all_sync(0xffffffffu, !row_ok || (key0 >= lo && key0 + TILE - 1 <= pos));
                 const float bias0 = slope2 * (float)(key0 - pos);
                 if constexpr (SCORES == CAPPED_SCORES) {
-                    float sums[2] = {0.f, 0.f};
-#pragma unroll
+                    const float u_in = cap_in * (0.5f / LOG2E);          // from a raw score to the argument of tanh
+                    uint64_t sums = 0ull;
+#pragma unroll 1
                     for (int h = 0; h < 2; ++h) {
                         uint32_t sc[HALF];
 #pragma unroll
                         for (int c = 0; c < HALF; c += 32) tmem_load<32>(tmem_s + h * HALF + c, *reinterpret_cast<uint32_t(*)[32]>(&sc[c]));
                         tmem_wait_ld();
-                        uint32_t packed[HALF / 2];
+                        float most = 0.f;
 #pragma unroll
                         for (int i = 0; i < HALF; i += 2) {
-                            float pr[2];
+                            float u0, u1, v0, v1;
+                            const uint64_t u = mul2(pack2(__uint_as_float(sc[i]), __uint_as_float(sc[i + 1])), pack2(u_in, u_in));
+                            unpack2(u, u0, u1);
+                            unpack2(mul2(u, u), v0, v1);
+                            sc[i] = __float_as_uint(u0);
+                            sc[i + 1] = __float_as_uint(u1);
+                            most = max3(most, v0, v1);
+                        }
+                        const float base = bias0 + slope2 * (float)(h * HALF) - cap_log2;      // the score's distance to the cap, which the probabilities are taken against
+                        uint32_t packed[HALF / 2];
+                        if (!__any_sync(0xffffffffu, most > NEAR * NEAR)) {
+                            uint64_t c2[6];
 #pragma unroll
-                            for (int e = 0; e < 2; ++e) {
-                                // cap tanh(s scale / cap) - cap = -2 cap / (exp(2 s scale / cap) + 1), and the bias
-                                const float r = fast_rcp(fast_exp2(__uint_as_float(sc[i + e]) * cap_in) + 1.f);
-                                pr[e] = fast_exp2(fmaf(-2.f * cap_log2, r, fmaf((float)(h * HALF + i + e), slope2, bias0)));
-                            }
-                            if (!whole) {
+                            for (int k = 0; k < 6; ++k) c2[k] = pack2(tanh_c(k) * cap_log2, tanh_c(k) * cap_log2);
 #pragma unroll
-                                for (int e = 0; e < 2; ++e) {
-                                    const int k = key0 + h * HALF + i + e;
-                                    if (!(k <= pos && k >= lo)) pr[e] = 0.f;
-                                }
+                            for (int i = 0; i < HALF; i += 2) {
+                                const uint64_t u = pack2(__uint_as_float(sc[i]), __uint_as_float(sc[i + 1])), v = mul2(u, u);
+                                uint64_t t = fma2(v, c2[5], c2[4]);
+#pragma unroll
+                                for (int k = 3; k >= 0; --k) t = fma2(v, t, c2[k]);
+                                float a0, a1;
+                                unpack2(fma2(u, t, pack2(fmaf((float)i, slope2, base), fmaf((float)(i + 1), slope2, base))), a0, a1);
+                                sc[i] = __float_as_uint(fast_exp2(a0));
+                                sc[i + 1] = __float_as_uint(fast_exp2(a1));
                             }
-                            sums[0] += pr[0];
-                            sums[1] += pr[1];
-                            packed[i / 2] = pack_bf16(pr[0], pr[1]);
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < HALF; ++i) {
+                                const float r = fast_rcp(fast_exp2(__uint_as_float(sc[i]) * (2.f * LOG2E)) + 1.f);
+                                sc[i] = __float_as_uint(fast_exp2(fmaf(-2.f * cap_log2, r, fmaf((float)i, slope2, base + cap_log2))));
+                            }
+                        }
+                        if (!whole) {
+#pragma unroll
+                            for (int i = 0; i < HALF; ++i) {
+                                const int k = key0 + h * HALF + i;
+                                if (!(k <= pos && k >= lo)) sc[i] = 0u;
+                            }
+                        }
+#pragma unroll
+                        for (int i = 0; i < HALF; i += 2) {
+                            sums = add2(sums, pack2(__uint_as_float(sc[i]), __uint_as_float(sc[i + 1])));
+                            packed[i / 2] = pack_bf16(__uint_as_float(sc[i]), __uint_as_float(sc[i + 1]));
                         }
                         tmem_store<32>(tmem_s + h * (HALF / 2), packed);
                     }
-                    l += sums[0] + sums[1];
+                    float s0, s1;
+                    unpack2(sums, s0, s1);
+                    l += s0 + s1;
                     tmem_wait_st();
                     fence_before_sync();
                     mbar_arrive(bar_p + grp);

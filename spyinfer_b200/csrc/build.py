@@ -30,7 +30,7 @@ NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--expt-relaxed-constexpr", "-Xc
               "-Xcompiler", "-fvisibility=default"]
 HOST_MODULES = ["engine_core"]                 # plain C++, built with the host compiler
 HOST_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-shared", "-fvisibility=default"]
-MODULES = ["embedding", "rmsnorm", "residual_norm", "layernorm", "group_norm", "dynamic_tanh", "time_conv", "qkv_store", "conv_qkv", "diff_attention", "gated_scan", "moe", "sink_attention", "attention_pool", "recurrence", "head_scan", "gated_norm", "qk_rope_store", "latent", "attention_generic", "attention_mma", "attention_tc", "attention_decode", "gemm_simt", "gemm_tcgen05", "gemm_grouped", "swiglu", "sampling"]
+MODULES = ["embedding", "rmsnorm", "residual_norm", "layernorm", "group_norm", "dynamic_tanh", "time_conv", "qkv_store", "conv_qkv", "diff_attention", "gated_scan", "moe", "sink_attention", "attention_pool", "recurrence", "head_scan", "gated_norm", "qk_rope_store", "latent", "head_gemm", "attention_generic", "attention_mma", "attention_tc", "attention_decode", "gemm_simt", "gemm_tcgen05", "gemm_grouped", "swiglu", "sampling"]
 
 _loaded: Dict[str, ctypes.CDLL] = {}
 _lock = threading.Lock()

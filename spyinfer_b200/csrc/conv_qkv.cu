@@ -117,97 +117,74 @@ conv_qkv_kernel(const TP* __restrict__ proj, TQ* __restrict__ q_out, TQ* __restr
     const int width = kind == 2 ? A.vdim : A.dim;
     const int channels = A.heads * A.dim + A.kv_heads * (A.dim + A.vdim);
     const int c = (kind == 0 ? 0 : (kind == 1 ? A.heads * A.dim : (A.heads + A.kv_heads) * A.dim)) + head * width + e0;
-    const bool content = e0 < width;
-    const int hist_n = A.taps - 1;
-    float k[MAXT][V], hist[MAXT][V];          // hist[i]: the input (taps - 1 - i) tokens back; hist[taps - 1] is unused
+    const int hist_n = A.taps - 1, pad = MAXT - A.taps;          // fewer taps than MAXT: the oldest ones weigh nothing
+    const long long row_at = (long long)(kind == 2 ? A.kv_heads + head : head) * A.page_size;      // a key or value head's rows within a page
+    auto place = [&](int t) -> TQ* {
+        if (kind == 0) return q_out + ((long long)t * A.heads + head) * A.hd + e0;
+        return page_s[t - t0] >= 0 ? pages + (page_s[t - t0] + row_at) * A.hd + e0 : nullptr;
+    };
+    if (e0 >= width) {                                            // behind a row's content
+        const float zero[V] = {};
+        for (int t = t0; t < t1; ++t)
+            if (TQ* dst = place(t)) put<V>(dst, zero);
+        return;
+    }
+    // buf: the MAXT - 1 inputs ahead of a group of AHEAD tokens, and theirs; all of a group's loads are under way together
+    constexpr int AHEAD = MAXT <= 4 ? PIECE : 4, HIST = MAXT - 1;
+    float k[MAXT][V], buf[HIST + AHEAD][V];
 #pragma unroll
     for (int j = 0; j < MAXT; ++j) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) k[j][e] = hist[j][e] = 0.f;
-        if (content && j < A.taps) take<V>(A.kernel + (long long)j * channels + c, k[j]);
+        for (int e = 0; e < V; ++e) k[j][e] = 0.f;
+        if (j >= pad) take<V>(A.kernel + (long long)(j - pad) * channels + c, k[j]);
     }
     const TP* in = proj + c;
-    if (content) {
-        if (piece == 0) {
-            float* st = A.state + (long long)A.state_slot[seq] * hist_n * channels + c;
+    float* st = piece == 0 && hist_n > 0 ? A.state + (long long)A.state_slot[seq] * hist_n * channels + c : nullptr;
 #pragma unroll
-            for (int i = 0; i < MAXT - 1; ++i)
-                if (i < hist_n) take<V>(st + (long long)i * channels, hist[i]);
-            // what the next step will find: the inputs at the run's last taps - 1 places, older ones taken from the old state
-            const int n = end - start;
+    for (int i = 0; i < HIST; ++i) {
 #pragma unroll
-            for (int i = 0; i < MAXT - 1; ++i) {
-                if (i < hist_n) {
-                    const int t = end - hist_n + i;
-                    float v[V];
-                    if (t >= start) columns<V>(in + (long long)t * A.ld, A.splits, A.split_stride, v);
-                    else {
-#pragma unroll
-                        for (int e = 0; e < V; ++e) v[e] = 0.f;
-#pragma unroll
-                        for (int o = 0; o < MAXT - 1; ++o)
-                            if (o == i + n) {
-#pragma unroll
-                                for (int e = 0; e < V; ++e) v[e] = hist[o][e];
-                            }
-                    }
-                    put<V>(st + (long long)i * channels, v);
-                }
-            }
-        } else {
-#pragma unroll
-            for (int i = 0; i < MAXT - 1; ++i)
-                if (i < hist_n) columns<V>(in + (long long)(t0 - hist_n + i) * A.ld, A.splits, A.split_stride, hist[i]);
+        for (int e = 0; e < V; ++e) buf[i][e] = 0.f;
+        if (i >= pad) {
+            if (piece == 0) take<V>(st + (long long)(i - pad) * channels, buf[i]);
+            else columns<V>(in + (long long)(t0 - HIST + i) * A.ld, A.splits, A.split_stride, buf[i]);
         }
     }
-    const long long row_at = (long long)(kind == 2 ? A.kv_heads + head : head) * A.page_size;      // a key or value head's rows within a page
-    // four tokens' inputs are requested together, then used in order
-    constexpr int AHEAD = 4;
     for (int tb = t0; tb < t1; tb += AHEAD) {
-        float xs[AHEAD][V];
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u)
+            if (tb + u < t1) columns<V>(in + (long long)(tb + u) * A.ld, A.splits, A.split_stride, buf[HIST + u]);
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
+            if (tb + u < t1) {
+                float acc[V];
 #pragma unroll
-            for (int e = 0; e < V; ++e) xs[u][e] = 0.f;
-            if (content && tb + u < t1) columns<V>(in + (long long)(tb + u) * A.ld, A.splits, A.split_stride, xs[u]);
+                for (int e = 0; e < V; ++e) acc[e] = k[0][e] * buf[u][e];
+#pragma unroll
+                for (int j = 1; j < MAXT; ++j)
+#pragma unroll
+                    for (int e = 0; e < V; ++e) acc[e] = fmaf(k[j][e], buf[u + j][e], acc[e]);
+                if (kind == 0) {
+                    const float f = temp_s[tb + u - t0];
+#pragma unroll
+                    for (int e = 0; e < V; ++e) acc[e] *= f;
+                }
+                if (TQ* dst = place(tb + u)) put<V>(dst, acc);
+            }
         }
 #pragma unroll
-        for (int u = 0; u < AHEAD; ++u) {
-            const int t = tb + u;
-            if (t >= t1) break;
-            float acc[V];
+        for (int i = 0; i < HIST; ++i)
 #pragma unroll
-            for (int e = 0; e < V; ++e) acc[e] = 0.f;
-#pragma unroll
-            for (int i = 0; i < MAXT - 1; ++i)
-                if (i < hist_n) {
-#pragma unroll
-                    for (int e = 0; e < V; ++e) acc[e] = fmaf(k[i][e], hist[i][e], acc[e]);
-                }
-#pragma unroll
-            for (int j = 0; j < MAXT; ++j)
-                if (j == hist_n) {
-#pragma unroll
-                    for (int e = 0; e < V; ++e) acc[e] = fmaf(k[j][e], xs[u][e], acc[e]);
-                }
-            TQ* dst = nullptr;
-            if (kind == 0) {
-                const float f = temp_s[t - t0];
-#pragma unroll
-                for (int e = 0; e < V; ++e) acc[e] *= f;
-                dst = q_out + ((long long)t * A.heads + head) * A.hd + e0;
-            } else if (page_s[t - t0] >= 0) {
-                dst = pages + (page_s[t - t0] + row_at) * A.hd + e0;
-            }
-            if (dst != nullptr) put<V>(dst, acc);
-#pragma unroll
-            for (int i = 0; i < MAXT - 1; ++i) {
-#pragma unroll
-                for (int e = 0; e < V; ++e) {
-                    if (i + 1 < hist_n) hist[i][e] = hist[i + 1][e];
-                    else if (i + 1 == hist_n) hist[i][e] = xs[u][e];
-                }
-            }
+            for (int e = 0; e < V; ++e) buf[i][e] = buf[AHEAD + i][e];
+    }
+    if (piece == 0) {
+        // what the next step will find: the inputs at the run's last taps - 1 places, older ones moved up from the old state
+        const int n = end - start;
+        for (int i = 0; i < hist_n; ++i) {
+            const int t = end - hist_n + i;
+            float v[V];
+            if (t >= start) columns<V>(in + (long long)t * A.ld, A.splits, A.split_stride, v);
+            else take<V>(st + (long long)(i + n) * channels, v);
+            put<V>(st + (long long)i * channels, v);
         }
     }
 }

@@ -31,9 +31,9 @@ __device__ __forceinline__ float rotated(const float* x, int j, int rot_half, in
     return first ? u * c - v * s : v * c + u * s;
 }
 
-template <typename TO, typename TC>
+template <typename TF, typename TO, typename TC>
 __global__ void __launch_bounds__(PREP_THREADS)
-latent_prep_kernel(const float* __restrict__ fused, long long ld, int off_q, int q_rank, const float* __restrict__ wq, TO* __restrict__ cq_out,
+latent_prep_kernel(const TF* __restrict__ fused, long long ld, int off_q, int q_rank, const float* __restrict__ wq, TO* __restrict__ cq_out,
                    int off_c, int kv_rank, const float* __restrict__ wc, int rot_dim, const float* __restrict__ rope, int rot_half, int table_rows,
                    int interleaved, const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
                    int table_width, TC* __restrict__ pages, int page_size, int num_pages, int planes, float eps, int* status)
@@ -43,13 +43,13 @@ latent_prep_kernel(const float* __restrict__ fused, long long ld, int off_q, int
     float* rot_s = sm;
     float* scratch = sm + rot_dim;
     const int t = blockIdx.x, tid = threadIdx.x;
-    const float* row = fused + (size_t)t * ld;
+    const TF* row = fused + (size_t)t * ld;
     if (q_rank > 0) {
         float ss = 0.f;
-        for (int i = tid; i < q_rank; i += PREP_THREADS) ss = fmaf(row[off_q + i], row[off_q + i], ss);
+        for (int i = tid; i < q_rank; i += PREP_THREADS) ss = fmaf(to_f32(row[off_q + i]), to_f32(row[off_q + i]), ss);
         ss = block_sum(ss, scratch);
         const float inv = 1.0f / sqrtf(ss / (float)q_rank + eps);
-        for (int i = tid; i < q_rank; i += PREP_THREADS) cq_out[(size_t)t * q_rank + i] = from_f32<TO>((row[off_q + i] * inv) * wq[i]);
+        for (int i = tid; i < q_rank; i += PREP_THREADS) cq_out[(size_t)t * q_rank + i] = from_f32<TO>((to_f32(row[off_q + i]) * inv) * wq[i]);
     }
     if (off_c < 0) return;
     const int pos = positions[t], seq = seq_of_token[t];
@@ -64,19 +64,19 @@ latent_prep_kernel(const float* __restrict__ fused, long long ld, int off_q, int
     const int width = kv_rank + rot_dim;
     TC* dst = pages + (((size_t)page * planes) * page_size + pos % page_size) * width;     // plane 0 of the page's one key/value head
     float ss = 0.f;
-    for (int i = tid; i < kv_rank; i += PREP_THREADS) ss = fmaf(row[off_c + i], row[off_c + i], ss);
-    for (int j = tid; j < rot_dim; j += PREP_THREADS) rot_s[j] = row[off_c + kv_rank + j];
+    for (int i = tid; i < kv_rank; i += PREP_THREADS) ss = fmaf(to_f32(row[off_c + i]), to_f32(row[off_c + i]), ss);
+    for (int j = tid; j < rot_dim; j += PREP_THREADS) rot_s[j] = to_f32(row[off_c + kv_rank + j]);
     ss = block_sum(ss, scratch);            // its barriers also publish rot_s
     const float inv = 1.0f / sqrtf(ss / (float)kv_rank + eps);
-    for (int i = tid; i < kv_rank; i += PREP_THREADS) dst[i] = from_f32<TC>((row[off_c + i] * inv) * wc[i]);
+    for (int i = tid; i < kv_rank; i += PREP_THREADS) dst[i] = from_f32<TC>((to_f32(row[off_c + i]) * inv) * wc[i]);
     const float* cs = rope + (size_t)(rot_half ? pos : 0) * rot_half * 2;
     for (int j = tid; j < rot_dim; j += PREP_THREADS) dst[kv_rank + j] = from_f32<TC>(rotated(rot_s, j, rot_half, interleaved, cs));
 }
 
-// fused [T, ld] float32: the query latent before its norm at off_q (q_rank columns; 0: none), the key/value latent and the
+// fused [T, ld] of fused_dtype: the query latent before its norm at off_q (q_rank columns; 0: none), the key/value latent and the
 // shared key part at off_c (kv_rank + rot_dim columns; off_c < 0: this layer stores nothing).  cq_out [T, q_rank].
 // pages [num_pages][planes][1][page_size][kv_rank + rot_dim].  rope [table_rows][rot_half][2] or null with rot_half 0.
-extern "C" int spy_latent_prep(const float* fused, long long ld, int off_q, int q_rank, const float* wq, void* cq_out, int out_dtype, int off_c,
+extern "C" int spy_latent_prep(const void* fused, int fused_dtype, long long ld, int off_q, int q_rank, const float* wq, void* cq_out, int out_dtype, int off_c,
                                int kv_rank, const float* wc, int rot_dim, const float* rope, int rot_half, int table_rows, int interleaved,
                                const int* positions, const int* seq_of_token, const int* block_table, int table_width, void* pages, int cache_dtype,
                                int page_size, int num_pages, int planes, float eps, int tokens, int* status, cudaStream_t stream)
@@ -89,12 +89,14 @@ extern "C" int spy_latent_prep(const float* fused, long long ld, int off_q, int 
         if (page_size <= 0 || num_pages <= 0 || table_width <= 0 || (planes != 1 && planes != 2)) SPY_FAIL("latent_prep: page_size, num_pages, table_width must be positive and planes 1 or 2");
     }
     const size_t smem = (size_t)((rot_dim > 0 ? rot_dim : 0) + 33) * sizeof(float);
+    SPY_DISPATCH_DTYPE(fused_dtype, TF, {
     SPY_DISPATCH_DTYPE(out_dtype, TO, {
         SPY_DISPATCH_DTYPE(cache_dtype, TC, {
-            spy_launch(latent_prep_kernel<TO, TC>, dim3(tokens), dim3(PREP_THREADS), smem, stream, fused, ld, off_q, q_rank, wq, (TO*)cq_out, off_c, kv_rank, wc,
+            spy_launch(latent_prep_kernel<TF, TO, TC>, dim3(tokens), dim3(PREP_THREADS), smem, stream, (const TF*)fused, ld, off_q, q_rank, wq, (TO*)cq_out, off_c, kv_rank, wc,
                        rot_dim, rope, rot_half, table_rows, interleaved, positions, seq_of_token, block_table, table_width, (TC*)pages, page_size, num_pages,
                        planes, eps, status);
         })
+    })
     })
     SPY_CHECK_LAUNCH("latent_prep");
     return 0;
@@ -106,7 +108,7 @@ struct HeadProductArgs {
     void* out;       long long out_ld; int out_head_stride;
     int tail;                 // elements after each head's K inputs that go, rotated, to the columns after its N outputs
     const float* rope; int rot_half, table_rows, interleaved; const int* positions;
-    const float* gate; long long gate_ld; int gate_off;      // null, or out *= sigmoid(gate[t, gate_off + h * N + n])
+    const void* gate; int gate_dtype; long long gate_ld; int gate_off;      // null, or out *= sigmoid(gate[t, gate_off + h * N + n])
     int T;
     int* status;
 };
@@ -177,7 +179,8 @@ __global__ void __launch_bounds__(128) head_product_kernel(HeadProductArgs A)
             if (u < n_tok) {
                 float r = acc[u];
                 if (A.gate != nullptr) {
-                    const float g = A.gate[(size_t)(t0 + u) * A.gate_ld + A.gate_off + (size_t)h * A.N + n];
+                    const size_t at = (size_t)(t0 + u) * A.gate_ld + A.gate_off + (size_t)h * A.N + n;
+                    const float g = A.gate_dtype == SPY_BF16 ? to_f32(((const bf16*)A.gate)[at]) : ((const float*)A.gate)[at];
                     r *= 1.0f / (1.0f + expf(-g));
                 }
                 out[(size_t)(t0 + u) * A.out_ld + (size_t)h * A.out_head_stride + n] = from_f32<TA>(r);
@@ -215,8 +218,8 @@ __global__ void __launch_bounds__(128) head_product_kernel(HeadProductArgs A)
 // float32: a part of a projection that was left in 32-bit), out act_dtype.
 extern "C" int spy_head_product(const void* in, int in_dtype, long long in_ld, int in_head_stride, int K, const void* W, int w_dtype, int N, void* out, long long out_ld,
                                 int out_head_stride, int act_dtype, int tail, const float* rope, int rot_half, int table_rows, int interleaved,
-                                const int* positions, const float* gate, long long gate_ld, int gate_off, int tokens, int heads, int* status,
-                                cudaStream_t stream)
+                                const int* positions, const void* gate, int gate_dtype, long long gate_ld, int gate_off, int tokens, int heads,
+                                int* status, cudaStream_t stream)
 {
     if (tokens <= 0) return 0;
     if (heads <= 0 || heads > 65535 || K <= 0 || N <= 0 || tail < 0) SPY_FAIL("head_product: %d heads, K %d, N %d, tail %d", heads, K, N, tail);
@@ -226,7 +229,7 @@ extern "C" int spy_head_product(const void* in, int in_dtype, long long in_ld, i
     const size_t smem = ((size_t)(nt + 4) * (K + tail) + (size_t)KC * NC) * sizeof(float);
     if (smem > 160 * 1024) SPY_FAIL("head_product: %d inputs a head do not fit a block's shared memory", K + tail);
     HeadProductArgs A = {in, in_ld, in_head_stride, K, W, N, out, out_ld, out_head_stride, tail, rope, rot_half, table_rows, interleaved, positions,
-                         gate, gate_ld, gate_off, tokens, status};
+                         gate, gate_dtype, gate_ld, gate_off, tokens, status};
     if (in_dtype != act_dtype && in_dtype != SPY_F32) SPY_FAIL("head_product: inputs of dtype code %d for results of dtype code %d", in_dtype, act_dtype);
     auto run = [&](auto kernel) -> cudaError_t {
         if (smem > 48 * 1024) {

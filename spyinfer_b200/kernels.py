@@ -928,13 +928,13 @@ def latent_prep(fused: torch.Tensor, q_offset: int, q_rank: int, q_weight: Optio
                 c_weight: Optional[torch.Tensor], rot_dim: int, rope_table: Optional[torch.Tensor], interleaved: bool, positions: torch.Tensor,
                 seq_of_token: torch.Tensor, block_table: Optional[torch.Tensor], pages: Optional[torch.Tensor], eps: float,
                 status: Optional[torch.Tensor] = None) -> None:
-    """The norms and the cache store of attention through a latent.  ``fused [T, ld]`` float32 holds, from column ``q_offset``,
+    """The norms and the cache store of attention through a latent.  ``fused [T, ld]`` (float32 or bfloat16) holds, from column ``q_offset``,
     the query latent (``q_rank`` columns; RMS-normed with ``q_weight`` into ``cq_out [T, q_rank]``) and, from ``c_offset``
     (negative: nothing is stored), the key/value latent (``kv_rank`` columns, RMS-normed with ``c_weight``) followed by the
     shared key part (``rot_dim`` columns, rotated by ``rope_table [positions, r, 2]``: pairs ``(j, j + r)`` or, ``interleaved``,
     ``(2j, 2j + 1)``).  The row ``[latent | rotated part]`` goes to plane 0 of ``pages [num_pages, planes, 1, page_size,
     kv_rank + rot_dim]`` through ``block_table``."""
-    _check(fused, "fused projection", torch.float32, 2)
+    _check(fused, "fused projection", ndim=2)
     T, ld = fused.shape
     _check(positions, "positions", torch.int32, 1)
     _check(seq_of_token, "seq_of_token", torch.int32, 1)
@@ -961,7 +961,7 @@ def latent_prep(fused: torch.Tensor, q_offset: int, q_rank: int, q_weight: Optio
             table_rows, rot_half = rope_table.shape[0], rope_table.shape[1]
             if 2 * rot_half > rot_dim:
                 raise KernelError(f"latent_prep: {rot_half} rotated pairs do not fit a rotated part of {rot_dim}")
-    _call("latent", "spy_latent_prep", _ptr(fused), ctypes.c_longlong(ld), int(q_offset), int(q_rank), _ptr(q_weight), _ptr(cq_out), out_code, int(c_offset),
+    _call("latent", "spy_latent_prep", _ptr(fused), _code(fused, "fused projection"), ctypes.c_longlong(ld), int(q_offset), int(q_rank), _ptr(q_weight), _ptr(cq_out), out_code, int(c_offset),
           int(kv_rank), _ptr(c_weight), int(rot_dim), _ptr(rope_table), rot_half, table_rows, int(bool(interleaved)), _ptr(positions), _ptr(seq_of_token),
           _ptr(block_table if c_offset >= 0 else None), width, _ptr(pages if c_offset >= 0 else None), cache_code, page_size, num_pages, planes,
           ctypes.c_float(eps), T, _ptr(status), _stream())
@@ -973,7 +973,7 @@ def head_product(x: torch.Tensor, in_head_stride: int, weight: torch.Tensor, out
     """``out[t, h * out_head_stride + n] = sum_k weight[h, k, n] * x[t, h * in_head_stride + k]`` (32-bit sums) for a weight
     ``[heads, K, N]``; x and out ``[T, >= heads * stride]`` of one dtype, or x float32.  ``tail`` elements that follow each head's K inputs go,
     rotated by ``rope_table`` at the token's position (pairs as in ``latent_prep``), to the columns after its N results.
-    ``gate`` (float32 ``[T, ld]``): the results are multiplied by ``sigmoid(gate[t, gate_offset + h * N + n])``."""
+    ``gate`` (``[T, ld]``): the results are multiplied by ``sigmoid(gate[t, gate_offset + h * N + n])``."""
     _check(x, "head_product input", ndim=2)
     _check(out, "head_product output", x.dtype if x.dtype != torch.float32 else None, 2)
     _check(weight, "head_product weight", ndim=3)
@@ -994,14 +994,56 @@ def head_product(x: torch.Tensor, in_head_stride: int, weight: torch.Tensor, out
                 raise KernelError(f"head_product: {rot_half} rotated pairs do not fit a tail of {tail}")
     gate_ld = 0
     if gate is not None:
-        _check(gate, "gate", torch.float32, 2)
+        _check(gate, "gate", ndim=2)
         gate_ld = gate.shape[1]
         if gate.shape[0] != T or gate_offset < 0 or gate_offset + H * N > gate_ld:
             raise KernelError("head_product: the gate's columns do not fit")
     _call("latent", "spy_head_product", _ptr(x), _code(x, "head_product input"), ctypes.c_longlong(x.shape[1]), int(in_head_stride), K, _ptr(weight),
           _code(weight, "head_product weight"), N, _ptr(out), ctypes.c_longlong(out.shape[1]), int(out_head_stride), _code(out, "head_product output"), int(tail), _ptr(rope_table), rot_half, table_rows,
-          int(bool(interleaved)), _ptr(positions), _ptr(gate), ctypes.c_longlong(gate_ld), int(gate_offset), T, H, _ptr(status), _stream())
+          int(bool(interleaved)), _ptr(positions), _ptr(gate), _code(gate, "gate") if gate is not None else 0, ctypes.c_longlong(gate_ld), int(gate_offset), T, H, _ptr(status), _stream())
     return out
+
+
+def head_gemm(x: torch.Tensor, in_head_stride: int, weight: torch.Tensor, out: torch.Tensor, out_head_stride: int, tail: int = 0,
+                 rope_table: Optional[torch.Tensor] = None, interleaved: bool = False, positions: Optional[torch.Tensor] = None,
+                 gate: Optional[torch.Tensor] = None, gate_offset: int = 0, status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``head_product`` on the tensor cores: bfloat16 throughout, the weight laid out ``[heads, N, K]``; K, the input's pitch and its head
+    stride are multiples of 8 (``head_gemm_takes``)."""
+    _check(x, "head_gemm input", torch.bfloat16, 2)
+    _check(out, "head_gemm output", torch.bfloat16, 2)
+    _check(weight, "head_gemm weight", torch.bfloat16, 3)
+    H, N, K = weight.shape
+    if status is None:
+        status = status_word(x.device)
+    T = x.shape[0]
+    if (out.shape[0] != T or in_head_stride < K + tail or out_head_stride < N + tail or (H - 1) * in_head_stride + K + tail > x.shape[1]
+            or (H - 1) * out_head_stride + N + tail > out.shape[1]):
+        raise KernelError(f"head_gemm: input {tuple(x.shape)}, weight {tuple(weight.shape)}, output {tuple(out.shape)} and the strides do not fit")
+    rot_half = table_rows = 0
+    if tail > 0:
+        _check(positions, "positions", torch.int32, 1)
+        if positions.shape[0] != T:
+            raise KernelError("head_gemm: positions must have one entry per token")
+        if rope_table is not None:
+            _check(rope_table, "rope table", torch.float32, 3)
+            table_rows, rot_half = rope_table.shape[0], rope_table.shape[1]
+            if 2 * rot_half > tail:
+                raise KernelError(f"head_gemm: {rot_half} rotated pairs do not fit a tail of {tail}")
+    gate_ld = 0
+    if gate is not None:
+        _check(gate, "gate", ndim=2)
+        gate_ld = gate.shape[1]
+        if gate.shape[0] != T or gate_offset < 0 or gate_offset + H * N > gate_ld:
+            raise KernelError("head_gemm: the gate's columns do not fit")
+    _call("head_gemm", "spy_head_gemm", _ptr(x), ctypes.c_longlong(x.shape[1]), int(in_head_stride), K, _ptr(weight), N, _ptr(out), ctypes.c_longlong(out.shape[1]),
+          int(out_head_stride), int(tail), _ptr(rope_table), rot_half, table_rows, int(bool(interleaved)), _ptr(positions), _ptr(gate),
+          _code(gate, "gate") if gate is not None else 0, ctypes.c_longlong(gate_ld), int(gate_offset), T, H, _ptr(status), _stream())
+    return out
+
+
+def head_gemm_takes(K: int, pitch: int, head_stride: int) -> bool:
+    """Whether the tensor-core kernel takes per-head products of these sizes (16-byte borders; any number of outputs and tokens)."""
+    return K > 0 and K % 8 == 0 and pitch % 8 == 0 and head_stride % 8 == 0
 
 
 def sample(logits: torch.Tensor, tokens: torch.Tensor, temperature: Optional[torch.Tensor] = None, seed: Optional[torch.Tensor] = None,

@@ -359,6 +359,7 @@ class LatentAttention(Attention):
         self.c_offset = self.q_rank if self.q_rank is not None else self.nh * (self.d + self.rd)
         self.gate_offset = self.c_offset + (0 if self.shares_cache else self.width)
         self.fused = self.uq = self.uk = self.uv = self.q_norm_w = self.c_norm_w = None
+        self.tc_absorb = self.tc_expand = False
 
     def weight_decls(self):
         p, H, W = self.prefix, self.nh, self.hidden
@@ -385,13 +386,19 @@ class LatentAttention(Attention):
             self.q_norm_w = tensors[p + "dq.norm"].float().contiguous()
         self.bind_scores(tensors)
         self.o = Linear(tensors[p + "o"], self.ctx.dtype)
-        self.uk = tensors[p + "uk"].reshape(H, self.d, self.kv_rank).contiguous()                      # [head][unrotated element][latent]: as stored
-        self.uv = tensors[p + "uv"].reshape(H, self.vd, self.kv_rank).transpose(1, 2).contiguous()     # [head][latent][value element]
+        uk, uv = tensors[p + "uk"].reshape(H, self.d, self.kv_rank), tensors[p + "uv"].reshape(H, self.vd, self.kv_rank)
+        # the per-head products on the tensor cores want a head's outputs as rows, the plain kernel its inputs
+        bf16 = self.ctx.dtype == torch.bfloat16
+        q_pitch = self.fused.out_features if self.uq is None else self.uq.out_features
+        self.tc_absorb = bf16 and uk.dtype == torch.bfloat16 and kernels.head_gemm_takes(self.d, q_pitch, self.d + self.rd)
+        self.tc_expand = bf16 and uv.dtype == torch.bfloat16 and kernels.head_gemm_takes(self.kv_rank, H * self.width, self.width)
+        self.uk = (uk.transpose(1, 2) if self.tc_absorb else uk).contiguous()          # [head][latent][unrotated element], or as stored
+        self.uv = (uv if self.tc_expand else uv.transpose(1, 2)).contiguous()          # as stored, or [head][latent][value element]
         if not self.shares_cache:
             self.c_norm_w = tensors[p + "dkv.norm"].float().contiguous()
 
     def modules(self):
-        mods = ["latent"] + (["attention_tc", "attention_decode"] if self.tc else []) + ["attention_generic"]
+        mods = ["latent"] + (["head_gemm"] if self.tc_absorb or self.tc_expand else []) + (["attention_tc", "attention_decode"] if self.tc else []) + ["attention_generic"]
         for lin in self.linears():
             mods += lin.modules()
         if self.position is not None:
@@ -411,19 +418,22 @@ class LatentAttention(Attention):
             raise ValueError("latent_attention: a layer with a key/value projection of its own owns its cache, one without reads another layer's")
         T, H = x.shape[0], self.nh
         interleaved = self.position is not None and self.position.pairing == "interleaved"
-        fused = self.fused(x, out_dtype=torch.float32)
+        # what the query latent's norm reads stays in 32-bit; queries that need no norm are rounded as any activation
+        fused = self.fused(x, out_dtype=torch.float32 if self.q_rank is not None else None)
         cq = torch.empty((T, self.q_rank), dtype=x.dtype, device=x.device) if self.q_rank is not None else None
         if cq is not None or cache.writes:
             kernels.latent_prep(fused, 0, self.q_rank or 0, self.q_norm_w, cq, self.c_offset if cache.writes else -1, self.kv_rank, self.c_norm_w, self.rd,
                                 self.rope_table, interleaved, batch.positions, batch.seq_of_token, cache.block_table, cache.pages, self.eps, status=batch.status)
         q = self.uq(cq) if cq is not None else fused          # without a query latent the queries are the projection's first columns
         q_abs = torch.empty((T, H * self.width), dtype=x.dtype, device=x.device)
-        kernels.head_product(q, self.d + self.rd, self.uk, q_abs, self.width, tail=self.rd, rope_table=self.rope_table, interleaved=interleaved,
-                             positions=batch.positions, status=batch.status)
+        absorb = kernels.head_gemm if self.tc_absorb else kernels.head_product
+        absorb(q, self.d + self.rd, self.uk, q_abs, self.width, tail=self.rd, rope_table=self.rope_table, interleaved=interleaved,
+               positions=batch.positions, status=batch.status)
         mixed = torch.empty((T, H * self.width), dtype=x.dtype, device=x.device)      # per head: [sum p c | sum p k_r]; the second part is not used
         self.attend(q_abs, mixed, batch, cache)
         o = torch.empty((T, H * self.vd), dtype=x.dtype, device=x.device)
-        kernels.head_product(mixed, self.width, self.uv, o, self.vd, gate=fused if self.gated else None, gate_offset=self.gate_offset)
+        expand = kernels.head_gemm if self.tc_expand else kernels.head_product
+        expand(mixed, self.width, self.uv, o, self.vd, gate=fused if self.gated else None, gate_offset=self.gate_offset, status=batch.status)
         return self.o(o, defer=self.defer_output)
 
 

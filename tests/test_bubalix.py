@@ -593,6 +593,69 @@ def test_the_absorbed_query_of_a_projection_left_in_32_bit(dtype, heads, dim, ro
 
 
 @gpu
+@pytest.mark.parametrize("gate_dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("T", [1, 128, 300])
+@pytest.mark.parametrize("heads,dim,rot_dim,kv_rank,vdim,pairing", [(4, 32, 32, 64, 40, "half"), (16, 128, 32, 96, 128, "half"), (3, 8, 8, 24, 12, "interleaved"),
+                                                                    (2, 64, 0, 512, 100, "half"), (1, 200, 24, 136, 300, "half"), (5, 16, 16, 40, 7, "interleaved")])
+def test_per_head_products_on_the_tensor_cores(heads, dim, rot_dim, kv_rank, vdim, pairing, T, gate_dtype):
+    """The same two products by the kernel that the bfloat16 path uses where the sizes allow: one and several tiles of tokens, blocks
+    of inputs (also more of them than are held at a time) and outputs, sizes that fill no tile, rows beyond the batch untouched."""
+    from spyinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(heads + dim + T)
+    qw, row = heads * (dim + rot_dim), kv_rank + rot_dim
+    bf = lambda *shape: torch.randn(*shape, generator=g).to(torch.bfloat16)
+    q, uk, uv, gate = bf(T, qw + 16), bf(heads, kv_rank, dim), bf(heads, vdim, kv_rank), torch.randn(T, 5 + heads * vdim, generator=g).to(gate_dtype)
+    assert kernels.head_gemm_takes(dim, qw + 16, dim + rot_dim) and kernels.head_gemm_takes(kv_rank, heads * row, row)
+    pos = torch.randint(0, 200, (T,), generator=g, dtype=torch.int32)
+    table, x = None, q.double()[:, :qw].reshape(T, heads, dim + rot_dim)
+    tail = x[..., dim:]
+    if rot_dim:
+        rot = {"base": 700.0, "dims": rot_dim}
+        ang = torch.arange(200, dtype=P.F)[:, None] * torch.tensor(P.stretched_frequencies(rot)[0], dtype=P.F)[None]
+        table = torch.stack([torch.cos(ang), torch.sin(ang)], dim=-1).float().cuda()
+        order = list(range(rot_dim)) if pairing == "half" else [e for e in range(0, rot_dim, 2)] + [e for e in range(1, rot_dim, 2)]
+        tail = P.rotate_halves(tail[..., order], pos, rot)[..., [order.index(e) for e in range(rot_dim)]]
+    want = torch.cat([torch.einsum("thd,hrd->thr", x[..., :dim], uk.double()), tail], dim=-1)
+    out = torch.full((T + 1, heads * row), 3.0, dtype=torch.bfloat16, device="cuda")
+    kernels.head_gemm(q.cuda(), dim + rot_dim, uk.cuda(), out[:T], row, tail=rot_dim, rope_table=table, interleaved=pairing == "interleaved", positions=pos.cuda())
+    tol = lambda w: dict(atol=2e-2 * float(w.abs().max()) ** 0.5, rtol=1e-2)
+    assert torch.allclose(out[:T].cpu().double().reshape(T, heads, row), want, **tol(want)) and bool((out[T] == 3.0).all())
+    mixed = bf(T, heads, row)
+    want = torch.einsum("thr,hvr->thv", mixed.double()[..., :kv_rank], uv.double()) * torch.sigmoid(gate.double()[:, 5:]).reshape(T, heads, vdim)
+    o = torch.full((T + 1, heads * vdim), 3.0, dtype=torch.bfloat16, device="cuda")
+    kernels.head_gemm(mixed.reshape(T, -1).cuda(), row, uv.cuda(), o[:T], vdim, gate=gate.cuda(), gate_offset=5)
+    assert torch.allclose(o[:T].cpu().double().reshape(T, heads, vdim), want, **tol(want)) and bool((o[T] == 3.0).all())
+
+
+@gpu
+@pytest.mark.parametrize("cap", [4.0, 25.0])
+def test_capped_scores_near_and_far_from_the_cap(cap):
+    """Prompt portions whose scores all stay well below the cap, all lie near it, or change from one to the other along the sequence:
+    the two ways in which the kernel for portions forms them agree with the plain scores."""
+    from spyinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(8)
+    T, hd = 400, 64
+    table, pages = _paged_setup([T], 16, 1, hd, torch.bfloat16)
+    k, v, base = (torch.randn(T, 1, hd, generator=g).to(torch.bfloat16) for _ in range(3))
+    pages_h = pages.cpu()
+    for j in range(T):
+        page = int(table[0, j // 16])
+        pages_h[page, 0, :, j % 16], pages_h[page, 1, :, j % 16] = k[j], v[j]
+    pages.copy_(pages_h)
+    pos = torch.arange(T, dtype=torch.int32)
+    for size in (torch.full((T, 1, 1), 0.1), torch.full((T, 1, 1), 5.0), torch.linspace(0.01, 4.0, T).reshape(T, 1, 1)):
+        q = (base.float() * size * cap / hd ** 0.5).to(torch.bfloat16)
+        s = _score(q.double(), k.double(), 1.0, cap, torch.tensor([0.01], dtype=P.F), pos, pos)[0]
+        want = P.softmax_with_sink(s, P.visibility(T, None), None) @ v.double()[:, 0]
+        out = torch.empty((T, hd), dtype=torch.bfloat16, device="cuda")
+        kernels.attention_tc(q.reshape(T, hd).cuda(), 1, hd, out, pages, table, pos.cuda(), torch.tensor([0, T], dtype=torch.int32).cuda(), 1, 1.0, softcap=cap,
+                             slopes=torch.tensor([0.01]).cuda())
+        assert float((out.cpu().double() - want).abs().max()) < 3e-2
+
+
+@gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("experts,top,ff,shared", [(6, 2, 24, 40), (4, 1, 16, 0), (5, 5, 12, 7), (64, 8, 8, 16), (3, 2, 10, 6)])
 def test_experts_by_table_weights_activations_and_pairs(dtype, experts, top, ff, shared):
