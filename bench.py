@@ -601,8 +601,7 @@ def daronex_workload(args) -> int:
                 rate("kernels_decode_b64", "recurrence.spy_gla_scan", nbytes=64.0 * 2 * z["gla_heads"] * 128 * 256 * 4 * n_gla)
                 # the absorbed query and the value expansion: two per-head products a latent layer
                 hp = 2.0 * T * H * (z["dim"] * z["kv_rank"] + z["kv_rank"] * z["vdim"]) * (n_full + n_win)
-                rate("kernels_prefill", "latent.spy_head_product", flops=hp)
-                rate("kernels_prefill", "gemm_tcgen05.spy_gemm_tcgen05_ex", flops=hp)      # where the per-head products run on the tensor cores, they are among these
+                rate("kernels_prefill", "head_gemm.spy_head_gemm", flops=hp)
                 # the norm on a sublayer's output: reads the result (bfloat16 or 32-bit parts) and the stream, writes the stream and its bfloat16 copy
                 rate("kernels_prefill", "residual_norm.spy_residual_norm", nbytes=float(2 * layers) * T * W * (4 + 4 + 4 + 2))
                 rate("kernels_prefill", "swiglu.spy_activation", nbytes=float(layers) * T * z["ff"] * 4)
@@ -997,7 +996,7 @@ def bubalix_workload(args) -> int:
                     rate(block, dec, nbytes=lat_bytes)
                     rate(block, "residual_norm.spy_residual_norm", nbytes=float(2 * layers) * rows * W * (4 + 4 + 4 + 2))
                 if name != "qwen3":
-                    rate(block, "latent.spy_head_product", flops=product * rows)
+                    rate(block, "head_gemm.spy_head_gemm", flops=product * rows)
                     rate(block, "latent.spy_latent_prep", nbytes=float(rows) * n_lat * row * 6)
 
         return _measure_design(args, cfg_json, vocab, page, T, ctx, annotate, tell_apart if name == "bubalix" else None)

@@ -45,6 +45,67 @@ __device__ __forceinline__ float rotated(const bf16* x, int j, int rot_half, int
     return first ? u * c - v * s : v * c + u * s;
 }
 
+// eight neighbouring elements from a 16-byte border
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8])
+{
+    const uint4 x = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = __uint_as_float(w[i] << 16);
+        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void load8(const float* p, float (&v)[8])
+{
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void store8(bf16* p, const float (&v)[8])
+{
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+}
+
+// The rotated tail of one token's head.  `vec`: the tail, its rotated pairs and the rows are multiples of eight elements.
+__device__ __forceinline__ void store_tail(const Args& A, const bf16* x, bf16* out, const float* cs, bool vec)
+{
+    if (!vec) {
+        for (int j = 0; j < A.tail; ++j) out[j] = __float2bfloat16_rn(rotated(x, j, A.rot_half, A.interleaved, cs));
+        return;
+    }
+    float c[2][8];
+    if (!A.interleaved) {
+        for (int a = 0; a < A.rot_half; a += 8) {
+            float u[8], v[8], ru[8], rv[8];
+            load8(x + a, u);
+            load8(x + A.rot_half + a, v);
+            load8(cs + 2 * a, c[0]);
+            load8(cs + 2 * a + 8, c[1]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float co = c[i >> 2][2 * (i & 3)], si = c[i >> 2][2 * (i & 3) + 1];
+                ru[i] = u[i] * co - v[i] * si;
+                rv[i] = v[i] * co + u[i] * si;
+            }
+            store8(out + a, ru);
+            store8(out + A.rot_half + a, rv);
+        }
+    } else {
+        for (int j = 0; j < 2 * A.rot_half; j += 8) {
+            float u[8], ru[8];
+            load8(x + j, u);
+            load8(cs + j, c[0]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                ru[2 * i] = u[2 * i] * c[0][2 * i] - u[2 * i + 1] * c[0][2 * i + 1];
+                ru[2 * i + 1] = u[2 * i + 1] * c[0][2 * i] + u[2 * i] * c[0][2 * i + 1];
+            }
+            store8(out + j, ru);
+        }
+    }
+    for (int j = 2 * A.rot_half; j < A.tail; j += 8) *reinterpret_cast<uint4*>(out + j) = *reinterpret_cast<const uint4*>(x + j);
+}
+
 __global__ void __launch_bounds__(NUM_THREADS)
 head_gemm_kernel(const __grid_constant__ CUtensorMap map_in, const __grid_constant__ CUtensorMap map_w, const Args A)
 {
@@ -119,8 +180,8 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap map_in, const __grid_consta
             else {
                 const bf16* x = A.in + (size_t)t * A.in_ld + (size_t)h * A.in_head_stride + A.K;
                 const float* cs = A.rope + (size_t)(A.rot_half ? pos : 0) * A.rot_half * 2;
-#pragma unroll 8
-                for (int j = 0; j < A.tail; ++j) out[A.N + j] = __float2bfloat16_rn(rotated(x, j, A.rot_half, A.interleaved, cs));
+                const bool vec = A.tail % 8 == 0 && A.rot_half % 8 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out + A.N) | reinterpret_cast<uintptr_t>(cs)) & 15) == 0;
+                store_tail(A, x, out + A.N, cs, vec);
             }
         }
         if (mbar_wait(acc_full, 0, abort_flag)) {
@@ -133,7 +194,18 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap map_in, const __grid_consta
                 tmem_wait_ld();
                 if (!row_ok) continue;
                 const int valid = min(32, A.N - n0 - c);
-                if (A.gate != nullptr) {
+                const size_t gate_c = gate_at + n0 + c;
+                const bool gate_bf16 = A.gate_dtype == SPY_BF16;
+                if (A.gate != nullptr && valid == 32 && (((reinterpret_cast<uintptr_t>(A.gate) + gate_c * (gate_bf16 ? 2 : 4)) & 15) == 0)) {
+                    float g[4][8];
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        if (gate_bf16) load8((const bf16*)A.gate + gate_c + 8 * i, g[i]);
+                        else load8((const float*)A.gate + gate_c + 8 * i, g[i]);
+                    }
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * (1.0f / (1.0f + expf(-g[i >> 3][i & 7]))));
+                } else if (A.gate != nullptr) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
                         if (i < valid) {
