@@ -208,7 +208,7 @@ extern "C" int spy_conv_qkv_store(const void* proj, int proj_dtype, long long ld
     const ConvArgs A = {ld, split_stride, splits, kernel, state, q_start, state_slot, positions, block_table, table_width, page_size, num_pages,
                         heads, kv_heads, dim, vdim, hd, taps, pieces, temp_coef, temp_every, gate_col, gate_out, status};
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    const bool vec = dim % 4 == 0 && vdim % 4 == 0 && hd % 4 == 0 && ld % 4 == 0 && split_stride % 4 == 0 && aligned(proj) && aligned(kernel) && aligned(state)
+    const bool vec = taps <= 4 && dim % 4 == 0 && vdim % 4 == 0 && hd % 4 == 0 && ld % 4 == 0 && split_stride % 4 == 0 && aligned(proj) && aligned(kernel) && aligned(state)
                      && aligned(q_out) && aligned(pages);
     const long long items = (long long)(heads + 2 * kv_heads) * hd / (vec ? 4 : 1) + (gate_out != nullptr ? heads : 0), blocks = (long long)seqs * pieces;
     if ((items + 127) / 128 > 65535 || blocks > 0x7fffffffLL) SPY_FAIL("conv_qkv: %lld elements a token, %d requests of up to %d tokens exceed the grid", items, seqs, longest);
@@ -216,7 +216,7 @@ extern "C" int spy_conv_qkv_store(const void* proj, int proj_dtype, long long ld
     SPY_DISPATCH_DTYPE(proj_dtype, TP, {
         SPY_DISPATCH_DTYPE(q_dtype, TQ, {
             auto run = [&](auto f) { spy_launch(f, grid, dim3(128), 0, stream, (const TP*)proj, (TQ*)q_out, (TQ*)pages, A); };
-            if (vec && taps <= 4) run(conv_qkv_kernel<TP, TQ, 4, 4>);
+            if (vec) run(conv_qkv_kernel<TP, TQ, 4, 4>);
             else if (taps <= 4) run(conv_qkv_kernel<TP, TQ, 1, 4>);
             else run(conv_qkv_kernel<TP, TQ, 1, 16>);
         })

@@ -392,7 +392,8 @@ def _paged_setup(lens, page_size, nkv, hd, dtype, seed=0, planes=2):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,taps,page_size,splits,temp,gate", [
     (4, 2, 16, 24, 3, 8, 1, (0.4, 16), True), (3, 1, 12, 20, 1, 4, 3, None, True), (8, 4, 64, 64, 4, 16, 2, (0.5, 64), True), (20, 1, 7, 5, 5, 8, 1, (1.5, 3), False),
-    (2, 1, 160, 192, 16, 16, 4, (0.2, 7), True), (2, 2, 10, 6, 2, 16, 1, None, False), (16, 2, 128, 128, 4, 16, 1, (0.1, 1), True), (6, 3, 32, 8, 9, 8, 2, (-0.3, 2.5), True)])
+    (2, 1, 160, 192, 16, 16, 4, (0.2, 7), True), (2, 2, 10, 6, 2, 16, 1, None, False), (16, 2, 128, 128, 4, 16, 1, (0.1, 1), True), (6, 3, 32, 8, 9, 8, 2, (-0.3, 2.5), True), (8, 4, 16, 32, 6, 16, 1, (0.5, 16), True),
+    (16, 4, 24, 40, 11, 16, 2, None, True), (4, 4, 64, 64, 16, 16, 1, (0.2, 64), True), (12, 4, 32, 32, 3, 8, 3, None, True)])
 def test_queries_and_cache_rows_behind_the_convolution(dtype, heads, kv_heads, dim, vdim, taps, page_size, splits, temp, gate):
     """Three requests' runs in one step (a long one, one token, a run shorter than the taps), twice in a row, in slots that are not
     in the batch's order: queries, keys and values equal the plain convolution of the whole sequences, the state carries what the second
@@ -1045,7 +1046,7 @@ def random_config(rng):
 
 
 @gpu
-@pytest.mark.parametrize("seed", [3, 11, 19, 27, 42, 58, 77, 91])
+@pytest.mark.parametrize("seed", [3, 11, 19, 27, 42, 58, 77, 91, 1009, 1011, 1020, 1036])
 def test_configurations_drawn_at_random_agree_with_the_plain_model_in_every_cut(tmp_path, seed):
     """Whole, the last 60 tokens one by one, and portions down to two tokens, in both formats; in float32 the cuts agree with each
     other to rounding."""
